@@ -20,7 +20,8 @@ from typing import Optional, Sequence
 @dataclass(frozen=True)
 class NormSpec:
     """A normalisation over the last axis.  kind "rmsnorm": y = x / sqrt(mean(x^2) + eps) * w;
-    kind "layernorm": y = (x - mean(x)) / sqrt(var(x) + eps) * w (no bias).  `weight_offset` c: the
+    kind "layernorm": y = (x - mean(x)) / sqrt(var(x) + eps) * w (+ b with `bias`, a tensor named as the weight with
+    `bias_suffix` added).  `weight_offset` c: the
     stored tensor is w - c (a weight kept around zero with c = 1), so the factor is c + stored."""
 
     dim: int
@@ -31,6 +32,8 @@ class NormSpec:
     # rmsnorm only: the axis is cut into this many equal consecutive parts and each part is divided by
     # its own root mean square; the weight still spans the whole axis
     groups: int = 1
+    bias: bool = False              # layernorm only
+    bias_suffix: str = ".b"
 
 
 @dataclass(frozen=True)
@@ -85,7 +88,9 @@ class LatentAttentionSpec:
     Per head: `nope_dim` unrotated and `rope_dim` rotated query/key channels, values of `v_dim`;
     queries through a latent of `q_rank` (None: straight from the input), keys and values from one
     of `kv_rank`, plus one rotated key part shared by all heads.  `sink`: a learned number per head
-    joins the softmax's denominator.  `gate`: the heads' outputs are multiplied by sigmoid(G h)."""
+    joins the softmax's denominator.  `gate`: the heads' outputs are multiplied by sigmoid(G h).  `position` is a
+    ScaledRotarySpec or a RotaryPairsSpec over the rotated channels.  `names`: pairs (role, tensor name) that replace the
+    mixer's defaults."""
 
     hidden_size: int
     num_heads: int
@@ -96,11 +101,12 @@ class LatentAttentionSpec:
     scale: float
     norm_eps: float
     q_rank: Optional[int] = None
-    position: Optional[ScaledRotarySpec] = None
+    position: Optional[object] = None
     window: Optional[int] = None
     sink: bool = False
     gate: bool = False
     kind: str = "latent_attention"
+    names: tuple = ()
 
 
 @dataclass(frozen=True)
@@ -150,7 +156,8 @@ class AttentionSpec:
     softcap: Optional[float] = None
     sink: bool = False
     names: tuple = ("q_proj.weight", "k_proj.weight", "v_proj.weight", "o_proj.weight", "sink")
-    # A third form, taken when `position` is a RotaryPairsSpec or any of the following is set:
+    # A third form, taken when `position` is a RotaryPairsSpec or a ScaledRotarySpec or any of the following is set (it
+    # takes `bias` too):
     # `value_dim`: the values' size per head where it differs from `head_dim` (the queries' and keys');
     # `whole_qk_norm`: one RMS norm over the whole q projection and one over the whole k projection
     #     (all heads at once, weights named by `norm_names`, eps of `qk_norm`), before the rotation;
@@ -170,6 +177,13 @@ class AttentionSpec:
     # `reads_kv`: the mixer has no key and value tensors: its schedule step reads what another step stored;
     # `cache_window`: how many of the last keys the cache must keep, where that differs from the mixer's own window
     #     (another step with a longer window reads this one's keys); -1: the mixer's window, None: every key.
+    # `difference` c: two softmax maps per head over the same values, subtracted.  q and k have twice the rows (head by head
+    #     map 1, map 2, each of `head_dim` and rotated alike); with lambda = exp(a1 . b1) - exp(a2 . b2) + c (four vectors of
+    #     head_dim, tensors `difference_names`) a head's result is o = map1 - lambda map2, divided by sqrt(mean(o^2) +
+    #     difference_eps) over its value channels and multiplied by 1 - c.
+    difference: Optional[float] = None
+    difference_eps: float = 0.0
+    difference_names: tuple = ("lq1", "lk1", "lq2", "lk2")
     key_weights: str = "softmax"
     key_bias_name: str = "pb"
     conv_taps: Optional[int] = None
@@ -237,6 +251,25 @@ class GeneralDeltaSpec:
 
 
 @dataclass(frozen=True)
+class Mamba2Spec:
+    """A state-space mixer: rows [z | x | B | C | dt] of one product; x, B and C together pass a short causal convolution with a
+    bias, then silu; per head (groups of heads share B and C) S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x with
+    dt = softplus(raw + dt_bias); y times silu(z), then an RMS norm in `norm_groups` equal parts of the row, times a weight,
+    and the output product."""
+
+    hidden_size: int
+    num_heads: int
+    value_dim: int
+    state_dim: int
+    groups: int
+    conv_taps: int
+    norm_groups: int
+    norm_eps: float
+    kind: str = "mamba2"
+    names: tuple = ()          # pairs (role, tensor name) that replace the mixer's defaults
+
+
+@dataclass(frozen=True)
 class TokenSideSpec:
     """A second input chosen by the token, added at the end of a layer: e = table[token][column0 : column0 + dim];
     y = P (gelu_tanh(G x) * e); x <- x + y / sqrt(mean(y^2) + eps) * w.  `names`: G, P and w under the block's prefix.
@@ -275,7 +308,8 @@ class PairEmbeddingSpec:
 
 @dataclass(frozen=True)
 class SwiGLUSpec:
-    """Dense gated feed-forward: down(act(gate(x)) * up(x)); act "silu", "gelu_tanh", "gelu" or "relu".
+    """Dense gated feed-forward: down(act(gate(x)) * up(x)); act "silu", "gelu_tanh", "gelu", "relu" or "swish_clamp", which
+    takes `act_limit` L: g = min(gate, L), u = clamp(up, -L, L), hidden = g sigmoid(1.702 g) (u + 1).
     `names`: the tensors of gate, up and down; with `bias` every projection adds a vector named as
     its matrix with `bias_suffix`."""
 
@@ -286,6 +320,7 @@ class SwiGLUSpec:
     names: tuple = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
     bias: bool = False
     bias_suffix: str = ".b"
+    act_limit: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -339,6 +374,9 @@ class BlockSpec:
     (None: no gates) names two matrices R with biases (R's name + `residual_gate_bias`): gate = sigmoid(R h + b), a
     number per channel, from the same h the sublayer reads; `ffn` may be None; `token_side` adds a token's own second
     input at the layer's end.
+    kind "streams": the residual is `streams` copies X_1 .. X_n; sublayer q (1 the mixer, 2 the feed-forward, which may be
+    None) computes u = sum_s in[s] X_s, y = sublayer(norm(u)), X_t <- sum_s mix[s, t] X_s + out[t] y; its three tensors are
+    `stream_names` formatted with q.  Every block of a model has the same number of copies (`ModelSpec.streams`).
     `names` maps the block's local part names to the sub-prefixes used in tensor names.
     """
 
@@ -355,6 +393,8 @@ class BlockSpec:
     residual_gates: Optional[tuple] = None
     residual_gate_bias: str = ".b"
     token_side: Optional[TokenSideSpec] = None
+    streams: int = 1
+    stream_names: tuple = ("hc{q}.in", "hc{q}.out", "hc{q}.mix")
     names: tuple = (
         ("norm1", "input_layernorm"),
         ("mixer", "self_attn"),
@@ -408,9 +448,19 @@ class ModelSpec:
     logit_softcap: Optional[float] = None
     # (tensor name, columns): a second table [vocab, columns] of which blocks with a `token_side` read their columns
     token_side_table: Optional[tuple] = None
+    # n: the residual is n copies of the stream, all equal to the embedding at the start and summed before the final norm
+    # (blocks of kind "streams"); None: one stream
+    streams: Optional[int] = None
     extra: dict = field(default_factory=dict)     # free for an architecture's own model class
 
 
 def identity_schedule(n: int) -> tuple:
     """Every layer once, in order, each with its own cache entry."""
     return tuple(ScheduleStep(i) for i in range(n))
+
+
+def looped_schedule(n: int, start: int, stop: int, times: int) -> tuple:
+    """Layers 0 .. start - 1 once, start .. stop - 1 `times` times in a row, the rest once; every run of a layer has a
+    cache entry of its own."""
+    order = list(range(start)) + list(range(start, stop)) * times + list(range(stop, n))
+    return tuple(ScheduleStep(i) for i in order)

@@ -30,9 +30,10 @@ extern "C" {
 
 // attention_decode.cu: decode attention over the paged cache (one query per sequence, keys cut into splits)
 long long hb_attention_decode_scratch_floats(int n_seqs, int nh, int hd, int nsplit);
-int hb_attention_decode_bf16(const void* q, int ldq, void* out, int ldo, const void* kcache, const void* vcache,
-    const int* seq_len, const int* seq_pages, int pages_stride, float* scratch, int n_seqs, int nh, int nkv, int hd,
-    int page_size, int nsplit, float scale, int window, float softcap, const float* sink, const float* gate_bias, const float* out_gate, int ldg, void* stream);
+int hb_attention_decode_bf16(const void* q, int ldq, void* out, int ldo, const void* kcache, const void* vcache, const
+    int* seq_len, const int* seq_pages, int pages_stride, float* scratch, int n_seqs, int nh, int nkv, int hd, int
+    page_size, int nsplit, float scale, int window, float softcap, const float* sink, const float* gate_bias, const
+    float* out_gate, int ldg, float diff_lambda, float diff_factor, float diff_eps, int diff_dv, void* stream);
 int hb_attention_decode_fused_bf16(const void* qkv, int ld, void* out, int ldo, void* kcache, void* vcache,
     const float* qw, const float* kw, float eps, const float* cos_tab, const float* sin_tab, int table_rows,
     int write_cache, const int* seq_len, const int* seq_pages, int pages_stride, float* scratch, int*
@@ -41,22 +42,25 @@ int hb_attention_decode_fused_bf16(const void* qkv, int ld, void* out, int ldo, 
 // attention_prefill.cu: prefill attention, mma.sync flash form, head sizes in steps of 16 up to 256
 int hb_attention_prefill_bf16(const void* q, int ldq, void* out, int ldo, const void* kcache, const void* vcache,
     const int* seq_start, const int* seq_pos0, const int* seq_pages, int pages_stride, int n_seqs, int max_q_len, int
-    nh, int nkv, int hd, int page_size, float scale, int window, float softcap, const float* sink, const float* gate_bias, const float* out_gate, int ldg, void* stream);
+    nh, int nkv, int hd, int page_size, float scale, int window, float softcap, const float* sink, const float*
+    gate_bias, const float* out_gate, int ldg, int out_f32, void* stream);
 
 // attention_prefill_tc.cu: prefill attention on tcgen05 tensor cores, head sizes 64 and 128
-int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens, void* out, int ldo, const void* kcache,
-    const void* vcache, int n_pages, const int* seq_start, const int* seq_pos0, const int* seq_pages, int
-    pages_stride, int n_seqs, int max_q_len, int nh, int nkv, int hd, int page_size, float scale, int window, float
-    softcap, const float* sink, const float* gate_bias, const float* out_gate, int ldg, int* error_flag, int* work_counter, void* stream);
+int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens, void* out, int ldo, const void* kcache, const
+    void* vcache, int n_pages, const int* seq_start, const int* seq_pos0, const int* seq_pages, int pages_stride, int
+    n_seqs, int max_q_len, int nh, int nkv, int hd, int page_size, float scale, int window, float softcap, const
+    float* sink, const float* gate_bias, const float* out_gate, int ldg, int out_f32, int* error_flag, int*
+    work_counter, void* stream);
 
 // attention_simt.cu: attention of any shape on the CUDA cores (the 32-bit path)
-int hb_attention_simt(int dtype, const void* q, int ldq, void* out, int ldo, const void* kcache, const void*
-    vcache, const int* tok_seq, const int* tok_pos, const int* seq_pages, int pages_stride, int n_tokens, int nh, int
-    nkv, int hd, int page_size, float scale, int window, float softcap, const float* sink, const float* gate_bias, const float* out_gate, int ldg, void* stream);
+int hb_attention_simt(int dtype, const void* q, int ldq, void* out, int ldo, const void* kcache, const void* vcache,
+    const int* tok_seq, const int* tok_pos, const int* seq_pages, int pages_stride, int n_tokens, int nh, int nkv, int
+    hd, int page_size, float scale, int window, float softcap, const float* sink, const float* gate_bias, const float*
+    out_gate, int ldg, int out_f32, void* stream);
 
 // elementwise.cu: embedding, RMSNorm, SwiGLU, head norm + rotation + cache write, residual sum, shared-norm finish
-int hb_embed(int dtype, const void* table, const int* ids, float* out, int n_tokens, int hidden, int vocab, float
-    scale, const void* pos_table, const int* positions, int n_positions, void* stream);
+int hb_embed(int dtype, const void* table, const int* ids, float* out, int copies, int n_tokens, int hidden, int
+    vocab, float scale, const void* pos_table, const int* positions, int n_positions, void* stream);
 int hb_rmsnorm(int dtype, const float* x, const float* w, void* out, const int* rows, int n_rows, int dim,
     float eps, void* stream);
 int hb_swiglu(int dtype, const void* gu, int ld, void* out, int ldo, int n_tokens, int inter, int interleave,
@@ -86,8 +90,8 @@ int hb_gemm_simt(int dtype, const void* A, int lda, const void* W, int ldw, void
     int K, int epi, void* stream);
 
 // gemm_skinny.cu: decode product (at most 64 activation rows), mma.sync, optional shared norm
-int hb_gemm_skinny_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K,
-    int epi, void* stream);
+int hb_gemm_skinny_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K, int
+    epi, float glu_limit, void* stream);
 int hb_gemm_skinny_norm_parts(int M, int N);
 int hb_gemm_skinny_norm_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N,
     int K, int epi, const float* in_sumsq, int in_parts, float in_eps, const float* out_w, void* out_xw, int
@@ -96,17 +100,17 @@ int hb_gemm_skinny_norm_bf16(const void* A, int lda, const void* W, int ldw, voi
 // gemm_stream.cu: decode product, TMA + tcgen05, K slices (the output head)
 long long hb_gemm_stream_scratch_floats(int M, int N, int K);
 int hb_gemm_stream_counters(int N);
-int hb_gemm_stream_bf16(const void* X, int ldx, const void* W, int ldw, void* C, int ldc, int M, int N, int K,
-    int epi, float* scratch, long long scratch_floats, int* counters, int n_counters, int* error_flag, void*
-    stream);
+int hb_gemm_stream_bf16(const void* X, int ldx, const void* W, int ldw, void* C, int ldc, int M, int N, int K, int
+    epi, float glu_limit, float* scratch, long long scratch_floats, int* counters, int n_counters, int* error_flag,
+    void* stream);
 
 // gemm_tcgen05.cu: prefill product, TMA + tcgen05, persistent; optional shared norm
 int hb_gemm_tcgen05_set_pairs(int on);
 int hb_gemm_tcgen05_set_ksplit(int on);
 long long hb_gemm_tcgen05_workspace_floats(int ctas);
 int hb_gemm_tcgen05_set_workspace(float* floats, int* counters, int ctas);
-int hb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int
-    K, int epi, int* error_flag, void* stream);
+int hb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K, int
+    epi, float glu_limit, int* error_flag, void* stream);
 int hb_gemm_tcgen05_grouped_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M_max, int
     N, int K, int E, int epi, float glu_limit, const int* rows_used, const int* tile_expert, int* error_flag, void*
     stream);
@@ -131,12 +135,12 @@ int hb_gla_output(int dtype, const float* o, int ldo, const float* w, float eps,
     void* y, int ldy, int n_tokens, int heads, int dv, void* stream);
 
 // latent_attention.cu: attention over a cached latent (one shared key/value vector per token), with a sink
-int hb_latent_kv_store(int dtype, const float* kv, int ld, const float* norm_w, float eps, const float* freq,
-    float mscale, int rank, int rot, const int* tok_seq, const int* tok_pos, const int* seq_pages, int
+int hb_latent_kv_store(int dtype, const float* kv, int ld, const float* norm_w, float eps, const float* freq, float
+    mscale, int halves, int rank, int rot, const int* tok_seq, const int* tok_pos, const int* seq_pages, int
     pages_stride, void* cache, int n_tokens, int page_size, void* stream);
 int hb_rotate_heads(const float* in, int ld_in, int in_head_stride, int in_offset, float* out, int ld_out, int
-    out_head_stride, int out_offset, const float* freq, float mscale, const int* tok_pos, int n_tokens, int
-    heads, int rot, float scale, void* stream);
+    out_head_stride, int out_offset, const float* freq, float mscale, int halves, const int* tok_pos, int n_tokens,
+    int heads, int rot, float scale, void* stream);
 int hb_headwise_gemm(int dtype, int out_dtype, const float* in, int ld_in, int in_head_stride, const void* w,
     void* out, int ld_out, int out_head_stride, const float* gate, int ld_gate, int n_tokens, int heads, int K,
     int N, float scale, void* stream);
@@ -150,9 +154,9 @@ int hb_latent_attention_mma_bf16(const float* q, int ldq, float* out, int ldo, c
     stream);
 long long hb_latent_attention_mma_scratch_floats(int n_seqs, int max_q_len, int heads, int rank, int nsplit);
 
-// layernorm.cu: layer normalisation (weight, no bias), alone and with the scaled residual sum after it
-int hb_layernorm(int dtype, const float* x, const float* w, void* out, const int* rows, int n_rows, int dim,
-    float eps, void* stream);
+// layernorm.cu: layer normalisation (alone with an optional bias), alone and with the scaled residual sum after it
+int hb_layernorm(int dtype, const float* x, const float* w, const float* bias, void* out, const int* rows, int n_rows,
+    int dim, float eps, void* stream);
 int hb_layernorm_residual(int dtype, const float* y, int ldy, const float* w, const float* scale, float* x, void*
     h, int n_rows, int dim, float eps, void* stream);
 
@@ -193,14 +197,14 @@ int hb_group_rmsnorm(int dtype, const float* x, const float* w, void* out, const
 int hb_group_rmsnorm_residual(int dtype, const float* y, int ldy, const float* z, int ldz, float a, float b,
     const float* bias, const float* w, float* x, void* h, int n_rows, int dim, int groups, float eps, void* stream);
 int hb_axpby(float* y, int ldy, float a, const float* z, int ldz, float b, int rows, int cols, void* stream);
-int hb_bias_glu(int dtype, const float* gu, int ld, const float* bias, void* out, int ldo, int n_tokens, int
-    inter, int interleave, int act, void* stream);
+int hb_bias_glu(int dtype, const float* gu, int ld, const float* bias, void* out, int ldo, int n_tokens, int inter,
+    int interleave, int act, float limit, void* stream);
 int hb_tanh_cap(float* x, int ld, float cap, int rows, int cols, void* stream);
 
 // short_conv.cu: a short causal convolution over time whose last inputs are state; an embedding plus a row chosen by (previous token, token)
-int hb_short_conv(int out_dtype, const float* in, int ld_in, const float* w, float* state, const int* seq_slot,
-    const int* seq_start, const int* seq_pos0, void* out, int ldo, int n_seqs, int max_q_len, int channels, int
-    taps, int add_input, int act_silu, void* stream);
+int hb_short_conv(int out_dtype, const float* in, int ld_in, const float* w, const float* bias, float* state, const
+    int* seq_slot, const int* seq_start, const int* seq_pos0, void* out, int ldo, int n_seqs, int max_q_len, int
+    channels, int taps, int add_input, int act_silu, void* stream);
 int hb_pair_embed(int dtype, const void* table, const void* pair_table, const int* ids, const int* tok_seq,
     const int* tok_pos, const int* seq_slot, const int* seq_start, int* last_id, float* out, int n_tokens, int
     hidden, int vocab, int buckets, long long mul_prev, long long mul_cur, float scale, void* stream);
@@ -213,16 +217,19 @@ int hb_delta_prepare(float* qk, int ld, int q_off, int k_off, int qk_heads, int 
 int hb_linear_scan(int delta, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const
     float* gates, const float* decay, float* state, const int* seq_slot, const int* seq_start, float* out, int ldo,
     int n_seqs, int max_q_len, int heads, int qk_heads, int dk, int dv, void* stream);
-int hb_gated_rmsnorm(int dtype, const float* o, int ldo, const float* w, float eps, const float* gate, int ldg,
-    void* y, int ldy, int n_tokens, int units, int n, int act, int w_stride, void* stream);
+int hb_gated_rmsnorm(int dtype, const float* o, int ldo, const float* w, float eps, const float* gate, int ldg, void*
+    y, int ldy, int n_tokens, int units, int n, int act, int w_stride, int gate_first, void* stream);
 
 // rotary_pairs.cu: whole-projection q/k norm, rotation of pairs by position (q, k and v), cache write; the turn back of the results
-int hb_qkv_rotary_cache(int dtype, const float* rows, int ld, const float* wq, const float* wk, float eps, int
-    whole_norm, const float* fqk, int rot, int halves, const float* fv, const int* tok_seq, const int* tok_pos,
-    const int* seq_pages, int pages_stride, void* q_out, int ldq, void* kcache, void* vcache, int n_tokens, int nh,
-    int nkv, int dk, int dv, int hd, int page_size, int write_cache, void* stream);
+int hb_qkv_rotary_cache(int dtype, const float* rows, int ld, const float* bias, const float* wq, const float* wk,
+    float eps, int whole_norm, const float* fqk, int rot, int halves, float mscale, const float* fv, const int*
+    tok_seq, const int* tok_pos, const int* seq_pages, int pages_stride, void* q_out, int ldq, void* kcache, void*
+    vcache, int n_tokens, int nh, int nkv, int maps, int dk, int dv, int hd, int page_size, int write_cache, void*
+    stream);
 int hb_rotate_heads_back(int dtype, const void* att, int ld, int hd, const float* fv, int halves, const int*
     tok_pos, void* y, int ldy, int n_tokens, int nh, int dv, void* stream);
+int hb_difference_heads(int dtype, const float* att, int ld, int hd, float lambda, float factor, float eps, void* y,
+    int ldy, int n_tokens, int nh, int dv, void* stream);
 int hb_head_gate(int dtype, const void* att, int ld, int hd, const float* gate, int ldg, void* y, int ldy, int
     n_tokens, int nh, int dv, void* stream);
 
@@ -238,6 +245,21 @@ int hb_gated_norm_residual(int dtype, const float* y, int ldy, const float* z, i
     w, float eps, float* x, const float* w2, float eps2, void* h, int n_rows, int D, void* stream);
 int hb_token_gate(int dtype, const float* s, int lds, const void* table, int ldt, int col0, const int* ids, void*
     out, int ldo, int n_tokens, int m, int vocab, void* stream);
+
+// streams.cu: a residual stream of several copies: result in, next input out, with its norm
+int hb_streams_join(int dtype, float* x, int n, const float* y, int ldy, const float* mix, const float* out_w, const
+    float* in_w, const float* w, const float* bias, float eps, int rms, void* h, const int* rows, int n_rows, int D,
+    void* stream);
+
+// state_space.cu: a state-space recurrence with one decay and step size per token and head
+int hb_ssd_scan(int dtype, const void* xbc, int ld, int b_off, int c_off, const float* dt, int lddt, const float*
+    dt_bias, const float* a_log, const float* dskip, float* state, const int* seq_slot, const int* seq_start, float*
+    out, int ldo, int n_seqs, int heads, int groups, int N, int dv, void* stream);
+int hb_ssd_chunks(int n_tokens, int n_seqs, int N, int dv);
+int hb_ssd_chunked_bf16(const void* xbc, int ld, int b_off, int c_off, const float* dt, int lddt, const float*
+    dt_bias, const float* a_log, const float* dskip, float* state, const int* seq_slot, const int* seq_start, float*
+    out, int ldo, int n_seqs, int max_q_len, int heads, int groups, int N, int dv, float* chunk_state, float*
+    chunk_decay, void* stream);
 
 #ifdef __cplusplus
 }

@@ -689,6 +689,50 @@ __global__ void attention_decode_combine_kernel(const float* __restrict__ part_o
   }
 }
 
+// The same for two attention maps of a head (query heads 2h and 2h + 1 over the same values), subtracted and normed:
+// o = a1 - lambda a2, out[b][h][:dv] = o / sqrt(mean(o^2) + eps) * factor over the dv value channels.
+struct DecodeDifference {
+  float lambda, factor, eps;
+  int dv;                    // 0: every query head on its own
+};
+__global__ void attention_decode_difference_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                   bf16* __restrict__ out, int ldo, int nh, int hd, int nsplit,
+                                                   DecodeDifference df) {
+  extern __shared__ float sh[];          // [2][nsplit] factors of the key ranges, then [dv]
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch();
+  const int h = blockIdx.x, b = blockIdx.y;
+  const size_t base = ((size_t)b * nh + 2 * h) * nsplit;
+  float* row = sh + 2 * nsplit;
+  if (threadIdx.x < 64) {
+    const int map = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float* ml = part_ml + (base + (size_t)map * nsplit) * 2;
+    float mm = -INFINITY, ll = 0.0f;
+    for (int s = lane; s < nsplit; s += 32) mm = fmaxf(mm, ml[2 * s]);
+    mm = warp_max(mm);
+    for (int s = lane; s < nsplit; s += 32)
+      if (ml[2 * s] != -INFINITY) ll += __expf(ml[2 * s] - mm) * ml[2 * s + 1];
+    ll = warp_sum(ll);
+    const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * (map ? -df.lambda : 1.0f);
+    for (int s = lane; s < nsplit; s += 32) sh[map * nsplit + s] = ml[2 * s] == -INFINITY ? 0.0f : __expf(ml[2 * s] - mm) * inv;
+  }
+  __syncthreads();
+  float ss = 0.0f;
+  for (int d = threadIdx.x; d < df.dv; d += blockDim.x) {
+    float acc = 0.0f;
+    for (int s = 0; s < 2 * nsplit; ++s) {
+      const float f = sh[s];
+      if (f != 0.0f) acc = fmaf(f, part_o[(base + s) * hd + d], acc);
+    }
+    row[d] = acc;
+    ss = fmaf(acc, acc, ss);
+  }
+  ss = block_sum(ss, red);
+  const float k = df.factor / sqrtf(ss / (float)df.dv + df.eps);
+  for (int d = threadIdx.x; d < df.dv; d += blockDim.x) out[(size_t)b * ldo + (size_t)h * df.dv + d] = __float2bfloat16_rn(row[d] * k);
+}
+
 static int decode_smem_bytes(int hd, int stages) {
   const int pipeline = stages * 2 * AD_TILE * (hd * 2 + 16);
   const int merge = (2 * AD_WARPS * 16 + AD_WARPS * 16 * hd) * 4;
@@ -708,7 +752,7 @@ extern "C" int hb_attention_decode_bf16(const void* q, int ldq, void* out, int l
                                         int pages_stride, float* scratch, int n_seqs, int nh, int nkv, int hd,
                                         int page_size, int nsplit, float scale, int window, float softcap,
                                         const float* sink, const float* gate_bias, const float* out_gate, int ldg,
-                                        void* stream) {
+                                        float diff_lambda, float diff_factor, float diff_eps, int diff_dv, void* stream) {
   HB_REQUIRE(n_seqs > 0 && nh > 0 && nkv > 0 && hd > 0, "attention_decode: sizes must be positive");
   HB_REQUIRE(softcap >= 0.0f, "attention_decode: the cap on the scores must be >= 0 (0: none)");
   HB_REQUIRE(gate_bias == nullptr || sink == nullptr, "attention_decode: sigmoid weights have no sink");
@@ -720,6 +764,8 @@ extern "C" int hb_attention_decode_bf16(const void* q, int ldq, void* out, int l
   HB_REQUIRE(ldq % 2 == 0 && ((uintptr_t)q & 3) == 0, "attention_decode: queries must be 4-byte aligned");
   HB_REQUIRE(((uintptr_t)kcache & 15) == 0 && ((uintptr_t)vcache & 15) == 0, "attention_decode: cache must be 16-byte aligned");
   HB_REQUIRE(window >= 0, "attention_decode: window must be >= 0");
+  HB_REQUIRE(diff_dv == 0 || (diff_dv > 0 && diff_dv <= hd && nh % 2 == 0 && sink == nullptr && gate_bias == nullptr && out_gate == nullptr && nsplit <= 1024),
+             "attention_decode: the difference of two maps takes pairs of query heads, no sink, no gate, no sigmoid weights");
   HB_REQUIRE((long long)pages_stride * (page_size / AD_TILE) <= (long long)AD_MAX_TILES * nsplit,
              "attention_decode: %d pages per sequence in %d splits exceed %d tiles per CTA", pages_stride, nsplit, AD_MAX_TILES);
   cudaStream_t s = (cudaStream_t)stream;
@@ -755,6 +801,13 @@ extern "C" int hb_attention_decode_bf16(const void* q, int ldq, void* out, int l
     hb_launch(attention_decode_kernel<256>, dim3(grid), dim3(AD_THREADS), smem, s, a);
   }
   HB_CHECK_LAUNCH("attention_decode");
+  if (diff_dv > 0) {
+    const DecodeDifference df{diff_lambda, diff_factor, diff_eps, diff_dv};
+    hb_launch(attention_decode_difference_kernel, dim3(nh / 2, n_seqs), dim3(128), (size_t)(2 * nsplit + diff_dv) * sizeof(float), s, part_o,
+              part_ml, (bf16*)out, ldo, nh, hd, nsplit, df);
+    HB_CHECK_LAUNCH("attention_decode_difference");
+    return 0;
+  }
   dim3 cgrid(nh, n_seqs);
   hb_launch(attention_decode_combine_kernel, dim3(cgrid), dim3(hd >= 128 ? 128 : 64), 0, s, part_o, part_ml, (bf16*)out, ldo, nh, hd, nsplit, sink, gate_bias != nullptr ? 1 : 0,
             out_gate, ldg);

@@ -45,6 +45,7 @@ struct PrefillArgs {
   const float* gate_bias;  // [nh] or null.  Not null: no softmax; a visible key weighs sigmoid(score + gate_bias[h]) as it is
   const float* out_gate;   // [tokens, ldg] or null: head h's result of a token is multiplied by sigmoid(out_gate[token * ldg + h])
   int ldg;
+  int out_f32;             // the output is float (something follows before it is rounded)
 };
 
 template <int HDM>
@@ -261,6 +262,19 @@ __global__ void __launch_bounds__(AP_THREADS) attention_prefill_kernel(PrefillAr
     if (v0) inv0 *= 1.0f / (1.0f + expf(-a.out_gate[(size_t)(row0 + qi0) * a.ldg + h]));
     if (v1) inv1 *= 1.0f / (1.0f + expf(-a.out_gate[(size_t)(row0 + qi1) * a.ldg + h]));
   }
+  if (a.out_f32) {
+    float* f0 = reinterpret_cast<float*>(a.out) + (size_t)(row0 + qi0) * a.ldo + (size_t)h * hd;
+    float* f1 = reinterpret_cast<float*>(a.out) + (size_t)(row0 + qi1) * a.ldo + (size_t)h * hd;
+#pragma unroll
+    for (int nd = 0; nd < HDM / 8; ++nd) {
+      if (nd * 8 < hd) {
+        const int d = nd * 8 + 2 * t;
+        if (v0) *reinterpret_cast<float2*>(f0 + d) = make_float2(o[nd][0] * inv0, o[nd][1] * inv0);
+        if (v1) *reinterpret_cast<float2*>(f1 + d) = make_float2(o[nd][2] * inv1, o[nd][3] * inv1);
+      }
+    }
+    return;
+  }
   bf16* o0 = a.out + (size_t)(row0 + qi0) * a.ldo + (size_t)h * hd;
   bf16* o1 = a.out + (size_t)(row0 + qi1) * a.ldo + (size_t)h * hd;
 #pragma unroll
@@ -277,14 +291,14 @@ extern "C" int hb_attention_prefill_bf16(const void* q, int ldq, void* out, int 
                                          const void* vcache, const int* seq_start, const int* seq_pos0,
                                          const int* seq_pages, int pages_stride, int n_seqs, int max_q_len,
                                          int nh, int nkv, int hd, int page_size, float scale, int window, float softcap,
-                                         const float* sink, const float* gate_bias, const float* out_gate, int ldg,
+                                         const float* sink, const float* gate_bias, const float* out_gate, int ldg, int out_f32,
                                          void* stream) {
   HB_REQUIRE(n_seqs > 0 && max_q_len > 0 && nh > 0 && nkv > 0 && hd > 0, "attention_prefill: sizes must be positive");
   HB_REQUIRE(nh % nkv == 0, "attention_prefill: %d query heads are not a multiple of %d key/value heads", nh, nkv);
   HB_REQUIRE(hd % 16 == 0 && hd <= 256, "attention_prefill: head size %d must be a multiple of 16, at most 256", hd);
   HB_REQUIRE(page_size % AP_TILE == 0, "attention_prefill: page size %d must be a multiple of %d", page_size, AP_TILE);
-  HB_REQUIRE(ldq % 2 == 0 && ldo % 2 == 0 && ((uintptr_t)q & 3) == 0 && ((uintptr_t)out & 3) == 0,
-             "attention_prefill: queries and output must be 4-byte aligned");
+  HB_REQUIRE(ldq % 2 == 0 && ldo % 2 == 0 && ((uintptr_t)q & 3) == 0 && ((uintptr_t)out & 3) == 0 && (!out_f32 || ((uintptr_t)out & 7) == 0),
+             "attention_prefill: queries and output must be 4-byte aligned (a float output 8-byte)");
   HB_REQUIRE(((uintptr_t)kcache & 15) == 0 && ((uintptr_t)vcache & 15) == 0, "attention_prefill: cache must be 16-byte aligned");
   HB_REQUIRE(nh <= 65535 && n_seqs <= 65535, "attention_prefill: grid too large");
   HB_REQUIRE(softcap >= 0.0f, "attention_prefill: the cap on the scores must be >= 0 (0: none)");
@@ -298,7 +312,7 @@ extern "C" int hb_attention_prefill_bf16(const void* q, int ldq, void* out, int 
     smem = stages * 2 * AP_TILE * (hd * 2 + 16);
   }
   PrefillArgs a{(const bf16*)q, ldq, (bf16*)out, ldo, (const bf16*)kcache, (const bf16*)vcache, seq_start, seq_pos0,
-                seq_pages, pages_stride, nh, nkv, hd, page_size, scale, window, stages, softcap, sink, gate_bias, out_gate, ldg};
+                seq_pages, pages_stride, nh, nkv, hd, page_size, scale, window, stages, softcap, sink, gate_bias, out_gate, ldg, out_f32};
   dim3 grid(ceil_div(max_q_len, AP_QTILE), nh, n_seqs);
   cudaStream_t s = (cudaStream_t)stream;
   cudaError_t e;

@@ -57,6 +57,7 @@ struct PrefillTcArgs {
   const float* gate_bias;  // [nh] or null.  Not null: sigmoid weights (see the head of this file)
   const float* out_gate;   // [tokens, ldg] or null: head h's result of a token is multiplied by sigmoid(out_gate[token * ldg + h])
   int ldg;
+  int out_f32;             // the output is float (something follows before it is rounded)
 };
 
 // One unit of work: 128 consecutive queries of two heads (or one) of one key/value head of one sequence.
@@ -456,6 +457,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         float inv = gated ? 1.0f : (l > 0.0f ? 1.0f / l : 0.0f);
         if (a.out_gate != nullptr && valid) inv *= 1.0f / (1.0f + expf(-a.out_gate[(size_t)(it.row0 + qi) * a.ldg + it.h0 + t]));
         bf16* dst = a.out + (size_t)(it.row0 + qi) * a.ldo + (size_t)(it.h0 + t) * HD;
+        float* dst_f = reinterpret_cast<float*>(a.out) + (size_t)(it.row0 + qi) * a.ldo + (size_t)(it.h0 + t) * HD;
 #pragma unroll
         for (int cc = 0; cc < HD / 32; ++cc) {
           float o[32];
@@ -467,7 +469,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             __syncwarp();
             if (lane == 0) mbar_arrive_cta(bar(19 + t));
           }
-          if (valid) {
+          if (valid && a.out_f32) {
+#pragma unroll
+            for (int i = 0; i < 32; i += 4)
+              *reinterpret_cast<float4*>(dst_f + cc * 32 + i) = make_float4(o[i] * inv, o[i + 1] * inv, o[i + 2] * inv, o[i + 3] * inv);
+          } else if (valid) {
 #pragma unroll
             for (int i = 0; i < 32; i += 8) {
               unsigned w[4];
@@ -497,7 +503,7 @@ extern "C" int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens
                                             const void* vcache, int n_pages, const int* seq_start, const int* seq_pos0,
                                             const int* seq_pages, int pages_stride, int n_seqs, int max_q_len, int nh,
                                             int nkv, int hd, int page_size, float scale, int window, float softcap,
-                                            const float* sink, const float* gate_bias, const float* out_gate, int ldg,
+                                            const float* sink, const float* gate_bias, const float* out_gate, int ldg, int out_f32,
                                             int* error_flag, int* work_counter, void* stream) {
   HB_REQUIRE(n_seqs > 0 && max_q_len > 0 && nh > 0 && nkv > 0 && n_tokens > 0 && n_pages > 0, "attention_prefill_tc: sizes must be positive");
   HB_REQUIRE(hd == 64 || hd == 128, "attention_prefill_tc: head size %d is not 64 or 128", hd);
@@ -521,7 +527,7 @@ extern "C" int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens
   if (rc) return rc;
   const int q_tiles = ceil_div(max_q_len, PT_Q);
   PrefillTcArgs a{(bf16*)out, ldo, seq_start, seq_pos0, seq_pages, pages_stride, nh, nkv, page_size,
-                  scale * 1.4426950408889634f, window, error_flag, n_seqs, q_tiles, work_counter, softcap, sink, gate_bias, out_gate, ldg};
+                  scale * 1.4426950408889634f, window, error_flag, n_seqs, q_tiles, work_counter, softcap, sink, gate_bias, out_gate, ldg, out_f32};
   cudaStream_t s = (cudaStream_t)stream;
   const int pairs = (nh / nkv + 1) / 2;
   const long long items = (long long)q_tiles * n_seqs * nkv * pairs;

@@ -41,6 +41,7 @@ struct AttnArgs {
   const float* gate_bias;
   const float* out_gate;   // [n_tokens, ldg] or null: head h's result of token t is multiplied by sigmoid(out_gate[t * ldg + h])
   int ldg;
+  int out_f32;              // the output is float whatever the activation type (something follows before it is rounded)
 };
 
 template <typename T>
@@ -108,10 +109,13 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attention_simt_kernel(AttnArgs
   float inv = gated ? 1.0f : (l > 0.0f ? 1.0f / l : 0.0f);
   if (a.out_gate != nullptr) inv *= 1.0f / (1.0f + expf(-a.out_gate[(size_t)t * a.ldg + h]));
   T* op = (T*)a.out + (size_t)t * a.ldo + (size_t)h * a.hd;
+  float* of = (float*)a.out + (size_t)t * a.ldo + (size_t)h * a.hd;
 #pragma unroll
   for (int i = 0; i < ATT_MAX_HD / 32; ++i) {
     const int d = lane + 32 * i;
-    if (d < a.hd) op[d] = from_f32<T>(o[i] * inv);
+    if (d >= a.hd) continue;
+    if (a.out_f32) of[d] = o[i] * inv;
+    else op[d] = from_f32<T>(o[i] * inv);
   }
 }
 
@@ -119,7 +123,7 @@ extern "C" int hb_attention_simt(int dtype, const void* q, int ldq, void* out, i
                                  const void* vcache, const int* tok_seq, const int* tok_pos,
                                  const int* seq_pages, int pages_stride, int n_tokens, int nh, int nkv,
                                  int hd, int page_size, float scale, int window, float softcap, const float* sink,
-                                 const float* gate_bias, const float* out_gate, int ldg, void* stream) {
+                                 const float* gate_bias, const float* out_gate, int ldg, int out_f32, void* stream) {
   HB_REQUIRE(n_tokens > 0 && nh > 0 && nkv > 0 && hd > 0 && page_size > 0, "attention: sizes must be positive");
   HB_REQUIRE(nh % nkv == 0, "attention: %d query heads are not a multiple of %d key/value heads", nh, nkv);
   HB_REQUIRE(hd <= ATT_MAX_HD, "attention: head size %d exceeds the supported maximum %d", hd, ATT_MAX_HD);
@@ -127,7 +131,7 @@ extern "C" int hb_attention_simt(int dtype, const void* q, int ldq, void* out, i
   HB_REQUIRE(softcap >= 0.0f, "attention: the cap on the scores must be >= 0 (0: none)");
   HB_REQUIRE(gate_bias == nullptr || sink == nullptr, "attention: sigmoid weights have no sink");
   AttnArgs a{q, ldq, out, ldo, kcache, vcache, tok_seq, tok_pos, seq_pages, pages_stride,
-             n_tokens, nh, nkv, hd, page_size, scale, window, softcap, sink, gate_bias, out_gate, ldg};
+             n_tokens, nh, nkv, hd, page_size, scale, window, softcap, sink, gate_bias, out_gate, ldg, out_f32};
   const long long blocks = ceil_div_ll((long long)n_tokens * nh, ATT_WARPS);
   HB_REQUIRE(blocks < 2147483647LL, "attention: too many (token, head) pairs");
   if (dtype == HB_F32)

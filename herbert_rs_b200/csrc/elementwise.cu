@@ -15,15 +15,15 @@
 // ---------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                             float* __restrict__ out, int hidden, int vocab, float scale,
+                             float* __restrict__ out, int copies, int hidden, int vocab, float scale,
                              const T* __restrict__ pos_table, const int* __restrict__ positions, int n_positions) {
   pdl_wait();
   pdl_launch();
   const int t = blockIdx.x;
   const int id = ids[t];
-  float* o = out + (size_t)t * hidden;
+  float* o = out + (size_t)t * copies * hidden;      // a stream of several copies starts from equal ones
   if (id < 0 || id >= vocab) {  // the host validates ids; an invalid one yields zeros, never a stray read
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = 0.0f;
+    for (int i = threadIdx.x; i < copies * hidden; i += blockDim.x) o[i] = 0.0f;
     return;
   }
   const T* row = table + (size_t)id * hidden;
@@ -37,27 +37,27 @@ __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict_
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     float v = to_f32(row[i]) * scale;
     if (prow) v += to_f32(prow[i]);
-    o[i] = v;
+    for (int c = 0; c < copies; ++c) o[(size_t)c * hidden + i] = v;
   }
 }
 
 template <typename T>
-static int embed_launch(const void* table, const int* ids, float* out, int n_tokens, int hidden,
+static int embed_launch(const void* table, const int* ids, float* out, int copies, int n_tokens, int hidden,
                         int vocab, float scale, const void* pos_table, const int* positions, int n_positions, void* stream) {
-  HB_REQUIRE(n_tokens > 0 && hidden > 0 && vocab > 0, "embed: sizes must be positive");
+  HB_REQUIRE(n_tokens > 0 && hidden > 0 && vocab > 0 && copies > 0, "embed: sizes must be positive");
   HB_REQUIRE(pos_table == nullptr || (positions != nullptr && n_positions > 0), "embed: a position table needs positions");
   int threads = hidden >= 1024 ? 256 : 128;
-  hb_launch(embed_kernel<T>, dim3(n_tokens), dim3(threads), 0, (cudaStream_t)stream, (const T*)table, ids, out, hidden, vocab, scale,
+  hb_launch(embed_kernel<T>, dim3(n_tokens), dim3(threads), 0, (cudaStream_t)stream, (const T*)table, ids, out, copies, hidden, vocab, scale,
             (const T*)pos_table, positions, n_positions);
   HB_CHECK_LAUNCH("embed");
   return 0;
 }
 
-extern "C" int hb_embed(int dtype, const void* table, const int* ids, float* out, int n_tokens,
+extern "C" int hb_embed(int dtype, const void* table, const int* ids, float* out, int copies, int n_tokens,
                         int hidden, int vocab, float scale, const void* pos_table, const int* positions,
                         int n_positions, void* stream) {
-  return dtype == HB_F32 ? embed_launch<float>(table, ids, out, n_tokens, hidden, vocab, scale, pos_table, positions, n_positions, stream)
-                         : embed_launch<bf16>(table, ids, out, n_tokens, hidden, vocab, scale, pos_table, positions, n_positions, stream);
+  return dtype == HB_F32 ? embed_launch<float>(table, ids, out, copies, n_tokens, hidden, vocab, scale, pos_table, positions, n_positions, stream)
+                         : embed_launch<bf16>(table, ids, out, copies, n_tokens, hidden, vocab, scale, pos_table, positions, n_positions, stream);
 }
 
 // ---------------------------------------------------------------------------------------------

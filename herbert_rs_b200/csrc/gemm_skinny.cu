@@ -48,6 +48,8 @@ struct SkinnyNorm {
   bf16* out_xw;            // [M, out_ld] = residual * out_w
   int out_ld;
   float* out_sumsq;        // [units][SK_NORM_ROWS]
+  // SwiGLU epilogue only (with and without a norm).  > 0: the clamped form with this limit (HB_ACT_SWISH_CLAMP)
+  float glu_limit;
 };
 
 // NT: 8-token tiles (M <= 8 * NT).  RG: groups of 16 weight rows per CTA; a warp multiplies each
@@ -184,7 +186,13 @@ gemm_skinny_kernel(const bf16* __restrict__ A, int lda, const bf16* __restrict__
           up *= inv_rms[m];
         }
         const int col = (unit * RG + rg) * 8 + ch;
-        if (row0 + rg * 16 + ch + 8 < N) ((bf16*)Cv)[(size_t)m * ldc + col] = __float2bfloat16_rn((gate / (1.0f + expf(-gate))) * up);
+        float slope = 1.0f;
+        if (nm.glu_limit > 0.0f) {
+          gate = fminf(gate, nm.glu_limit);
+          up = fminf(fmaxf(up, -nm.glu_limit), nm.glu_limit) + 1.0f;
+          slope = HB_SWISH_CLAMP_SLOPE;
+        }
+        if (row0 + rg * 16 + ch + 8 < N) ((bf16*)Cv)[(size_t)m * ldc + col] = __float2bfloat16_rn((gate / (1.0f + expf(-slope * gate))) * up);
       }
     } else {
       // 16 * RG * NT * 8 is a multiple of 128: whole warps enter an iteration, and the 16 * RG
@@ -257,7 +265,7 @@ static int skinny_launch(const bf16* A, int lda, const bf16* W, int ldw, void* C
 static bool skinny_two_groups(int M, int N) { return M <= 16 && N >= 8192; }
 
 extern "C" int hb_gemm_skinny_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N,
-                                   int K, int epi, void* stream) {
+                                   int K, int epi, float glu_limit, void* stream) {
   HB_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_skinny: sizes must be positive");
   HB_REQUIRE(M <= 64, "gemm_skinny: at most 64 activation rows, got %d", M);
   HB_REQUIRE(K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0, "gemm_skinny: K (%d) and the leading dimensions (%d, %d) must be multiples of 8", K, lda, ldw);
@@ -267,12 +275,14 @@ extern "C" int hb_gemm_skinny_bf16(const void* A, int lda, const void* W, int ld
   const bf16* a = (const bf16*)A;
   const bf16* w = (const bf16*)W;
   const bool two = skinny_two_groups(M, N);
-  if (M <= 8) return two ? skinny_launch<1, 2, 2>(a, lda, w, ldw, C, ldc, M, N, K, epi, s)
-                         : skinny_launch<1, 1, 4>(a, lda, w, ldw, C, ldc, M, N, K, epi, s);
-  if (M <= 16) return two ? skinny_launch<2, 2, 2>(a, lda, w, ldw, C, ldc, M, N, K, epi, s)
-                          : skinny_launch<2, 1, 4>(a, lda, w, ldw, C, ldc, M, N, K, epi, s);
-  if (M <= 32) return skinny_launch<4, 1, 2>(a, lda, w, ldw, C, ldc, M, N, K, epi, s);
-  return skinny_launch<8, 1, 2>(a, lda, w, ldw, C, ldc, M, N, K, epi, s);
+  SkinnyNorm nm{};
+  nm.glu_limit = epi == HB_EPI_SWIGLU ? glu_limit : 0.0f;
+  if (M <= 8) return two ? skinny_launch<1, 2, 2>(a, lda, w, ldw, C, ldc, M, N, K, epi, s, nm)
+                         : skinny_launch<1, 1, 4>(a, lda, w, ldw, C, ldc, M, N, K, epi, s, nm);
+  if (M <= 16) return two ? skinny_launch<2, 2, 2>(a, lda, w, ldw, C, ldc, M, N, K, epi, s, nm)
+                          : skinny_launch<2, 1, 4>(a, lda, w, ldw, C, ldc, M, N, K, epi, s, nm);
+  if (M <= 32) return skinny_launch<4, 1, 2>(a, lda, w, ldw, C, ldc, M, N, K, epi, s, nm);
+  return skinny_launch<8, 1, 2>(a, lda, w, ldw, C, ldc, M, N, K, epi, s, nm);
 }
 
 // How many groups of output columns the product of an [M, K] activation with an [N, K] matrix

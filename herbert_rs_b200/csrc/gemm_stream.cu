@@ -48,6 +48,7 @@ struct StreamArgs {
   float* partials;  // [tiles][slices][NP][128]
   int* counters;    // [tiles], zero between launches
   int* error_flag;
+  float glu_limit;  // SwiGLU epilogue: > 0 takes the clamped form with this limit (HB_ACT_SWISH_CLAMP)
 };
 
 template <int EPI>
@@ -187,8 +188,13 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
           if (m < a.NP) {
             const float up = __shfl_down_sync(0xffffffffu, acc[m], 8);
             if ((lane & 8) == 0 && m < a.M && n + 8 < a.N) {
-              const float gate = acc[m];
-              ((bf16*)a.C)[(size_t)m * a.ldc + col] = __float2bfloat16_rn((gate / (1.0f + expf(-gate))) * up);
+              float gate = acc[m], u = up, slope = 1.0f;
+              if (a.glu_limit > 0.0f) {
+                gate = fminf(gate, a.glu_limit);
+                u = fminf(fmaxf(u, -a.glu_limit), a.glu_limit) + 1.0f;
+                slope = HB_SWISH_CLAMP_SLOPE;
+              }
+              ((bf16*)a.C)[(size_t)m * a.ldc + col] = __float2bfloat16_rn((gate / (1.0f + expf(-slope * gate))) * u);
             }
           }
         }
@@ -272,7 +278,7 @@ static int stream_launch(const CUtensorMap& mw, const CUtensorMap& mx, const Str
 // counters: hb_gemm_stream_counters(N) ints, zero before the first call (the kernel leaves them zero).
 // scratch: hb_gemm_stream_scratch_floats(M, N, K) floats (may be null when that is 0).
 extern "C" int hb_gemm_stream_bf16(const void* X, int ldx, const void* W, int ldw, void* C, int ldc, int M, int N, int K,
-                                   int epi, float* scratch, long long scratch_floats, int* counters, int n_counters,
+                                   int epi, float glu_limit, float* scratch, long long scratch_floats, int* counters, int n_counters,
                                    int* error_flag, void* stream) {
   HB_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_stream: sizes must be positive");
   HB_REQUIRE(M <= GS_MAX_NP, "gemm_stream: at most %d activation rows, got %d", GS_MAX_NP, M);
@@ -291,7 +297,7 @@ extern "C" int hb_gemm_stream_bf16(const void* X, int ldx, const void* W, int ld
   if (rc) return rc;
   rc = make_map(&mx, X, M, K, ldx, p.NP);
   if (rc) return rc;
-  StreamArgs a{C, ldc, M, N, K, p.NP, p.stages, p.tmem_cols, scratch, counters, error_flag};
+  StreamArgs a{C, ldc, M, N, K, p.NP, p.stages, p.tmem_cols, scratch, counters, error_flag, epi == HB_EPI_SWIGLU ? glu_limit : 0.0f};
   cudaStream_t s = (cudaStream_t)stream;
   switch (epi) {
     case HB_EPI_STORE: return stream_launch<HB_EPI_STORE>(mw, mx, a, p, s);

@@ -766,7 +766,7 @@ extern "C" int hb_gemm_tcgen05_set_workspace(float* floats, int* counters, int c
 // error_flag: one int in device memory, zero before the call; non-zero afterwards means a bounded
 // wait ran out inside the kernel (1 producer, 2 MMA issuer, 3 epilogue) and C is not valid.
 extern "C" int hb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N,
-                                    int K, int epi, int* error_flag, void* stream) {
+                                    int K, int epi, float glu_limit, int* error_flag, void* stream) {
   HB_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_tcgen05: sizes must be positive");
   HB_REQUIRE(K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0, "gemm_tcgen05: K (%d) and the leading dimensions (%d, %d) must be multiples of 8 (16-byte rows for TMA)", K, lda, ldw);
   HB_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_tcgen05: operands must be 16-byte aligned");
@@ -780,7 +780,8 @@ extern "C" int hb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int l
   rc = make_map(&mw, W, N, K, ldw, pairs ? 128 : BN);
   if (rc) return rc;
   cudaStream_t s = (cudaStream_t)stream;
-  const TgNorm none{};
+  TgNorm none{};
+  none.glu_limit = epi == HB_EPI_SWIGLU ? glu_limit : 0.0f;
   if (const int went = tg_try_pairk(false, A, lda, W, ldw, C, ldc, M, N, K, epi, error_flag, s, none)) return went > 0 ? 0 : -went;
   if (pairs) return tg_dispatch_pair<false>(ma, mw, C, ldc, M, N, K, epi, error_flag, s, none);
   if (const int went = tg_try_ksplit(false, A, lda, W, ldw, C, ldc, M, N, K, epi, error_flag, s, none)) return went > 0 ? 0 : -went;

@@ -111,6 +111,7 @@ extern "C" int hb_axpby(float* y, int ldy, float a, const float* z, int ldz, flo
 // gu [n_tokens, 2 inter] floats (a product's sums), bias [2 inter] in the same column layout (or null):
 // out = act(gate + b_gate) * (up + b_up) in the activation type.  interleave 0: gate columns [0, inter), up columns
 // [inter, 2 inter); interleave n: blocks of 2n columns, n gate then n up.
+// (HB_ACT_SWISH_CLAMP, with a limit L: min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1).)
 __device__ __forceinline__ float bias_glu_act(float g, int act) {
   return act == HB_ACT_RELU        ? fmaxf(g, 0.0f)
          : act == HB_ACT_GELU_TANH ? 0.5f * g * (1.0f + tanhf(0.79788456080286535588f * (g + 0.044715f * g * g * g)))
@@ -119,7 +120,7 @@ __device__ __forceinline__ float bias_glu_act(float g, int act) {
 }
 template <typename T>
 __global__ void bias_glu_kernel(const float* __restrict__ gu, int ld, const float* __restrict__ bias, T* __restrict__ out, int ldo,
-                                int inter, int interleave, int act) {
+                                int inter, int interleave, int act, float limit) {
   pdl_wait();
   pdl_launch();
   const int t = blockIdx.y;
@@ -132,21 +133,29 @@ __global__ void bias_glu_kernel(const float* __restrict__ gu, int ld, const floa
   }
   const float* row = gu + (size_t)t * ld;
   const float g = row[gi] + (bias ? bias[gi] : 0.0f), u = row[ui] + (bias ? bias[ui] : 0.0f);
-  out[(size_t)t * ldo + i] = from_f32<T>(bias_glu_act(g, act) * u);
+  float r;
+  if (act == HB_ACT_SWISH_CLAMP) {
+    const float gc = fminf(g, limit);
+    r = gc / (1.0f + expf(-HB_SWISH_CLAMP_SLOPE * gc)) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+  } else {
+    r = bias_glu_act(g, act) * u;
+  }
+  out[(size_t)t * ldo + i] = from_f32<T>(r);
 }
 
 extern "C" int hb_bias_glu(int dtype, const float* gu, int ld, const float* bias, void* out, int ldo, int n_tokens, int inter,
-                           int interleave, int act, void* stream) {
+                           int interleave, int act, float limit, void* stream) {
   HB_REQUIRE(n_tokens > 0 && inter > 0, "bias_glu: sizes must be positive");
   HB_REQUIRE(interleave == 0 || (interleave > 0 && inter % interleave == 0),
              "bias_glu: intermediate size %d is no multiple of the interleave %d", inter, interleave);
   HB_REQUIRE(n_tokens <= 65535, "bias_glu: at most 65535 tokens per call, got %d", n_tokens);
-  HB_REQUIRE(act >= HB_ACT_SILU && act <= HB_ACT_RELU, "bias_glu: unknown activation %d", act);
+  HB_REQUIRE(act >= HB_ACT_SILU && act <= HB_ACT_SWISH_CLAMP, "bias_glu: unknown activation %d", act);
+  HB_REQUIRE(act != HB_ACT_SWISH_CLAMP || limit > 0.0f, "bias_glu: the clamped activation needs a limit > 0");
   dim3 grid(ceil_div(inter, 256), n_tokens);
   if (dtype == HB_F32)
-    hb_launch(bias_glu_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, gu, ld, bias, (float*)out, ldo, inter, interleave, act);
+    hb_launch(bias_glu_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, gu, ld, bias, (float*)out, ldo, inter, interleave, act, limit);
   else
-    hb_launch(bias_glu_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, gu, ld, bias, (bf16*)out, ldo, inter, interleave, act);
+    hb_launch(bias_glu_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, gu, ld, bias, (bf16*)out, ldo, inter, interleave, act, limit);
   HB_CHECK_LAUNCH("bias_glu");
   return 0;
 }

@@ -11,7 +11,7 @@
 //
 //   softmax     p_j = exp(s_j) / (sum_i exp(s_i) + exp(sink_h)): the sink has no key and no value
 //   range       keys lo..p of the query at position p, lo = max(0, p - window + 1) (window 0: all)
-//   rotation    pair (i, i + rot/2) at position p turns by a = p * f_i; cos a and sin a are both
+//   rotation    pair i, (i, i + rot/2) ("halves") or (2i, 2i + 1), at position p turns by a = p * f_i; cos a and sin a are both
 //               multiplied by one constant m (frequency scaling folds into f and m on the host)
 //   cache       one plane [pages][page_size][rank + rot] in the activation dtype
 //
@@ -24,7 +24,7 @@
 // One warp per token: c = RMSNorm(kv[:rank]) * w, r = rotate(kv[rank:]), both into the cache.
 template <typename T>
 __global__ void latent_kv_store_kernel(const float* __restrict__ kv, int ld, const float* __restrict__ nw, float eps,
-                                       const float* __restrict__ freq, float mscale, int rank, int rot,
+                                       const float* __restrict__ freq, float mscale, int halves, int rank, int rot,
                                        const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                                        const int* __restrict__ seq_pages, int pages_stride, T* __restrict__ cache,
                                        int n_tokens, int page_size) {
@@ -47,14 +47,15 @@ __global__ void latent_kv_store_kernel(const float* __restrict__ kv, int ld, con
     sincosf((float)p * freq[i], &s, &c);
     s *= mscale;
     c *= mscale;
-    const float u = row[rank + i], v = row[rank + half + i];
-    dst[rank + i] = from_f32<T>(u * c - v * s);
-    dst[rank + half + i] = from_f32<T>(v * c + u * s);
+    const int j0 = rank + (halves ? i : 2 * i), j1 = halves ? j0 + half : j0 + 1;
+    const float u = row[j0], v = row[j1];
+    dst[j0] = from_f32<T>(u * c - v * s);
+    dst[j1] = from_f32<T>(v * c + u * s);
   }
 }
 
 extern "C" int hb_latent_kv_store(int dtype, const float* kv, int ld, const float* norm_w, float eps, const float* freq,
-                                  float mscale, int rank, int rot, const int* tok_seq, const int* tok_pos,
+                                  float mscale, int halves, int rank, int rot, const int* tok_seq, const int* tok_pos,
                                   const int* seq_pages, int pages_stride, void* cache, int n_tokens, int page_size,
                                   void* stream) {
   HB_REQUIRE(n_tokens > 0 && rank > 0 && rot >= 0 && rot % 2 == 0 && page_size > 0, "latent_kv_store: bad sizes");
@@ -62,10 +63,10 @@ extern "C" int hb_latent_kv_store(int dtype, const float* kv, int ld, const floa
   const int warps = 4;
   dim3 grid(ceil_div(n_tokens, warps));
   if (dtype == HB_F32)
-    hb_launch(latent_kv_store_kernel<float>, grid, dim3(warps * 32), 0, (cudaStream_t)stream, kv, ld, norm_w, eps, freq, mscale, rank,
+    hb_launch(latent_kv_store_kernel<float>, grid, dim3(warps * 32), 0, (cudaStream_t)stream, kv, ld, norm_w, eps, freq, mscale, halves, rank,
               rot, tok_seq, tok_pos, seq_pages, pages_stride, (float*)cache, n_tokens, page_size);
   else
-    hb_launch(latent_kv_store_kernel<bf16>, grid, dim3(warps * 32), 0, (cudaStream_t)stream, kv, ld, norm_w, eps, freq, mscale, rank,
+    hb_launch(latent_kv_store_kernel<bf16>, grid, dim3(warps * 32), 0, (cudaStream_t)stream, kv, ld, norm_w, eps, freq, mscale, halves, rank,
               rot, tok_seq, tok_pos, seq_pages, pages_stride, (bf16*)cache, n_tokens, page_size);
   HB_CHECK_LAUNCH("latent_kv_store");
   return 0;
@@ -75,7 +76,7 @@ extern "C" int hb_latent_kv_store(int dtype, const float* kv, int ld, const floa
 // The rotated part of every head of every token: in[t, h*in_hs + in_off + ..rot] -> out[t, h*out_hs + out_off + ..rot],
 // rotated at the token's position and multiplied by `scale`.  One thread per pair.
 __global__ void rotate_heads_kernel(const float* __restrict__ in, int ld_in, int in_hs, int in_off, float* __restrict__ out,
-                                    int ld_out, int out_hs, int out_off, const float* __restrict__ freq, float mscale,
+                                    int ld_out, int out_hs, int out_off, const float* __restrict__ freq, float mscale, int halves,
                                     const int* __restrict__ tok_pos, int n_tokens, int H, int rot, float scale) {
   pdl_wait();
   pdl_launch();
@@ -89,19 +90,20 @@ __global__ void rotate_heads_kernel(const float* __restrict__ in, int ld_in, int
   c *= mscale;
   const float* src = in + (size_t)t * ld_in + (size_t)h * in_hs + in_off;
   float* dst = out + (size_t)t * ld_out + (size_t)h * out_hs + out_off;
-  const float u = src[i], v = src[half + i];
-  dst[i] = (u * c - v * s) * scale;
-  dst[half + i] = (v * c + u * s) * scale;
+  const int j0 = halves ? i : 2 * i, j1 = halves ? half + i : 2 * i + 1;
+  const float u = src[j0], v = src[j1];
+  dst[j0] = (u * c - v * s) * scale;
+  dst[j1] = (v * c + u * s) * scale;
 }
 
 extern "C" int hb_rotate_heads(const float* in, int ld_in, int in_head_stride, int in_offset, float* out, int ld_out,
-                               int out_head_stride, int out_offset, const float* freq, float mscale, const int* tok_pos,
+                               int out_head_stride, int out_offset, const float* freq, float mscale, int halves, const int* tok_pos,
                                int n_tokens, int heads, int rot, float scale, void* stream) {
   HB_REQUIRE(n_tokens > 0 && heads > 0 && rot >= 0 && rot % 2 == 0, "rotate_heads: bad sizes");
   if (rot == 0) return 0;
   const long long n = (long long)n_tokens * heads * (rot / 2);
   hb_launch(rotate_heads_kernel, dim3((unsigned)ceil_div_ll(n, 256)), dim3(256), 0, (cudaStream_t)stream, in, ld_in, in_head_stride,
-            in_offset, out, ld_out, out_head_stride, out_offset, freq, mscale, tok_pos, n_tokens, heads, rot, scale);
+            in_offset, out, ld_out, out_head_stride, out_offset, freq, mscale, halves, tok_pos, n_tokens, heads, rot, scale);
   HB_CHECK_LAUNCH("rotate_heads");
   return 0;
 }

@@ -1,7 +1,7 @@
-// Layer normalisation with a weight and no bias, alone and fused with what follows a sublayer whose
+// Layer normalisation with a weight (and, alone, an optional bias), alone and fused with what follows a sublayer whose
 // result is normed before it joins the residual stream.
 //
-//   LN(y)_i = (y_i - mean(y)) / sqrt(var(y) + eps) * w_i,   var = mean((y - mean)^2)
+//   LN(y)_i = (y_i - mean(y)) / sqrt(var(y) + eps) * w_i (+ b_i),   var = mean((y - mean)^2)
 //   alone:     out[r] = LN(x[rows[r]] or x[r])                       (activation dtype)
 //   residual:  x[r] += LN(y[r]) * s        (s: a per-channel scale, or none)
 //              h[r]  = x[r] in the activation dtype, if asked for: what the next sublayer reads
@@ -12,7 +12,7 @@
 #include "common.cuh"
 
 template <typename T>
-__global__ void layernorm_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ out,
+__global__ void layernorm_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, T* __restrict__ out,
                                  const int* __restrict__ rows, int dim, float eps) {
   __shared__ float red[32];
   pdl_wait();
@@ -29,7 +29,7 @@ __global__ void layernorm_kernel(const float* __restrict__ x, const float* __res
   }
   const float inv = 1.0f / sqrtf(block_sum(q, red) / (float)dim + eps);
   T* o = out + (size_t)r * dim;
-  for (int i = threadIdx.x; i < dim; i += blockDim.x) o[i] = from_f32<T>(((xr[i] - mean) * inv) * w[i]);
+  for (int i = threadIdx.x; i < dim; i += blockDim.x) o[i] = from_f32<T>(((xr[i] - mean) * inv) * w[i] + (bias ? bias[i] : 0.0f));
 }
 
 template <typename T>
@@ -62,13 +62,13 @@ __global__ void layernorm_residual_kernel(const float* __restrict__ y, int ldy, 
 
 static int ln_threads(int dim) { return dim >= 2048 ? 512 : (dim >= 512 ? 256 : 128); }
 
-extern "C" int hb_layernorm(int dtype, const float* x, const float* w, void* out, const int* rows, int n_rows,
+extern "C" int hb_layernorm(int dtype, const float* x, const float* w, const float* bias, void* out, const int* rows, int n_rows,
                             int dim, float eps, void* stream) {
   HB_REQUIRE(n_rows > 0 && dim > 0, "layernorm: sizes must be positive");
   if (dtype == HB_F32)
-    hb_launch(layernorm_kernel<float>, dim3(n_rows), dim3(ln_threads(dim)), 0, (cudaStream_t)stream, x, w, (float*)out, rows, dim, eps);
+    hb_launch(layernorm_kernel<float>, dim3(n_rows), dim3(ln_threads(dim)), 0, (cudaStream_t)stream, x, w, bias, (float*)out, rows, dim, eps);
   else
-    hb_launch(layernorm_kernel<bf16>, dim3(n_rows), dim3(ln_threads(dim)), 0, (cudaStream_t)stream, x, w, (bf16*)out, rows, dim, eps);
+    hb_launch(layernorm_kernel<bf16>, dim3(n_rows), dim3(ln_threads(dim)), 0, (cudaStream_t)stream, x, w, bias, (bf16*)out, rows, dim, eps);
   HB_CHECK_LAUNCH("layernorm");
   return 0;
 }

@@ -16,7 +16,8 @@
 //                       beta = sigmoid(b);  g = exp(-exp(A_log) * softplus(a + dt_bias))
 //   hb_linear_scan      the recurrence: token by token (decode, short steps, several sequences), or for one long
 //                       prompt alone the delta rule sixteen tokens at a time
-//   hb_gated_rmsnorm    y = o / rms(o) * w * gate-activation(g), the norm per head (w [dv]) or over all heads (w [H dv])
+//   hb_gated_rmsnorm    y = o / rms(o) * w * gate-activation(g), the norm per head (w [dv]) or over all heads (w [H dv]);
+//                       with gate_first the gate comes before the norm: v = o * gate-activation(g), y = v / rms(v) * w
 #include "api.h"
 #include "common.cuh"
 
@@ -550,32 +551,39 @@ extern "C" int hb_linear_scan(int delta, const float* q, int ldq, const float* k
 // ---------------------------------------------------------------------------------------------
 // y[t, u, :] = o / sqrt(mean(o^2) + eps) * w * act(gate): a unit u is one head (w [n] shared by the heads, or with
 // w_stride = n a weight [units * n] with a part for every head) or the whole row of all heads (one unit).
-// act: 0 silu, 1 sigmoid.  One CTA per (token, unit).
+// act: 0 silu, 1 sigmoid.  gate_first: the gate multiplies o before the norm instead of its result.  One CTA per (token, unit).
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ w, float eps, const float* __restrict__ gate,
-                     int ldg, T* __restrict__ y, int ldy, int units, int n, int act, int w_stride) {
+                     int ldg, T* __restrict__ y, int ldy, int units, int n, int act, int w_stride, int gate_first) {
   __shared__ float red[32];
   pdl_wait();
   pdl_launch();
   const int t = blockIdx.x / units, u = blockIdx.x % units;
   const float* orow = o + (size_t)t * ldo + (size_t)u * n;
+  const float* g = gate + (size_t)t * ldg + (size_t)u * n;
+  auto gate_of = [&](int i) {
+    const float gv = g[i], sg = 1.0f / (1.0f + expf(-gv));
+    return act == 0 ? gv * sg : sg;
+  };
   float ss = 0.0f;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(orow[i], orow[i], ss);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const float v = gate_first ? orow[i] * gate_of(i) : orow[i];
+    ss = fmaf(v, v, ss);
+  }
   ss = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(ss / (float)n + eps);
-  const float* g = gate + (size_t)t * ldg + (size_t)u * n;
   T* yr = y + (size_t)t * ldy + (size_t)u * n;
   w += (size_t)u * w_stride;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float gv = g[i];
-    const float sg = 1.0f / (1.0f + expf(-gv));
-    yr[i] = from_f32<T>(((orow[i] * inv) * w[i]) * (act == 0 ? gv * sg : sg));
+    const float ga = gate_of(i);
+    yr[i] = from_f32<T>(gate_first ? ((orow[i] * ga) * inv) * w[i] : ((orow[i] * inv) * w[i]) * ga);
   }
 }
 
 extern "C" int hb_gated_rmsnorm(int dtype, const float* o, int ldo, const float* w, float eps, const float* gate, int ldg,
-                                void* y, int ldy, int n_tokens, int units, int n, int act, int w_stride, void* stream) {
+                                void* y, int ldy, int n_tokens, int units, int n, int act, int w_stride, int gate_first,
+                                void* stream) {
   HB_REQUIRE(n_tokens > 0 && units > 0 && n > 0, "gated_rmsnorm: sizes must be positive");
   HB_REQUIRE(act == 0 || act == 1, "gated_rmsnorm: the gate's activation is 0 (silu) or 1 (sigmoid)");
   HB_REQUIRE(w_stride == 0 || w_stride == n, "gated_rmsnorm: the weight is shared by the units (stride 0) or has a part for each (stride %d)", n);
@@ -584,10 +592,10 @@ extern "C" int hb_gated_rmsnorm(int dtype, const float* o, int ldo, const float*
   const int threads = n >= 1024 ? 256 : n >= 128 ? 128 : (n >= 64 ? 64 : 32);
   if (dtype == HB_F32)
     hb_launch(gated_rmsnorm_kernel<float>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, o, ldo, w, eps, gate,
-              ldg, (float*)y, ldy, units, n, act, w_stride);
+              ldg, (float*)y, ldy, units, n, act, w_stride, gate_first);
   else
     hb_launch(gated_rmsnorm_kernel<bf16>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, o, ldo, w, eps, gate,
-              ldg, (bf16*)y, ldy, units, n, act, w_stride);
+              ldg, (bf16*)y, ldy, units, n, act, w_stride, gate_first);
   HB_CHECK_LAUNCH("gated_rmsnorm");
   return 0;
 }

@@ -4,14 +4,6 @@
 #include "api.h"
 #include "common.cuh"
 
-extern "C" long long hb_attention_decode_scratch_floats(int n_seqs, int nh, int hd, int nsplit);
-extern "C" int hb_attention_decode_bf16(const void* q, int ldq, void* out, int ldo, const void* kcache,
-                                        const void* vcache, const int* seq_len, const int* seq_pages,
-                                        int pages_stride, float* scratch, int n_seqs, int nh, int nkv, int hd,
-                                        int page_size, int nsplit, float scale, int window, float softcap,
-                                        const float* sink, const float* gate_bias, const float* out_gate, int ldg,
-                                        void* stream);
-
 // The partial (m, l, o) results of the key splits.  In host code this name is only a handle for
 // the runtime's symbol calls, never a pointer a kernel could use; its device address is looked up
 // once per device below.
@@ -43,5 +35,5 @@ extern "C" int hb_attention_decode_bf16_noalloc(const void* q, int ldq, void* ou
   }
   return hb_attention_decode_bf16(q, ldq, out, ldo, kcache, vcache, seq_len, seq_pages, pages_stride,
                                   g_scratch_addr[device], n_seqs, nh, nkv, hd, page_size, nsplit, scale, window, 0.0f, nullptr,
-                                  nullptr, nullptr, 0, stream);
+                                  nullptr, nullptr, 0, 0.0f, 0.0f, 0.0f, 0, stream);
 }

@@ -4,11 +4,17 @@
 //   q <- q / sqrt(mean_all(q^2) + eps) * wq     over all heads of the row at once (likewise k; optional)
 //   pair m of the first `rot` channels of every q and k head turns by  p * fqk[m]
 //   pair m of all dv channels of every v head turns by                p * fv[m]      (optional)
+//   cos and sin of q's and k's angles are multiplied by one constant (scaled frequencies); a bias vector may be added
+//   to the row before anything else
 //   (u, v) -> (u cos a - v sin a, v cos a + u sin a);  pair m is (2m, 2m + 1) ("interleaved") or (m, m + n/2) ("halves")
 //
-// The product's rows arrive as floats [q: nh x dk | k: nkv x dk | v: nkv x dv]; q leaves in the activation type with
-// heads of `hd` channels, k and v go into the paged cache whose heads have `hd` channels as well.  hd >= max(dk, dv):
-// channels beyond dk (dv) are written as zeros, so an attention kernel over heads of hd sees the same scores and
+// With `maps` > 1 a head has that many queries and keys of dk channels (attention maps over one value): the query of
+// map m becomes a query head of its own whose channels m dk .. (m + 1) dk are set and whose others are zero, a key head
+// holds its maps side by side, so the score of query (h, m) with a key is the score of map m alone.
+//
+// The product's rows arrive as floats [q: nh x maps x dk | k: nkv x maps x dk | v: nkv x dv]; q leaves in the activation type with
+// heads of `hd` channels, k and v go into the paged cache whose heads have `hd` channels as well.  hd >= max(maps dk, dv):
+// channels beyond those are written as zeros, so an attention kernel over heads of hd sees the same scores and
 // returns the values' channels followed by zeros.  Angles are float products of the integer position and a float
 // frequency, sine and cosine are the accurate ones.
 //
@@ -21,24 +27,26 @@
 
 struct RotPrepArgs {
   const float* rows; int ld;
+  const float* bias;               // in the rows' layout, added first; null: none
   const float* wq; const float* wk; float eps; int whole_norm;
-  const float* fqk; int rot; int halves;
+  const float* fqk; int rot; int halves; float mscale;
   const float* fv;                 // null: values are stored as they are
   const int* tok_seq; const int* tok_pos; const int* seq_pages; int pages_stride;
   void* q_out; int ldq;
   void* kcache; void* vcache;
-  int nh, nkv, dk, dv, hd, page_size, write_cache;
+  int nh, nkv, maps, dk, dv, hd, page_size, write_cache;
 };
 
-// own * cos + (-/+ partner) * sin for channel j of a head whose first `rot` channels are rotated
-__device__ __forceinline__ float turn_channel(const float* head, const float* w, float inv, int j, int rot, int halves,
-                                              const float* freq, float pos, float dir) {
-  const float own = head[j] * inv * (w ? w[j] : 1.0f);
+// own * cos + (-/+ partner) * sin for channel j of a head whose first `rot` channels are rotated; cs holds the
+// token's cosines of all pairs, then the sines
+__device__ __forceinline__ float turn_channel(const float* head, const float* bias, const float* w, float inv, int j, int rot,
+                                              int halves, const float* cs) {
+  const float own = (head[j] + (bias ? bias[j] : 0.0f)) * inv * (w ? w[j] : 1.0f);
   if (j >= rot) return own;
+  const int half = rot >> 1;
   int m, partner;
   bool first;
   if (halves) {
-    const int half = rot >> 1;
     first = j < half;
     m = first ? j : j - half;
     partner = first ? j + half : j - half;
@@ -47,39 +55,64 @@ __device__ __forceinline__ float turn_channel(const float* head, const float* w,
     m = j >> 1;
     partner = j ^ 1;
   }
-  const float other = head[partner] * inv * (w ? w[partner] : 1.0f);
-  float s, c;
-  sincosf(pos * freq[m], &s, &c);
-  s *= dir;
+  const float other = (head[partner] + (bias ? bias[partner] : 0.0f)) * inv * (w ? w[partner] : 1.0f);
+  const float c = cs[m], s = cs[half + m];
   return first ? own * c - other * s : own * c + other * s;
 }
 
 template <typename T>
 __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
+  extern __shared__ float tab[];          // cos and sin of the token's angles: [rot] for q and k, [dv] for values
   __shared__ float red[32];
   pdl_wait();
   pdl_launch();
   const int t = blockIdx.x, p = a.tok_pos[t];
   const float pos = (float)p;
+  float* tab_v = tab + a.rot;
+  for (int m = threadIdx.x; m < a.rot / 2; m += blockDim.x) {
+    float s, c;
+    sincosf(pos * a.fqk[m], &s, &c);
+    tab[m] = c * a.mscale;
+    tab[a.rot / 2 + m] = s * a.mscale;
+  }
+  if (a.fv)
+    for (int m = threadIdx.x; m < a.dv / 2; m += blockDim.x) {
+      float s, c;
+      sincosf(pos * a.fv[m], &s, &c);
+      tab_v[m] = c;
+      tab_v[a.dv / 2 + m] = s;
+    }
+  __syncthreads();
+  const int qn = a.nh * a.maps * a.dk, kn = a.nkv * a.maps * a.dk;
   const float* q = a.rows + (size_t)t * a.ld;
-  const float* k = q + (size_t)a.nh * a.dk;
-  const float* v = k + (size_t)a.nkv * a.dk;
+  const float* k = q + qn;
+  const float* v = k + kn;
+  const float* bq = a.bias;
+  const float* bk = a.bias ? a.bias + qn : nullptr;
+  const float* bv = a.bias ? a.bias + qn + kn : nullptr;
   float inv_q = 1.0f, inv_k = 1.0f;
   if (a.whole_norm) {
-    const int nq = a.nh * a.dk, nk = a.nkv * a.dk;
     float sq = 0.0f, sk = 0.0f;
-    for (int i = threadIdx.x; i < nq; i += blockDim.x) sq = fmaf(q[i], q[i], sq);
-    for (int i = threadIdx.x; i < nk; i += blockDim.x) sk = fmaf(k[i], k[i], sk);
+    for (int i = threadIdx.x; i < qn; i += blockDim.x) {
+      const float x = q[i] + (bq ? bq[i] : 0.0f);
+      sq = fmaf(x, x, sq);
+    }
+    for (int i = threadIdx.x; i < kn; i += blockDim.x) {
+      const float x = k[i] + (bk ? bk[i] : 0.0f);
+      sk = fmaf(x, x, sk);
+    }
     sq = block_sum(sq, red);
     sk = block_sum(sk, red);
-    inv_q = 1.0f / sqrtf(sq / (float)nq + a.eps);
-    inv_k = 1.0f / sqrtf(sk / (float)nk + a.eps);
+    inv_q = 1.0f / sqrtf(sq / (float)qn + a.eps);
+    inv_k = 1.0f / sqrtf(sk / (float)kn + a.eps);
   }
+  // map m of a head lies in channels m * dk ..: a query of map m is zero elsewhere, a key holds all maps side by side
   T* qo = (T*)a.q_out + (size_t)t * a.ldq;
-  for (int i = threadIdx.x; i < a.nh * a.hd; i += blockDim.x) {
-    const int h = i / a.hd, j = i - h * a.hd;
+  for (int i = threadIdx.x; i < a.nh * a.maps * a.hd; i += blockDim.x) {
+    const int h = i / a.hd, j = i - h * a.hd - (h % a.maps) * a.dk;
+    const size_t at = (size_t)h * a.dk;
     float r = 0.0f;
-    if (j < a.dk) r = turn_channel(q + (size_t)h * a.dk, a.wq ? a.wq + (size_t)h * a.dk : nullptr, inv_q, j, a.rot, a.halves, a.fqk, pos, 1.0f);
+    if (j >= 0 && j < a.dk) r = turn_channel(q + at, bq ? bq + at : nullptr, a.wq ? a.wq + at : nullptr, inv_q, j, a.rot, a.halves, tab);
     qo[i] = from_f32<T>(r);
   }
   if (!a.write_cache) return;
@@ -89,31 +122,37 @@ __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
     const int g = i / a.hd, j = i - g * a.hd;
     const size_t at = (((size_t)page * a.nkv + g) * a.page_size + in_page) * a.hd + j;
     float rk = 0.0f, rv = 0.0f;
-    if (j < a.dk) rk = turn_channel(k + (size_t)g * a.dk, a.wk ? a.wk + (size_t)g * a.dk : nullptr, inv_k, j, a.rot, a.halves, a.fqk, pos, 1.0f);
-    if (j < a.dv) rv = turn_channel(v + (size_t)g * a.dv, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, a.fv, pos, 1.0f);
+    if (j < a.maps * a.dk) {
+      const int m = j / a.dk;
+      const size_t head = (size_t)(g * a.maps + m) * a.dk;
+      rk = turn_channel(k + head, bk ? bk + head : nullptr, a.wk ? a.wk + head : nullptr, inv_k, j - m * a.dk, a.rot, a.halves, tab);
+    }
+    if (j < a.dv) rv = turn_channel(v + (size_t)g * a.dv, bv ? bv + (size_t)g * a.dv : nullptr, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, tab_v);
     ((T*)a.kcache)[at] = from_f32<T>(rk);
     ((T*)a.vcache)[at] = from_f32<T>(rv);
   }
 }
 
-extern "C" int hb_qkv_rotary_cache(int dtype, const float* rows, int ld, const float* wq, const float* wk, float eps,
-                                   int whole_norm, const float* fqk, int rot, int halves, const float* fv, const int* tok_seq,
+extern "C" int hb_qkv_rotary_cache(int dtype, const float* rows, int ld, const float* bias, const float* wq, const float* wk, float eps,
+                                   int whole_norm, const float* fqk, int rot, int halves, float mscale, const float* fv, const int* tok_seq,
                                    const int* tok_pos, const int* seq_pages, int pages_stride, void* q_out, int ldq, void* kcache,
-                                   void* vcache, int n_tokens, int nh, int nkv, int dk, int dv, int hd, int page_size,
+                                   void* vcache, int n_tokens, int nh, int nkv, int maps, int dk, int dv, int hd, int page_size,
                                    int write_cache, void* stream) {
-  HB_REQUIRE(n_tokens > 0 && nh > 0 && nkv > 0 && dk > 0 && dv > 0 && page_size > 0, "qkv_rotary_cache: sizes must be positive");
-  HB_REQUIRE(hd >= dk && hd >= dv, "qkv_rotary_cache: cache heads of %d channels cannot hold keys of %d and values of %d", hd, dk, dv);
+  HB_REQUIRE(n_tokens > 0 && nh > 0 && nkv > 0 && maps > 0 && dk > 0 && dv > 0 && page_size > 0, "qkv_rotary_cache: sizes must be positive");
+  HB_REQUIRE(hd >= maps * dk && hd >= dv, "qkv_rotary_cache: cache heads of %d channels cannot hold keys of %d x %d and values of %d", hd, maps, dk, dv);
   HB_REQUIRE(rot >= 0 && rot <= dk && rot % 2 == 0, "qkv_rotary_cache: %d rotated channels must be even and at most %d", rot, dk);
   HB_REQUIRE(rot == 0 || fqk != nullptr, "qkv_rotary_cache: rotated channels need their frequencies");
   HB_REQUIRE(fv == nullptr || dv % 2 == 0, "qkv_rotary_cache: rotated values need an even size, got %d", dv);
   // a step that stores nothing (it reads another layer's keys and values) brings rows of queries only
-  HB_REQUIRE(ld >= nh * dk + (write_cache ? nkv * (dk + dv) : 0) && ldq >= nh * hd, "qkv_rotary_cache: rows are shorter than their heads");
-  RotPrepArgs a{rows, ld, wq, wk, eps, whole_norm, fqk, rot, halves, fv, tok_seq, tok_pos, seq_pages, pages_stride, q_out, ldq,
-                kcache, vcache, nh, nkv, dk, dv, hd, page_size, write_cache};
+  HB_REQUIRE(ld >= nh * maps * dk + (write_cache ? nkv * (maps * dk + dv) : 0) && ldq >= nh * maps * hd, "qkv_rotary_cache: rows are shorter than their heads");
+  const size_t smem = (size_t)(rot + (fv ? dv : 0)) * sizeof(float);
+  HB_REQUIRE(smem <= 48 * 1024, "qkv_rotary_cache: %d rotated channels exceed a block's shared memory", rot);
+  RotPrepArgs a{rows, ld, bias, wq, wk, eps, whole_norm, fqk, rot, halves, mscale, fv, tok_seq, tok_pos, seq_pages, pages_stride, q_out, ldq,
+                kcache, vcache, nh, nkv, maps, dk, dv, hd, page_size, write_cache};
   if (dtype == HB_F32)
-    hb_launch(qkv_rotary_cache_kernel<float>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, a);
+    hb_launch(qkv_rotary_cache_kernel<float>, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, a);
   else
-    hb_launch(qkv_rotary_cache_kernel<bf16>, dim3(n_tokens), dim3(256), 0, (cudaStream_t)stream, a);
+    hb_launch(qkv_rotary_cache_kernel<bf16>, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, a);
   HB_CHECK_LAUNCH("qkv_rotary_cache");
   return 0;
 }
@@ -183,5 +222,48 @@ extern "C" int hb_head_gate(int dtype, const void* att, int ld, int hd, const fl
     hb_launch(head_gate_kernel<bf16>, dim3(n_tokens), dim3(128), 0, (cudaStream_t)stream, (const bf16*)att, ld, hd, gate, ldg,
               (bf16*)y, ldy, nh, dv);
   HB_CHECK_LAUNCH("head_gate");
+  return 0;
+}
+
+
+// ---------------------------------------------------------------------------------------------
+// Two attention maps of a head over the same values, subtracted and normed:
+//   o = a1 - lambda * a2;   y[t, h, :] = o / sqrt(mean(o^2) + eps) * factor       (over the dv value channels)
+// att holds floats, the maps of head h at heads 2h and 2h + 1 of hd channels.  One warp per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(128)
+difference_heads_kernel(const float* __restrict__ att, int ld, int hd, float lambda, float factor, float eps, T* __restrict__ y,
+                        int ldy, int n_tokens, int nh, int dv) {
+  pdl_wait();
+  pdl_launch();
+  const int lane = threadIdx.x & 31;
+  const long long unit = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (unit >= (long long)n_tokens * nh) return;
+  const int t = (int)(unit / nh), h = (int)(unit % nh);
+  const float* a1 = att + (size_t)t * ld + (size_t)(2 * h) * hd;
+  const float* a2 = a1 + hd;
+  float ss = 0.0f;
+  for (int i = lane; i < dv; i += 32) {
+    const float o = a1[i] - lambda * a2[i];
+    ss = fmaf(o, o, ss);
+  }
+  ss = warp_sum(ss);
+  const float k = factor / sqrtf(ss / (float)dv + eps);
+  T* yr = y + (size_t)t * ldy + (size_t)h * dv;
+  for (int i = lane; i < dv; i += 32) yr[i] = from_f32<T>((a1[i] - lambda * a2[i]) * k);
+}
+
+extern "C" int hb_difference_heads(int dtype, const float* att, int ld, int hd, float lambda, float factor, float eps, void* y,
+                                   int ldy, int n_tokens, int nh, int dv, void* stream) {
+  HB_REQUIRE(n_tokens > 0 && nh > 0 && dv > 0 && hd >= dv, "difference_heads: sizes must be positive and heads wide enough");
+  const long long blocks = ceil_div_ll((long long)n_tokens * nh, 4);
+  HB_REQUIRE(blocks < 2147483647LL, "difference_heads: too many (token, head) pairs");
+  if (dtype == HB_F32)
+    hb_launch(difference_heads_kernel<float>, dim3((unsigned)blocks), dim3(128), 0, (cudaStream_t)stream, att, ld, hd, lambda, factor,
+              eps, (float*)y, ldy, n_tokens, nh, dv);
+  else
+    hb_launch(difference_heads_kernel<bf16>, dim3((unsigned)blocks), dim3(128), 0, (cudaStream_t)stream, att, ld, hd, lambda, factor,
+              eps, (bf16*)y, ldy, n_tokens, nh, dv);
+  HB_CHECK_LAUNCH("difference_heads");
   return 0;
 }

@@ -1,7 +1,7 @@
 // A short causal convolution over time, channel by channel, whose last inputs are a sequence's state;
 // and an embedding to which a row chosen by (previous token, token) is added, whose previous token is state too.
 //
-//   conv:   c_t = sum_j w[:, j] * u_{t - taps + 1 + j}      (w [channels, taps]; the last column weighs u_t itself;
+//   conv:   c_t = b + sum_j w[:, j] * u_{t - taps + 1 + j}  (b optional; w [channels, taps]; the last column weighs u_t itself;
 //                                                            zeros before the sequence's start)
 //           out_t = u_t + c_t (add_input)  or  c_t,  then silu if asked
 //   state:  [slots, taps - 1, channels] floats: the inputs u of the sequence's last taps - 1 positions, zero when
@@ -18,7 +18,7 @@
 
 template <typename TO>
 __global__ void __launch_bounds__(SC_THREADS)
-short_conv_kernel(const float* __restrict__ in, int ld_in, const float* __restrict__ w, float* __restrict__ state,
+short_conv_kernel(const float* __restrict__ in, int ld_in, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
                   const int* __restrict__ seq_slot, const int* __restrict__ seq_start, const int* __restrict__ seq_pos0,
                   TO* __restrict__ out, int ldo, int C, int taps, int add_input, int act_silu, int span) {
   pdl_wait();
@@ -33,8 +33,9 @@ short_conv_kernel(const float* __restrict__ in, int ld_in, const float* __restri
   const int pos0 = seq_pos0[b];
   float* st = state ? state + (size_t)seq_slot[b] * back * C + c : nullptr;
   const float* wr = w + (size_t)c * taps;
+  const float b0 = bias ? bias[c] : 0.0f;
   for (int i = lo; i < hi; ++i) {
-    float acc = 0.0f;
+    float acc = b0;
     for (int j = 0; j < taps; ++j) {
       const int s = i - back + j;          // index among this step's tokens; negative: before the step
       float u = 0.0f;
@@ -56,7 +57,7 @@ short_conv_kernel(const float* __restrict__ in, int ld_in, const float* __restri
   }
 }
 
-extern "C" int hb_short_conv(int out_dtype, const float* in, int ld_in, const float* w, float* state, const int* seq_slot,
+extern "C" int hb_short_conv(int out_dtype, const float* in, int ld_in, const float* w, const float* bias, float* state, const int* seq_slot,
                              const int* seq_start, const int* seq_pos0, void* out, int ldo, int n_seqs, int max_q_len,
                              int channels, int taps, int add_input, int act_silu, void* stream) {
   HB_REQUIRE(n_seqs > 0 && max_q_len > 0 && channels > 0, "short_conv: sizes must be positive");
@@ -74,10 +75,10 @@ extern "C" int hb_short_conv(int out_dtype, const float* in, int ld_in, const fl
     span /= 2;
   dim3 grid(ceil_div(channels, SC_THREADS), ceil_div(max_q_len, span), n_seqs);
   if (out_dtype == HB_F32)
-    hb_launch(short_conv_kernel<float>, grid, dim3(SC_THREADS), 0, (cudaStream_t)stream, in, ld_in, w, state, seq_slot, seq_start,
+    hb_launch(short_conv_kernel<float>, grid, dim3(SC_THREADS), 0, (cudaStream_t)stream, in, ld_in, w, bias, state, seq_slot, seq_start,
               seq_pos0, (float*)out, ldo, channels, taps, add_input, act_silu, span);
   else
-    hb_launch(short_conv_kernel<bf16>, grid, dim3(SC_THREADS), 0, (cudaStream_t)stream, in, ld_in, w, state, seq_slot, seq_start,
+    hb_launch(short_conv_kernel<bf16>, grid, dim3(SC_THREADS), 0, (cudaStream_t)stream, in, ld_in, w, bias, state, seq_slot, seq_start,
               seq_pos0, (bf16*)out, ldo, channels, taps, add_input, act_silu, span);
   HB_CHECK_LAUNCH("short_conv");
   return 0;

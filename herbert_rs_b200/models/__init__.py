@@ -3,6 +3,7 @@
 from ..config.begupel import BegupelConfig
 from ..config.kebisun import KebisunConfig
 from ..config.nefivik import NefivikConfig
+from ..config.putazen import PutazenConfig
 from ..config.qwen3 import Qwen3Config
 from ..config.votapel import VotapelConfig
 from ..registry import register_architecture
@@ -24,5 +25,8 @@ register_architecture("Begupel", BegupelConfig)
 # later layer may read) and of a generalised delta rule, each sublayer between two norms and behind a gate; routed
 # experts in groups with a clamped activation; a second input by token id at every layer's end.
 register_architecture("Nefivik", NefivikConfig)
+# A residual of several mixed copies; layers of differential attention, latent attention and a Mamba-2 state-space mixer,
+# a run of them several times with the same weights; clamped dense feed-forwards, layer norms with biases.
+register_architecture("Putazen", PutazenConfig)
 
 __all__ = ["DecoderModel"]

@@ -13,7 +13,8 @@ earlier step instead of storing its own.
 Options of the spec: a scaled embedding, a learned vector per position, a second table chosen by (previous
 token, token) whose previous token is kept per sequence in the cache's fixed-size region (the first schedule
 step's entry carries it under the name "embedding.last_id"), a tanh cap on the logits, a second table by token id
-of which blocks read their own columns (`ModelSpec.token_side_table`).
+of which blocks read their own columns (`ModelSpec.token_side_table`), a residual of several copies of the stream
+(`ModelSpec.streams`): equal at the start, mixed by the blocks, summed before the final norm.
 """
 
 from __future__ import annotations
@@ -45,6 +46,12 @@ class DecoderModel:
         self.position_table = None      # [max_position, hidden] learned vectors, if the spec names one
         self.pair_table = None          # [buckets + 1, hidden], if the spec has a pair embedding
         self.token_side_table = None    # [vocab, columns], if blocks add a second input chosen by the token
+        self.streams = spec.streams
+        for i, b in enumerate(self.blocks):
+            if b.streams != self.streams:
+                raise ConfigError(f"layer {i} works on {b.streams or 'one'} copies of the stream, the model on {self.streams or 'one'}")
+        if self.streams is not None and (spec.pair_embedding is not None or self.final_norm.as_stream_norm() is None):
+            raise ConfigError("a stream of several copies starts from a plain embedding and ends in a norm over their sum")
         for i, st in enumerate(spec.schedule):
             if not (0 <= st.layer < len(self.blocks)):
                 raise ConfigError(f"schedule step {i} names layer {st.layer}, but there are {len(self.blocks)} layers")
@@ -140,7 +147,8 @@ class DecoderModel:
         The result lives in the workspace and is valid until the next step."""
         ws = self.rt.workspace
         ws.rewind()
-        x = ws.take((batch.n_tokens, self.spec.hidden_size), torch.float32)
+        shape = (batch.n_tokens, self.spec.hidden_size)
+        x = ws.take(shape if self.streams is None else (shape[0], self.streams, shape[1]), torch.float32)
         pe = self.spec.pair_embedding
         if pe is not None:
             ops.pair_embed(self.embed, self.pair_table, batch, cache.view(0).states[_LAST_ID], x, pe.buckets, pe.mul_prev,
@@ -164,7 +172,10 @@ class DecoderModel:
         if batch.n_want == 0:
             return None
         hn = ws.take((batch.n_want, self.spec.hidden_size), self.rt.dtype)
-        self.final_norm.forward(x, hn, rows=batch.want_rows)
+        if self.streams is None:
+            self.final_norm.forward(x, hn, rows=batch.want_rows)
+        else:
+            ops.streams_join(x, norm=self.final_norm.as_stream_norm(), h=hn, rows=batch.want_rows)
         logits = ws.take((batch.n_want, self.spec.vocab_size), torch.float32)
         ops.gemm(hn, self.head, logits, ops.EPI_STORE_F32)
         if self.spec.logit_softcap:

@@ -28,7 +28,7 @@ SKINNY_MAX_ROWS = 64
 options = KernelOptions()
 
 _SIGS = {
-    "hb_embed": [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p],
+    "hb_embed": [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p],
     "hb_scaled_residual_norm": [c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
     "hb_qk_prepare_cache": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_void_p,
                             c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -39,7 +39,7 @@ _SIGS = {
                               c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                               c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "hb_gemm_simt": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "hb_gemm_skinny_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "hb_gemm_skinny_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
     "hb_gemm_skinny_norm_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                                  c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "hb_finish_norm": [c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -51,35 +51,35 @@ _SIGS = {
                                  c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
                                  c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                  c_void_p, c_void_p],
-    "hb_gemm_tcgen05_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
-    "hb_gemm_stream_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
+    "hb_gemm_tcgen05_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
+    "hb_gemm_stream_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p,
                             ctypes.c_longlong, c_void_p, c_int, c_void_p, c_void_p],
     "hb_attention_simt": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p,
-                          c_int, c_void_p],
+                          c_int, c_int, c_void_p],
     "hb_attention_decode_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p,
-                                 c_void_p, c_int, c_void_p],
+                                 c_void_p, c_int, c_float, c_float, c_float, c_int, c_void_p],
     "hb_attention_decode_fused_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float,
                                        c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                        c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
     "hb_attention_prefill_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                   c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p,
-                                  c_void_p, c_int, c_void_p],
+                                  c_void_p, c_int, c_int, c_void_p],
     "hb_attention_prefill_tc_bf16": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                      c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p,
-                                     c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
+                                     c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "hb_argmax": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p],
     "hb_gemm_skinny_norm_parts": [c_int, c_int],
     "hb_sample": [c_void_p, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
     "hb_rng_normal": [c_int, c_void_p, ctypes.c_longlong, ctypes.c_ulonglong, c_float, c_float, c_void_p],
     "hb_fill": [c_int, c_void_p, ctypes.c_longlong, c_float, c_void_p],
     "hb_cast": [c_int, c_void_p, c_int, c_void_p, ctypes.c_longlong, c_int, c_void_p],
-    "hb_layernorm": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
+    "hb_layernorm": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
     "hb_layernorm_residual": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
-    "hb_latent_kv_store": [c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_float, c_int, c_int, c_void_p, c_void_p,
+    "hb_latent_kv_store": [c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_float, c_int, c_int, c_int, c_void_p, c_void_p,
                            c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
-    "hb_rotate_heads": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int,
+    "hb_rotate_heads": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_int, c_void_p, c_int,
                         c_int, c_int, c_float, c_void_p],
     "hb_headwise_gemm": [c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
                          c_int, c_int, c_int, c_float, c_void_p],
@@ -106,9 +106,9 @@ _SIGS = {
     "hb_group_rmsnorm_residual": [c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
                                   c_int, c_int, c_int, c_float, c_void_p],
     "hb_axpby": [c_void_p, c_int, c_float, c_void_p, c_int, c_float, c_int, c_int, c_void_p],
-    "hb_bias_glu": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "hb_bias_glu": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
     "hb_tanh_cap": [c_void_p, c_int, c_float, c_int, c_int, c_void_p],
-    "hb_short_conv": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+    "hb_short_conv": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                       c_int, c_int, c_int, c_int, c_void_p],
     "hb_pair_embed": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                       c_int, c_int, c_int, ctypes.c_longlong, ctypes.c_longlong, c_float, c_void_p],
@@ -118,10 +118,19 @@ _SIGS = {
     "hb_linear_scan": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "hb_gated_rmsnorm": [c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
-                         c_int, c_int, c_void_p],
-    "hb_qkv_rotary_cache": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_void_p,
-                            c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-                            c_int, c_int, c_int, c_int, c_int, c_void_p],
+                         c_int, c_int, c_int, c_void_p],
+    "hb_qkv_rotary_cache": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_float,
+                            c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "hb_difference_heads": [c_int, c_void_p, c_int, c_int, c_float, c_float, c_float, c_void_p, c_int, c_int, c_int, c_int,
+                            c_void_p],
+    "hb_streams_join": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int,
+                        c_void_p, c_void_p, c_int, c_int, c_void_p],
+    "hb_ssd_scan": [c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                    c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "hb_ssd_chunks": [c_int, c_int, c_int, c_int],
+    "hb_ssd_chunked_bf16": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "hb_rotate_heads_back": [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                              c_void_p],
     "hb_head_gate": [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -152,7 +161,7 @@ def _fn(name: str):
 
 # kernels each launcher starts (for honest launch counts)
 _KERNELS_PER_CALL = {"hb_attention_decode_bf16": 2, "hb_argmax": 2, "hb_sample": 2, "hb_moe_experts": 2,
-                     "hb_moe_experts_grouped_bf16": 4, "hb_moe_experts_tc_bf16": 5}
+                     "hb_moe_experts_grouped_bf16": 4, "hb_moe_experts_tc_bf16": 5, "hb_ssd_chunked_bf16": 3}
 _launches = 0
 
 
@@ -334,13 +343,16 @@ def cast(src: torch.Tensor, dtype: torch.dtype, round_bf16: bool = False) -> tor
 def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0,
           pos_table: torch.Tensor | None = None, positions: torch.Tensor | None = None) -> None:
     """out[t, :] = float(table[ids[t], :]) * scale (+ float(pos_table[positions[t], :]) with a table of
-    learned position vectors, in the embedding's dtype); out is the float residual stream [T, H]."""
+    learned position vectors, in the embedding's dtype); out is the float residual stream [T, H], or [T, n, H] for a
+    stream of n copies, which start equal."""
     _check(table, None, "table"); _check(ids, torch.int32, "ids"); _check(out, torch.float32, "out")
     if pos_table is not None:
         _check(pos_table, table.dtype, "pos_table"); _check(positions, torch.int32, "positions")
         if pos_table.shape[1] != table.shape[1] or not pos_table.is_contiguous():
             raise BackendError("embed: the position table must be contiguous and as wide as the embedding")
-    _run("hb_embed", dtype_code(table.dtype), table.data_ptr(), ids.data_ptr(), out.data_ptr(),
+    if not out.is_contiguous():
+        raise BackendError("embed: out must be contiguous")
+    _run("hb_embed", dtype_code(table.dtype), table.data_ptr(), ids.data_ptr(), out.data_ptr(), out.shape[1] if out.dim() == 3 else 1,
          ids.numel(), table.shape[1], table.shape[0], float(scale), _ptr(pos_table),
          _ptr(positions) if pos_table is not None else None, 0 if pos_table is None else pos_table.shape[0], _stream())
 
@@ -380,10 +392,13 @@ def to_activation(x: torch.Tensor, out: torch.Tensor) -> None:
     _run("hb_cast", 0, x.data_ptr(), dtype_code(out.dtype), out.data_ptr(), x.numel(), 0, _stream())
 
 
-def layernorm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, eps: float, rows: torch.Tensor | None = None) -> None:
-    """out[r] = (x - mean) / sqrt(var + eps) * w of row rows[r] (or r) of x; x and w float."""
+def layernorm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, eps: float, rows: torch.Tensor | None = None,
+              bias: torch.Tensor | None = None) -> None:
+    """out[r] = (x - mean) / sqrt(var + eps) * w (+ bias) of row rows[r] (or r) of x; x, w and bias float."""
     _check(x, torch.float32, "x"); _check(w, torch.float32, "w"); _check(out, None, "out")
-    _run("hb_layernorm", dtype_code(out.dtype), x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(rows),
+    if bias is not None:
+        _check(bias, torch.float32, "bias")
+    _run("hb_layernorm", dtype_code(out.dtype), x.data_ptr(), w.data_ptr(), _ptr(bias), out.data_ptr(), _ptr(rows),
          out.shape[0], x.shape[-1], float(eps), _stream())
 
 
@@ -400,22 +415,22 @@ def layernorm_residual(y: torch.Tensor, w: torch.Tensor, scale: torch.Tensor | N
          _ptr(h), x.shape[0], x.shape[1], float(eps), _stream())
 
 
-def latent_kv_store(kv, norm_w, eps, freq, mscale, rank, rot, tok_seq, tok_pos, seq_pages, cache, page_size) -> None:
+def latent_kv_store(kv, norm_w, eps, freq, mscale, rank, rot, tok_seq, tok_pos, seq_pages, cache, page_size, halves=True) -> None:
     """Rows [c | r] of kv (float, [T, >= rank + rot]): c normed (RMS, weight norm_w), r rotated at the
     token's position; both stored at the token's place of the one-plane paged cache."""
     _check(kv, torch.float32, "kv"); _check(norm_w, torch.float32, "norm_w"); _check(freq, torch.float32, "freq")
     _run("hb_latent_kv_store", dtype_code(cache.dtype), kv.data_ptr(), kv.stride(0), norm_w.data_ptr(), float(eps),
-         freq.data_ptr(), float(mscale), int(rank), int(rot), tok_seq.data_ptr(), tok_pos.data_ptr(), seq_pages.data_ptr(),
+         freq.data_ptr(), float(mscale), 1 if halves else 0, int(rank), int(rot), tok_seq.data_ptr(), tok_pos.data_ptr(), seq_pages.data_ptr(),
          seq_pages.stride(0), cache.data_ptr(), kv.shape[0], int(page_size), _stream())
 
 
 def rotate_heads(src, src_head_stride, src_offset, out, out_head_stride, out_offset, freq, mscale, tok_pos, heads, rot,
-                 scale=1.0) -> None:
+                 scale=1.0, halves=True) -> None:
     """out[t, h*out_head_stride + out_offset + ..rot] = scale * rotation of src[t, h*src_head_stride + src_offset + ..rot]
-    at position tok_pos[t] (pairs (i, i + rot/2), angle p * freq[i], cos and sin times mscale)."""
+    at position tok_pos[t] (pairs (i, i + rot/2), or (2i, 2i + 1) without `halves`; angle p * freq[i], cos and sin times mscale)."""
     _check(src, torch.float32, "src"); _check(out, torch.float32, "out"); _check(freq, torch.float32, "freq")
     _run("hb_rotate_heads", src.data_ptr(), src.stride(0), int(src_head_stride), int(src_offset), out.data_ptr(), out.stride(0),
-         int(out_head_stride), int(out_offset), freq.data_ptr(), float(mscale), tok_pos.data_ptr(), src.shape[0], int(heads),
+         int(out_head_stride), int(out_offset), freq.data_ptr(), float(mscale), 1 if halves else 0, tok_pos.data_ptr(), src.shape[0], int(heads),
          int(rot), float(scale), _stream())
 
 
@@ -539,13 +554,14 @@ def add_row_bias(y, bias) -> None:
     _run("hb_axpby", y.data_ptr(), y.stride(0), 1.0, bias.data_ptr(), 0, 1.0, y.shape[0], y.shape[1], _stream())
 
 
-def bias_glu(gu, bias, out, interleave, act) -> None:
-    """out = act(gate + b) * (up + b) from float sums gu [T, 2 inter] (bias in gu's column layout, or None)."""
+def bias_glu(gu, bias, out, interleave, act, act_limit=0.0) -> None:
+    """out = act(gate + b) * (up + b) from float sums gu [T, 2 inter] (bias in gu's column layout, or None);
+    act ACT_SWISH_CLAMP takes `act_limit`."""
     _check(gu, torch.float32, "gu"); _check(out, None, "out")
     if bias is not None:
         _check(bias, torch.float32, "bias")
     _run("hb_bias_glu", dtype_code(out.dtype), gu.data_ptr(), gu.stride(0), _ptr(bias), out.data_ptr(), out.stride(0),
-         gu.shape[0], out.shape[1], int(interleave), int(act), _stream())
+         gu.shape[0], out.shape[1], int(interleave), int(act), float(act_limit), _stream())
 
 
 def tanh_cap(x, cap) -> None:
@@ -554,8 +570,8 @@ def tanh_cap(x, cap) -> None:
     _run("hb_tanh_cap", x.data_ptr(), x.stride(0), float(cap), x.shape[0], x.shape[1], _stream())
 
 
-def short_conv(inp, w, state, batch, out, add_input=False, silu=False) -> None:
-    """A causal convolution over time per channel: out_t = (in_t +) sum_j w[:, j] in_{t - taps + 1 + j} (then silu);
+def short_conv(inp, w, state, batch, out, add_input=False, silu=False, bias=None) -> None:
+    """A causal convolution over time per channel: out_t = (in_t +) (bias +) sum_j w[:, j] in_{t - taps + 1 + j} (then silu);
     inp float [T, C] (rows may be strided), w float [C, taps], state float [slots, taps - 1, C] (the sequence's
     last inputs: read for a step's first tokens, then replaced by the step's last inputs), out [T, C] in its dtype."""
     _check(inp, torch.float32, "inp"); _check(w, torch.float32, "w"); _check(out, None, "out")
@@ -566,7 +582,9 @@ def short_conv(inp, w, state, batch, out, add_input=False, silu=False) -> None:
             raise BackendError(f"short_conv: state of shape {tuple(state.shape)} does not hold {taps - 1} inputs of {inp.shape[1]} channels")
     if not w.is_contiguous():
         raise BackendError("short_conv: w must be contiguous")
-    _run("hb_short_conv", dtype_code(out.dtype), inp.data_ptr(), inp.stride(0), w.data_ptr(), _ptr(state),
+    if bias is not None:
+        _check(bias, torch.float32, "bias")
+    _run("hb_short_conv", dtype_code(out.dtype), inp.data_ptr(), inp.stride(0), w.data_ptr(), _ptr(bias), _ptr(state),
          batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), batch.seq_pos0.data_ptr(), out.data_ptr(), out.stride(0),
          batch.n_seqs, batch.max_q_len, inp.shape[1], taps, 1 if add_input else 0, 1 if silu else 0, _stream())
 
@@ -620,32 +638,34 @@ def linear_scan(q, k, v, state, batch, out, heads, qk_heads, dk, dv, gates=None,
          out.data_ptr(), out.stride(0), batch.n_seqs, batch.max_q_len, int(heads), int(qk_heads), int(dk), int(dv), _stream())
 
 
-def gated_rmsnorm(o, w, eps, gate, out, units, n, sigmoid_gate=False) -> None:
+def gated_rmsnorm(o, w, eps, gate, out, units, n, sigmoid_gate=False, gate_first=False) -> None:
     """out[t, u, :] = o[t, u, :] / sqrt(mean(o[t, u, :]^2) + eps) * w * act(gate[t, u, :]) for `units` runs of n columns;
     w [n] is shared by the units (units == 1: one norm over the whole row), or w [units * n] has a part for each.
-    act: silu, or the sigmoid."""
+    act: silu, or the sigmoid.  With `gate_first` the gate multiplies o before the norm: v = o * act(gate), v / rms(v) * w."""
     _check(o, torch.float32, "o"); _check(w, torch.float32, "w"); _check(gate, torch.float32, "gate"); _check(out, None, "out")
     if w.numel() not in (n, units * n):
         raise BackendError(f"gated_rmsnorm: the weight has {w.numel()} numbers, a unit {n}, all units {units * n}")
     _run("hb_gated_rmsnorm", dtype_code(out.dtype), o.data_ptr(), o.stride(0), w.data_ptr(), float(eps), gate.data_ptr(),
          gate.stride(0), out.data_ptr(), out.stride(0), o.shape[0], int(units), int(n), 1 if sigmoid_gate else 0,
-         int(n) if (units > 1 and w.numel() == units * n) else 0, _stream())
+         int(n) if (units > 1 and w.numel() == units * n) else 0, 1 if gate_first else 0, _stream())
 
 
 def qkv_rotary_cache(rows, wq, wk, eps, fqk, rot, halves, fv, batch, seq_pages, q_out, k_cache, v_cache, num_heads,
-                     num_kv_heads, dk, dv, hd, page_size, write_cache=True) -> None:
-    """Float rows [q: heads x dk | k: kv heads x dk | v: kv heads x dv]: q and k normed over the whole projection
+                     num_kv_heads, dk, dv, hd, page_size, write_cache=True, bias=None, mscale=1.0, maps=1) -> None:
+    """Float rows [q: heads x dk | k: kv heads x dk | v: kv heads x dv] (+ bias in the same layout): q and k normed over the whole projection
     (weights wq, wk; None: no norm), pair m of their first `rot` channels turned by p * fqk[m], pair m of all value
-    channels by p * fv[m] (fv None: values as they are); q into q_out (heads of hd channels), k and v into the paged
-    cache (heads of hd channels, zeros beyond dk and dv)."""
+    channels by p * fv[m] (fv None: values as they are; q's and k's cos and sin times `mscale`); q into q_out (heads of hd
+    channels), k and v into the paged cache (heads of hd channels, zeros beyond dk and dv).  With `maps` > 1 every head has
+    that many queries and keys of dk channels: the query of map m is a query head of its own (heads x maps of them in q_out)
+    whose channels from m * dk are set, a key head of the cache holds its maps side by side."""
     _check(rows, torch.float32, "rows"); _check(q_out, k_cache.dtype, "q_out")
-    for t, n in ((wq, "wq"), (wk, "wk"), (fqk, "fqk"), (fv, "fv")):
+    for t, n in ((wq, "wq"), (wk, "wk"), (fqk, "fqk"), (fv, "fv"), (bias, "bias")):
         if t is not None:
             _check(t, torch.float32, n)
-    _run("hb_qkv_rotary_cache", dtype_code(q_out.dtype), rows.data_ptr(), rows.stride(0), _ptr(wq), _ptr(wk), float(eps),
-         1 if wq is not None else 0, _ptr(fqk), int(rot), 1 if halves else 0, _ptr(fv), batch.tok_seq.data_ptr(),
+    _run("hb_qkv_rotary_cache", dtype_code(q_out.dtype), rows.data_ptr(), rows.stride(0), _ptr(bias), _ptr(wq), _ptr(wk), float(eps),
+         1 if wq is not None else 0, _ptr(fqk), int(rot), 1 if halves else 0, float(mscale), _ptr(fv), batch.tok_seq.data_ptr(),
          batch.tok_pos.data_ptr(), seq_pages.data_ptr(), seq_pages.stride(0), q_out.data_ptr(), q_out.stride(0),
-         k_cache.data_ptr(), v_cache.data_ptr(), rows.shape[0], int(num_heads), int(num_kv_heads), int(dk), int(dv), int(hd),
+         k_cache.data_ptr(), v_cache.data_ptr(), rows.shape[0], int(num_heads), int(num_kv_heads), int(maps), int(dk), int(dv), int(hd),
          int(page_size), 1 if write_cache else 0, _stream())
 
 
@@ -655,6 +675,73 @@ def rotate_heads_back(att, hd, fv, halves, tok_pos, out, num_heads, dv) -> None:
     _check(att, out.dtype, "att")
     _run("hb_rotate_heads_back", dtype_code(out.dtype), att.data_ptr(), att.stride(0), int(hd), _ptr(fv), 1 if halves else 0,
          tok_pos.data_ptr(), out.data_ptr(), out.stride(0), att.shape[0], int(num_heads), int(dv), _stream())
+
+
+def difference_heads(att, hd, lam, factor, eps, out, num_heads, dv) -> None:
+    """out[t, h, :dv] = o / sqrt(mean(o^2) + eps) * factor with o = a1 - lam * a2, a1 and a2 the first dv channels of heads 2h
+    and 2h + 1 of att (float, heads of hd channels)."""
+    _check(att, torch.float32, "att"); _check(out, None, "out")
+    _run("hb_difference_heads", dtype_code(out.dtype), att.data_ptr(), att.stride(0), int(hd), float(lam), float(factor), float(eps),
+         out.data_ptr(), out.stride(0), att.shape[0], int(num_heads), int(dv), _stream())
+
+
+def streams_join(x, y=None, mix=None, out_w=None, in_w=None, norm=None, h=None, rows=None) -> None:
+    """A stream x [T, n, D] of n copies (float).  With y [T, D]: x_t <- sum_s mix[s, t] x_s + out_w[t] y, all copies from
+    the old ones.  With h [rows, D]: h = norm of u = sum_t in_w[t] x_t (in_w None: the plain sum) in h's dtype, with norm =
+    (weight, bias or None, eps, rms): a layer norm, or an RMS norm if `rms`.  `rows` (only without y) chooses the rows of x."""
+    _check(x, torch.float32, "x")
+    if x.dim() != 3 or not x.is_contiguous():
+        raise BackendError("streams_join: x must be a contiguous [tokens, copies, width] array")
+    T, n, D = x.shape
+    for t, name in ((mix, "mix"), (out_w, "out_w"), (in_w, "in_w"), (y, "y")):
+        if t is not None:
+            _check(t, torch.float32, name)
+    if y is not None and (tuple(y.shape) != (T, D) or mix is None or tuple(mix.shape) != (n, n) or not mix.is_contiguous()
+                          or out_w is None or out_w.numel() != n):
+        raise BackendError(f"streams_join: a result of shape {[T, D]} needs a [{n}, {n}] matrix and {n} output weights")
+    if in_w is not None and in_w.numel() != n:
+        raise BackendError(f"streams_join: {in_w.numel()} input weights for {n} copies")
+    w, bias, eps, rms = norm if norm is not None else (None, None, 0.0, False)
+    for t, name in ((w, "w"), (bias, "bias")):
+        if t is not None:
+            _check(t, torch.float32, name)
+            if t.numel() != D:
+                raise BackendError(f"streams_join: the norm's {name} must have {D} numbers")
+    if h is not None:
+        _check(h, None, "h")
+        if not h.is_contiguous() or h.shape[1] != D or (rows is None and h.shape[0] != T):
+            raise BackendError("streams_join: h must be contiguous, a row of the width for every row asked for")
+    _run("hb_streams_join", dtype_code(h.dtype) if h is not None else F32, x.data_ptr(), n, _ptr(y), y.stride(0) if y is not None else 0,
+         _ptr(mix) if y is not None else None, _ptr(out_w) if y is not None else None, _ptr(in_w), _ptr(w), _ptr(bias), float(eps),
+         1 if rms else 0, _ptr(h), _ptr(rows), T if rows is None else h.shape[0], D, _stream())
+
+
+SSD_CHUNKED_MIN_TOKENS = 16
+
+
+def ssd_scan(xbc, b_off, c_off, dt, dt_bias, a_log, dskip, state, batch, out, heads, groups, n_state, dv, scratch) -> None:
+    """S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + dskip x over every sequence's tokens of the step, in order, from and
+    into state[slot] ([slots, heads, n_state, dv] float), with dt = softplus(raw + dt_bias).  xbc rows hold x (heads * dv)
+    from column 0, B from b_off and C from c_off (groups * n_state each; head h reads group h / (heads / groups)); dt raw,
+    float [T, heads]; out float [T, heads * dv].  bfloat16 steps that bring many tokens run chunk by chunk on the tensor cores."""
+    _check(xbc, None, "xbc")
+    for t, n in ((dt, "dt"), (dt_bias, "dt_bias"), (a_log, "a_log"), (dskip, "dskip"), (state, "state"), (out, "out")):
+        _check(t, torch.float32, n)
+    if not state.is_contiguous() or tuple(state.shape[1:]) != (heads, n_state, dv):
+        raise BackendError(f"ssd_scan: state of shape {tuple(state.shape)} is not [slots, {heads}, {n_state}, {dv}]")
+    args = (xbc.data_ptr(), xbc.stride(0), int(b_off), int(c_off), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr(), a_log.data_ptr(),
+            dskip.data_ptr(), state.data_ptr(), batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), out.data_ptr(), out.stride(0),
+            batch.n_seqs)
+    chunks = 0
+    if options.ssd_chunked and xbc.dtype == torch.bfloat16 and batch.max_q_len >= SSD_CHUNKED_MIN_TOKENS:
+        chunks = int(_fn("hb_ssd_chunks")(batch.n_tokens, batch.n_seqs, int(n_state), int(dv)))
+    if chunks > 0:
+        cs = scratch((chunks, heads, n_state, dv), torch.float32)
+        cd = scratch((chunks, heads), torch.float32)
+        _run("hb_ssd_chunked_bf16", *args, batch.max_q_len, int(heads), int(groups), int(n_state), int(dv), cs.data_ptr(), cd.data_ptr(),
+             _stream())
+        return
+    _run("hb_ssd_scan", dtype_code(xbc.dtype), *args, int(heads), int(groups), int(n_state), int(dv), _stream())
 
 
 def head_gate(att, hd, gate, out, num_heads, dv) -> None:
@@ -845,7 +932,7 @@ def gemm_simt(a, w, c, epilogue=EPI_STORE) -> None:
 
 def attention_simt(q, ldq, out, k_cache, v_cache, tok_seq, tok_pos, seq_pages, num_heads, num_kv_heads,
                    head_dim, page_size, scale, window, softcap=None, sink=None, gate_bias=None, out_gate=None) -> None:
-    """Any shape, both precisions.  softcap c: score <- c * tanh(score / c); sink [num_heads] float: exp(sink)
+    """Any shape, both precisions (out float or in the cache's dtype).  softcap c: score <- c * tanh(score / c); sink [num_heads] float: exp(sink)
     joins each head's softmax denominator.  v_cache may be k_cache (values that are the keys).  gate_bias
     [num_heads] float: no softmax, a visible key weighs sigmoid(score + gate_bias[head]) as it is.  out_gate
     [tokens, num_heads] float (rows may be strided): a head's result is multiplied by sigmoid(out_gate[token, head])."""
@@ -854,10 +941,10 @@ def attention_simt(q, ldq, out, k_cache, v_cache, tok_seq, tok_pos, seq_pages, n
     if gate_bias is not None:
         _check(gate_bias, torch.float32, "gate_bias")
     og, ldg = _out_gate(out_gate, out.shape[0], num_heads)
-    _run("hb_attention_simt", dtype_code(out.dtype), q.data_ptr(), int(ldq), out.data_ptr(), out.stride(0),
+    _run("hb_attention_simt", dtype_code(k_cache.dtype), q.data_ptr(), int(ldq), out.data_ptr(), out.stride(0),
          k_cache.data_ptr(), v_cache.data_ptr(), tok_seq.data_ptr(), tok_pos.data_ptr(), seq_pages.data_ptr(),
          seq_pages.stride(0), out.shape[0], num_heads, num_kv_heads, head_dim, page_size, float(scale),
-         int(window or 0), float(softcap or 0.0), _ptr(sink), _ptr(gate_bias), og, ldg, _stream())
+         int(window or 0), float(softcap or 0.0), _ptr(sink), _ptr(gate_bias), og, ldg, 1 if out.dtype == torch.float32 else 0, _stream())
 
 
 def _out_gate(out_gate, rows, num_heads):
@@ -900,12 +987,12 @@ def sample(logits, temperature, top_k, top_p, uniforms, out) -> None:
          int(top_k), float(top_p), uniforms.data_ptr(), out.data_ptr(), _sample_flags[key].data_ptr(), _stream())
 
 
-def gemm_skinny(a, w, c, epilogue=EPI_STORE) -> None:
+def gemm_skinny(a, w, c, epilogue=EPI_STORE, glu_limit=0.0) -> None:
     """c (op)= a @ w.T for at most 64 rows of a (bfloat16), streaming w once; EPI_SWIGLU: w holds
-    gate/up rows in groups of 8 and c is [M, N/2]."""
+    gate/up rows in groups of 8 and c is [M, N/2] (glu_limit > 0: the clamped activation in silu's place)."""
     _check(a, torch.bfloat16, "a"); _check(w, torch.bfloat16, "w"); _check(c, None, "c")
     _run("hb_gemm_skinny_bf16", a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), c.data_ptr(), c.stride(0),
-         a.shape[0], w.shape[0], a.shape[1], epilogue, _stream())
+         a.shape[0], w.shape[0], a.shape[1], epilogue, float(glu_limit), _stream())
 
 
 SHARED_NORM_MAX_ROWS = 16
@@ -1022,12 +1109,12 @@ def _tcgen05_workspace(device) -> None:
     _tcgen05_ws[key] = (floats, counters)
 
 
-def gemm_tcgen05(a, w, c, epilogue=EPI_STORE) -> None:
-    """c (op)= a @ w.T on tcgen05 tensor cores with TMA-fed tiles (bfloat16, K a multiple of 8)."""
+def gemm_tcgen05(a, w, c, epilogue=EPI_STORE, glu_limit=0.0) -> None:
+    """c (op)= a @ w.T on tcgen05 tensor cores with TMA-fed tiles (bfloat16, K a multiple of 8); glu_limit as in gemm_skinny."""
     _check(a, torch.bfloat16, "a"); _check(w, torch.bfloat16, "w"); _check(c, None, "c")
     _tcgen05_workspace(c.device)
     _run("hb_gemm_tcgen05_bf16", a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), c.data_ptr(), c.stride(0),
-         a.shape[0], w.shape[0], a.shape[1], epilogue, _error_flag(a.device).data_ptr(), _stream())
+         a.shape[0], w.shape[0], a.shape[1], epilogue, float(glu_limit), _error_flag(a.device).data_ptr(), _stream())
 
 
 _stream_bufs: dict = {}
@@ -1096,15 +1183,15 @@ def _stream_buffers(device):
     return _stream_bufs[key]
 
 
-def gemm_stream(a, w, c, epilogue=EPI_STORE) -> None:
+def gemm_stream(a, w, c, epilogue=EPI_STORE, glu_limit=0.0) -> None:
     """c (op)= a @ w.T for at most 64 rows of a (bfloat16): weights streamed once through TMA into
-    tcgen05 tensor cores, K cut into slices that the last-arriving CTA of a tile sums in order."""
+    tcgen05 tensor cores, K cut into slices that the last-arriving CTA of a tile sums in order; glu_limit as in gemm_skinny."""
     _check(a, torch.bfloat16, "a"); _check(w, torch.bfloat16, "w"); _check(c, None, "c")
     scratch, counters = _stream_buffers(a.device)
     if w.shape[0] > STREAM_COUNTERS * 128:
         raise BackendError(f"gemm_stream: {w.shape[0]} weight rows exceed the {STREAM_COUNTERS * 128} the counters cover")
     _run("hb_gemm_stream_bf16", a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), c.data_ptr(), c.stride(0),
-         a.shape[0], w.shape[0], a.shape[1], epilogue, scratch.data_ptr(), scratch.numel(), counters.data_ptr(),
+         a.shape[0], w.shape[0], a.shape[1], epilogue, float(glu_limit), scratch.data_ptr(), scratch.numel(), counters.data_ptr(),
          counters.numel(), _error_flag(a.device).data_ptr(), _stream())
 
 
@@ -1175,9 +1262,12 @@ def gemm(a, w: torch.Tensor, c: torch.Tensor, epilogue: int = EPI_STORE, next_no
         gemm_simt(a, w, c, epilogue)
 
 
-def gemm_swiglu(a, wgu: torch.Tensor, out: torch.Tensor, interleave: int, scratch) -> None:
-    """out = silu(gate) * up with [gate | up] = a @ wgu.T.  Fused into the product where a kernel can;
-    otherwise the product goes to `scratch(shape, dtype)` and the SwiGLU kernel follows."""
+def gemm_swiglu(a, wgu: torch.Tensor, out: torch.Tensor, interleave: int, scratch, glu_limit: float = 0.0) -> None:
+    """out = silu(gate) * up with [gate | up] = a @ wgu.T (glu_limit > 0: the clamped activation ACT_SWISH_CLAMP with that
+    limit instead).  Fused into the product where a kernel can; otherwise the product goes to `scratch(shape, dtype)` and
+    an activation kernel follows."""
+    if isinstance(a, PendingNorm) and glu_limit > 0.0:
+        a = _plain_input(a, scratch)
     if isinstance(a, PendingNorm):
         if interleave == 8 and _skinny_ok(a.xw, wgu) and a.xw.shape[0] <= SHARED_NORM_MAX_ROWS:
             gemm_skinny_norm(a, wgu, out, EPI_SWIGLU)
@@ -1188,10 +1278,15 @@ def gemm_swiglu(a, wgu: torch.Tensor, out: torch.Tensor, interleave: int, scratc
             return
         a = _plain_input(a, scratch)
     if interleave == 8 and _skinny_ok(a, wgu):
-        _decode_gemm(a, wgu)(a, wgu, out, EPI_SWIGLU)
+        _decode_gemm(a, wgu)(a, wgu, out, EPI_SWIGLU, glu_limit)
         return
     if interleave == 8 and _tcgen05_ok(a, wgu):
-        gemm_tcgen05(a, wgu, out, EPI_SWIGLU)
+        gemm_tcgen05(a, wgu, out, EPI_SWIGLU, glu_limit)
+        return
+    if glu_limit > 0.0:
+        gu = scratch((a.shape[0], wgu.shape[0]), torch.float32)
+        gemm(a, wgu, gu, EPI_STORE_F32)
+        bias_glu(gu, None, out, interleave, ACT_SWISH_CLAMP, glu_limit)
         return
     gu = scratch((a.shape[0], wgu.shape[0]), a.dtype)
     gemm(a, wgu, gu)
@@ -1225,9 +1320,11 @@ def decode_splits(n_seqs: int, num_kv_heads: int, max_tiles: int, device=None) -
 
 
 def attention_decode(q, ldq, out, k_cache, v_cache, seq_len, seq_pages, scratch, num_heads, num_kv_heads,
-                     head_dim, page_size, nsplit, scale, window, softcap=None, sink=None, gate_bias=None, out_gate=None) -> None:
+                     head_dim, page_size, nsplit, scale, window, softcap=None, sink=None, gate_bias=None, out_gate=None,
+                     difference=None) -> None:
     """One query per sequence (row b of q) over the cache; scratch holds the splits' partial results.
-    softcap, sink and gate_bias as in `attention`; the sink joins the denominator where the splits are combined."""
+    softcap, sink, gate_bias and difference as in `attention`; the sink joins the denominator, and the difference is
+    taken, where the splits are combined."""
     if sink is not None:
         _check(sink, torch.float32, "sink")
     if gate_bias is not None:
@@ -1239,7 +1336,12 @@ def attention_decode(q, ldq, out, k_cache, v_cache, seq_len, seq_pages, scratch,
     _run("hb_attention_decode_bf16", q.data_ptr(), int(ldq), out.data_ptr(), out.stride(0), k_cache.data_ptr(),
          v_cache.data_ptr(), seq_len.data_ptr(), seq_pages.data_ptr(), seq_pages.stride(0), scratch.data_ptr(),
          n, num_heads, num_kv_heads, head_dim, page_size, int(nsplit), float(scale), int(window or 0),
-         float(softcap or 0.0), _ptr(sink), _ptr(gate_bias), *_out_gate(out_gate, n, num_heads), _stream())
+         float(softcap or 0.0), _ptr(sink), _ptr(gate_bias), *_out_gate(out_gate, n, num_heads), *_difference(difference), _stream())
+
+
+def _difference(d):
+    """(lambda, factor, eps, dv) of a difference of two maps; dv 0 without one."""
+    return (0.0, 0.0, 0.0, 0) if d is None else (float(d[0]), float(d[1]), float(d[2]), int(d[3]))
 
 
 _DECODE_COUNTERS = 65536
@@ -1274,8 +1376,8 @@ def attention_decode_fused(qkv, out, k_cache, v_cache, q_weight, k_weight, eps, 
 def attention_prefill(q, ldq, out, k_cache, v_cache, seq_start, seq_pos0, seq_pages, n_seqs, max_q_len,
                       num_heads, num_kv_heads, head_dim, page_size, scale, window, softcap=None, sink=None,
                       gate_bias=None, out_gate=None) -> None:
-    """Causal attention of packed query rows (seq_start marks the sequences) over the cache."""
-    _check(out, torch.bfloat16, "out")
+    """Causal attention of packed query rows (seq_start marks the sequences) over the cache; out bfloat16 or float."""
+    _check(out, None, "out")
     if sink is not None:
         _check(sink, torch.float32, "sink")
     if gate_bias is not None:
@@ -1283,14 +1385,15 @@ def attention_prefill(q, ldq, out, k_cache, v_cache, seq_start, seq_pos0, seq_pa
     _run("hb_attention_prefill_bf16", q.data_ptr(), int(ldq), out.data_ptr(), out.stride(0), k_cache.data_ptr(),
          v_cache.data_ptr(), seq_start.data_ptr(), seq_pos0.data_ptr(), seq_pages.data_ptr(), seq_pages.stride(0),
          int(n_seqs), int(max_q_len), num_heads, num_kv_heads, head_dim, page_size, float(scale), int(window or 0),
-         float(softcap or 0.0), _ptr(sink), _ptr(gate_bias), *_out_gate(out_gate, out.shape[0], num_heads), _stream())
+         float(softcap or 0.0), _ptr(sink), _ptr(gate_bias), *_out_gate(out_gate, out.shape[0], num_heads),
+         1 if out.dtype == torch.float32 else 0, _stream())
 
 
 def attention_prefill_tc(q, ldq, out, k_cache, v_cache, seq_start, seq_pos0, seq_pages, n_seqs, max_q_len,
                          num_heads, num_kv_heads, head_dim, page_size, scale, window, softcap=None, sink=None,
                          gate_bias=None, out_gate=None) -> None:
     """The same on tcgen05 tensor cores (head sizes 64 and 128): S and O in tensor memory."""
-    _check(out, torch.bfloat16, "out")
+    _check(out, None, "out")
     if sink is not None:
         _check(sink, torch.float32, "sink")
     if gate_bias is not None:
@@ -1299,7 +1402,7 @@ def attention_prefill_tc(q, ldq, out, k_cache, v_cache, seq_start, seq_pos0, seq
          k_cache.data_ptr(), v_cache.data_ptr(), k_cache.shape[0], seq_start.data_ptr(), seq_pos0.data_ptr(),
          seq_pages.data_ptr(), seq_pages.stride(0), int(n_seqs), int(max_q_len), num_heads, num_kv_heads, head_dim,
          page_size, float(scale), int(window or 0), float(softcap or 0.0), _ptr(sink), _ptr(gate_bias),
-         *_out_gate(out_gate, out.shape[0], num_heads), _error_flag(out.device).data_ptr(), _work_counter(out.device).data_ptr(),
+         *_out_gate(out_gate, out.shape[0], num_heads), 1 if out.dtype == torch.float32 else 0, _error_flag(out.device).data_ptr(), _work_counter(out.device).data_ptr(),
          _stream())
 
 
@@ -1316,12 +1419,12 @@ def _work_counter(device) -> torch.Tensor:
 
 
 def _prefill_tc_ok(q, ldq, out, head_dim, page_size) -> bool:
-    return (options.prefill_attention == "tcgen05" and out.dtype == torch.bfloat16 and head_dim in (64, 128) and page_size % 64 == 0
+    return (options.prefill_attention == "tcgen05" and q.dtype == torch.bfloat16 and head_dim in (64, 128) and page_size % 64 == 0
             and ldq % 8 == 0 and out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0)
 
 
-def _prefill_kernel_ok(out, head_dim, page_size) -> bool:
-    return out.dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256 and page_size % 64 == 0
+def _prefill_kernel_ok(q, head_dim, page_size) -> bool:
+    return q.dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256 and page_size % 64 == 0
 
 
 def _decode_kernel_ok(out, num_heads, num_kv_heads, head_dim, page_size) -> bool:
@@ -1330,7 +1433,7 @@ def _decode_kernel_ok(out, num_heads, num_kv_heads, head_dim, page_size) -> bool
 
 
 def attention(q, ldq, out, k_cache, v_cache, batch, num_heads, num_kv_heads, head_dim, page_size,
-              scale, window, seq_pages, scratch=None, softcap=None, sink=None, gate_bias=None, out_gate=None) -> None:
+              scale, window, seq_pages, scratch=None, softcap=None, sink=None, gate_bias=None, out_gate=None, difference=None) -> None:
     """Attention of every token of the step over its sequence's cached keys and values.
 
     bfloat16 steps of one token per sequence take the split-key tensor-core kernel, other bfloat16
@@ -1338,7 +1441,25 @@ def attention(q, ldq, out, k_cache, v_cache, batch, num_heads, num_kv_heads, hea
     the any-shape kernel.  Every kernel takes a cap on the scores (softcap c: s <- c * tanh(s / c)) and a sink
     (a float per query head whose exponential joins the softmax's denominator); v_cache may be k_cache.  With
     `gate_bias` (a float per query head) there is no softmax: a visible key weighs sigmoid(score + gate_bias[head]).  With
-    `out_gate` (float [tokens, num_heads]) a head's result is multiplied by sigmoid(out_gate[token, head]) before it is rounded."""
+    `out_gate` (float [tokens, num_heads]) a head's result is multiplied by sigmoid(out_gate[token, head]) before it is rounded.
+
+    `difference` = (lambda, factor, eps, dv): query heads 2h and 2h + 1 are two attention maps over the same values; out
+    [tokens, num_heads / 2 * dv] receives (a1 - lambda a2) / sqrt(mean(.^2) + eps) * factor of their first dv channels,
+    taken from the float results: where the key ranges of a decode step are combined, by a kernel of its own otherwise."""
+    if difference is not None and not (options.attention != "simt" and batch.is_decode
+                                       and _decode_kernel_ok(out, num_heads, num_kv_heads, head_dim, page_size)):
+        lam, factor, eps, dv = difference
+        maps = scratch((out.shape[0], num_heads * head_dim), torch.float32)
+        _attention_rows(q, ldq, maps, k_cache, v_cache, batch, num_heads, num_kv_heads, head_dim, page_size, scale, window, seq_pages,
+                        None, softcap, sink, gate_bias, out_gate)
+        difference_heads(maps, head_dim, lam, factor, eps, out, num_heads // 2, dv)
+        return
+    _attention_rows(q, ldq, out, k_cache, v_cache, batch, num_heads, num_kv_heads, head_dim, page_size, scale, window, seq_pages,
+                    scratch, softcap, sink, gate_bias, out_gate, difference)
+
+
+def _attention_rows(q, ldq, out, k_cache, v_cache, batch, num_heads, num_kv_heads, head_dim, page_size, scale, window, seq_pages,
+                    scratch, softcap, sink, gate_bias, out_gate, difference=None) -> None:
     if options.attention == "simt":
         attention_simt(q, ldq, out, k_cache, v_cache, batch.tok_seq, batch.tok_pos, seq_pages, num_heads,
                        num_kv_heads, head_dim, page_size, scale, window, softcap, sink, gate_bias, out_gate)
@@ -1348,14 +1469,14 @@ def attention(q, ldq, out, k_cache, v_cache, batch, num_heads, num_kv_heads, hea
         nsplit = decode_splits(batch.n_seqs, num_kv_heads, tiles)
         buf = scratch((attention_decode_scratch_floats(batch.n_seqs, num_heads, head_dim, nsplit),), torch.float32)
         attention_decode(q, ldq, out, k_cache, v_cache, batch.seq_len, seq_pages, buf, num_heads, num_kv_heads,
-                         head_dim, page_size, nsplit, scale, window, softcap, sink, gate_bias, out_gate)
+                         head_dim, page_size, nsplit, scale, window, softcap, sink, gate_bias, out_gate, difference)
         return
     if _prefill_tc_ok(q, ldq, out, head_dim, page_size):
         attention_prefill_tc(q, ldq, out, k_cache, v_cache, batch.seq_start, batch.seq_pos0, seq_pages, batch.n_seqs,
                              batch.max_q_len, num_heads, num_kv_heads, head_dim, page_size, scale, window, softcap, sink, gate_bias,
                              out_gate)
         return
-    if _prefill_kernel_ok(out, head_dim, page_size):
+    if _prefill_kernel_ok(q, head_dim, page_size):
         attention_prefill(q, ldq, out, k_cache, v_cache, batch.seq_start, batch.seq_pos0, seq_pages, batch.n_seqs,
                           batch.max_q_len, num_heads, num_kv_heads, head_dim, page_size, scale, window, softcap, sink, gate_bias,
                           out_gate)

@@ -43,5 +43,7 @@ class KernelOptions:
     moe_grouped: bool = True
     # ... and, for gated experts with silu and 512 (token, expert) pairs or more, those tiles on tcgen05.
     moe_tc: bool = True
+    # State-space recurrence, bfloat16, steps that bring many tokens: 64 tokens at a time on the tensor cores.
+    ssd_chunked: bool = True
     # Steps of 512 rows and more, heads of 128: per-head norm, rotation and cache write in the q/k/v product's epilogue.
     qkv_epilogue: bool = True

@@ -28,6 +28,10 @@ after the projection (its last inputs are state of the sequence); sigmoid weight
 every visible key with nothing normalised over the keys; one output gate per token and head, sigmoid(G h), whose
 rows are part of the one projection; and a mixer without keys and values of its own, whose schedule step reads
 another step's cache with its own queries, window and gates.
+It also takes biases on the projections, scaled rotary frequencies (cos and sin times a constant) and `difference`: two
+attention maps per head over the same values.  Their keys lie side by side in one cache head (so the values are stored
+once), the query of either map is a query head that is zero in the other map's channels, and the attention kernels run
+over 2 x heads such query heads; the difference, its norm and its factor are taken from their float results.
 """
 
 from __future__ import annotations
@@ -54,8 +58,8 @@ class AttentionMixer(Mixer):
         # the plain form (no option set) keeps the path with the fused kernels of the dense decoder
         self.plain = not (spec.bias or spec.values_are_keys or spec.q_temperature or spec.softcap or spec.sink)
         self.pairs = bool(spec.whole_qk_norm or spec.value_dim is not None or spec.value_rotation is not None
-                          or getattr(spec.position, "kind", None) == "rope_pairs" or spec.key_weights != "softmax"
-                          or spec.conv_taps is not None or spec.head_gate or spec.reads_kv)
+                          or getattr(spec.position, "kind", None) in ("rope_pairs", "scaled_rope") or spec.key_weights != "softmax"
+                          or spec.difference is not None or spec.conv_taps is not None or spec.head_gate or spec.reads_kv)
         if self.pairs:
             self._init_pairs()
             return
@@ -75,16 +79,21 @@ class AttentionMixer(Mixer):
     # -- the third form ------------------------------------------------------------------------
     def _init_pairs(self):
         s = self.spec
-        if not self.plain or s.qk_norm is not None and not s.whole_qk_norm:
+        if s.values_are_keys or s.q_temperature or s.softcap or s.sink or s.qk_norm is not None and not s.whole_qk_norm:
             raise ConfigError("attention with rotated pairs, a norm over the whole projection or rotated values has "
-                              "none of the other options (biases, shared values, temperature, cap, sink, head norm)")
+                              "none of the other options (shared values, temperature, cap, sink, head norm)")
         if s.whole_qk_norm and s.qk_norm is None:
             raise ConfigError("a norm over the whole q and k projections needs its eps (qk_norm)")
         self.plain = False
         self.dk = s.head_dim
         self.dv = s.value_dim if s.value_dim is not None else s.head_dim
-        self.hd = max(self.dk, self.dv)              # the cache's and the attention kernels' head size
-        self.q_dim, self.kv_dim = self.nh * self.dk, self.nkv * self.dk
+        self.maps = 1 if s.difference is None else 2
+        self.hd = max(self.maps * self.dk, self.dv)  # the cache's and the attention kernels' head size
+        if self.maps > 1:
+            if s.key_weights != "softmax" or s.head_gate or s.reads_kv or s.value_rotation is not None:
+                raise ConfigError("the difference of two attention maps has softmax weights, keys of its own, no gates and no rotated values")
+            self.hd = (self.hd + 15) // 16 * 16      # what the tensor-core kernels take; the channels added are zeros
+        self.q_dim, self.kv_dim = self.nh * self.maps * self.dk, self.nkv * self.maps * self.dk
         if s.key_weights not in ("softmax", "sigmoid"):
             raise ConfigError(f"unknown key weights {s.key_weights!r}: softmax, sigmoid")
         self.sigmoid_keys = s.key_weights == "sigmoid"
@@ -95,7 +104,7 @@ class AttentionMixer(Mixer):
         # what the projection's rows hold: q, then (unless another step's are read) k and v, then one gate per head
         self.qkv_dim = self.q_dim + (0 if self.reads_kv else self.kv_dim + self.nkv * self.dv)
         self.proj_dim = self.qkv_dim + (self.nh if s.head_gate else 0)
-        self.key_bias = self.w_conv = None
+        self.key_bias = self.w_conv = self.difference = None
         self.value_position = build_part("position", s.value_rotation, rt=self.rt) if s.value_rotation is not None else None
         if self.value_position is not None and self.value_position.rotary_dim != self.dv:
             raise ConfigError(f"values of {self.dv} channels are turned over all of them, not {self.value_position.rotary_dim}")
@@ -123,6 +132,12 @@ class AttentionMixer(Mixer):
             p[s.key_bias_name] = ParamSpec((self.nh,), role="vector", init="wide")
         if s.head_gate:
             p[s.head_gate_name] = ParamSpec((self.nh, s.hidden_size))
+        if s.bias:
+            for n, rows in self._projections():
+                p[n + s.bias_suffix] = ParamSpec((rows,), role="vector", init="normal")
+        if self.maps > 1:
+            for n in s.difference_names:
+                p[n] = ParamSpec((self.dk,), role="vector", init="zeros_noise")
         if s.whole_qk_norm:
             p[s.norm_names[0]] = ParamSpec((self.q_dim,), role="vector", init="ones_noise")
             p[s.norm_names[1]] = ParamSpec((self.kv_dim,), role="vector", init="ones_noise")
@@ -135,6 +150,12 @@ class AttentionMixer(Mixer):
         self.wo = tensors[self.n_o].contiguous()
         if self.taps:
             self.w_conv = torch.cat([tensors[n + s.conv_suffix] for n, _ in self._projections()], dim=0).contiguous()
+        if s.bias:
+            self.bias = torch.cat([tensors[n + s.bias_suffix] for n, _ in self._projections()], dim=0).contiguous()
+        if self.maps > 1:
+            a1, b1, a2, b2 = (tensors[n].double() for n in s.difference_names)
+            lam = float(torch.exp((a1 * b1).sum()) - torch.exp((a2 * b2).sum())) + float(s.difference)
+            self.difference = (lam, 1.0 - float(s.difference), s.difference_eps, self.dv)
         if self.sigmoid_keys:
             self.key_bias = tensors[s.key_bias_name].contiguous()
         if s.whole_qk_norm:
@@ -146,10 +167,15 @@ class AttentionMixer(Mixer):
         proj = ws.take((T, self.proj_dim), torch.float32)
         ops.gemm(h, self.wqkv, proj, ops.EPI_STORE_F32, scratch=ws.take)
         rows = proj
+        bias = self.bias
         if self.taps:
+            if bias is not None:
+                ops.add_row_bias(proj[:, :self.qkv_dim], bias)       # before the convolution: part of the projection
+                bias = None
             rows = ws.take((T, self.qkv_dim), torch.float32)
             ops.short_conv(proj[:, :self.qkv_dim], self.w_conv, cache.states.get("conv"), batch, rows)
-        q = ws.take((T, self.nh * self.hd), h.dtype)
+        nq = self.nh * self.maps                     # query heads as the attention kernels see them
+        q = ws.take((T, nq * self.hd), h.dtype)
         pages = batch.pages[cache.kv_group]
         pos, vpos = self.position, self.value_position
         halves = pos.halves if pos is not None else (vpos.halves if vpos is not None else False)
@@ -157,7 +183,14 @@ class AttentionMixer(Mixer):
         ops.qkv_rotary_cache(rows, self.q_norm, self.k_norm, s.qk_norm.eps if s.qk_norm is not None else 0.0,
                              pos.freq if pos is not None else None, pos.rotary_dim if pos is not None else 0, halves, fv,
                              batch, pages, q, cache.k, cache.v, self.nh, self.nkv, self.dk, self.dv, self.hd,
-                             cache.page_size, write_cache=cache.writes_kv and not self.reads_kv)
+                             cache.page_size, write_cache=cache.writes_kv and not self.reads_kv, bias=bias,
+                             mscale=pos.mscale if pos is not None else 1.0, maps=self.maps)
+        if self.maps > 1:
+            y = ws.take((T, self.nh * self.dv), h.dtype)
+            ops.attention(q, q.stride(0), y, cache.k, cache.v, batch, nq, self.nkv, self.hd, cache.page_size, s.scale, s.window, pages,
+                          scratch=ws.take, difference=self.difference)
+            ops.gemm(y, self.wo, residual, ops.EPI_RESIDUAL if accumulate else ops.EPI_STORE_F32, scratch=ws.take)
+            return
         att = ws.take((T, self.nh * self.hd), h.dtype)
         # the gate per token and head multiplies a head's float result inside the attention kernel, before it is rounded
         ops.attention(q, q.stride(0), att, cache.k, cache.v, batch, self.nh, self.nkv, self.hd, cache.page_size, s.scale,

@@ -82,6 +82,11 @@ class Norm(Part):
         before it and a product after it can compute between them; else None."""
         return None
 
+    def as_stream_norm(self):
+        """(weight [D] float, bias [D] float or None, eps, rms) if this is a layer norm, or (rms True) a plain RMS norm, which
+        the kernel that joins a sublayer's result to a stream of several copies can apply to what it mixes; else None."""
+        return None
+
 
 class Mixer(Part):
     def cache_need(self) -> CacheNeed:
@@ -103,6 +108,8 @@ class Block(Part):
     # True if forward() takes the keywords `normed` and `next_norm` below; a block without the flag is
     # called as forward(x, batch, cache) and its neighbours run their norms themselves.
     chains_norms = False
+    # How many copies of the stream forward() works on, as an array [T, streams, H]; None: one stream [T, H].
+    streams = None
 
     def first_norm(self):
         """The norm this block applies to the stream before anything else, which the block before
@@ -110,7 +117,9 @@ class Block(Part):
         return None
 
     def forward(self, x, batch, cache, normed=None, next_norm=None):
-        """Update x.  With `chains_norms`: `normed` is the PendingNorm of x under `first_norm()`,
+        """Update x.  `next_norm` is whatever the following block's `first_norm().shareable()` gave, None if nothing;
+        `normed` is what the block before returned for it: a PendingNorm, or the finished input as a tensor.
+          With `chains_norms`: `normed` is the PendingNorm of x under `first_norm()`,
         begun by the block before (or None); `next_norm` is the following block's first norm as
         (weight, eps); the block may return the PendingNorm of its result under it, or None."""
         raise NotImplementedError

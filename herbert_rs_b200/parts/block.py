@@ -422,6 +422,116 @@ class SandwichBlock(Block):
         return h if next_norm is not None else None
 
 
+class _StreamEntry:
+    """How a block of several streams takes its first input, for the block before it to begin."""
+
+    def __init__(self, block):
+        self.block = block
+
+    def shareable(self):
+        return self.block.hc[1][0], self.block.norm1.as_stream_norm()
+
+
+class StreamsBlock(Block):
+    """A residual of n copies X_1 .. X_n ("hyper-connections").  For sublayer q (1: mixer, 2: feed-forward):
+
+        u = sum_s in_q[s] X_s;   y = sublayer(norm_q(u));   X_t <- sum_s mix_q[s, t] X_s + out_q[t] y   (all from the old ones)
+
+    A sublayer stores its result as floats; the mixing of the copies, the next sublayer's input mixture and its norm are one
+    kernel, across the block's end too (`first_norm` tells the block before what this one reads), so that between two
+    sublayers every copy is read and written once.  The spec may leave out the feed-forward."""
+
+    chains_norms = True
+
+    def __init__(self, spec, rt):
+        self.spec, self.rt = spec, rt
+        self.streams = int(spec.streams)
+        if self.streams < 1:
+            raise ConfigError("a block of several streams has at least one")
+        self.norm1 = build_part("norm", spec.norm1, rt=rt)
+        self.mixer = build_part("mixer", spec.mixer, rt=rt)
+        self.ffn = build_part("ffn", spec.ffn, rt=rt) if spec.ffn is not None else None
+        self.norm2 = build_part("norm", spec.norm2, rt=rt) if self.ffn is not None else None
+        for norm in (self.norm1, self.norm2):
+            if norm is not None and norm.as_stream_norm() is None:
+                raise ConfigError("a block of several streams applies a layer norm or a plain RMS norm")
+        for part in (self.mixer, self.ffn):
+            if part is not None and not part.can_store:
+                raise ConfigError(f"{type(part).__name__} cannot store its result apart from the residual stream, "
+                                  "which a block of several streams needs")
+        self._names = dict(spec.names)
+        self.hc = {}                   # sublayer -> (in [n], out [n], mix [n, n])
+
+    @property
+    def graph_safe(self):
+        return all(p.graph_safe for _, p in self.children())
+
+    def children(self):
+        parts = [("norm1", self.norm1), ("mixer", self.mixer)]
+        if self.ffn is not None:
+            parts += [("norm2", self.norm2), ("ffn", self.ffn)]
+        return tuple(parts)
+
+    def _key(self, local, name):
+        prefix = self._names[local]
+        return f"{prefix}.{name}" if prefix else name
+
+    def _stream_tensors(self, q):
+        return tuple(n.format(q=q) for n in self.spec.stream_names)
+
+    def param_specs(self):
+        out = {self._key(local, name): ps for local, part in self.children() for name, ps in part.param_specs().items()}
+        n = self.streams
+        for q in (1, 2) if self.ffn is not None else (1,):
+            a, b, m = self._stream_tensors(q)
+            out[a] = ParamSpec((n,), role="vector", init="ones_noise")
+            out[b] = ParamSpec((n,), role="vector", init="ones_noise")
+            out[m] = ParamSpec((n, n), role="vector", init="zeros_noise")
+        return out
+
+    def load(self, tensors):
+        for local, part in self.children():
+            part.load({name: tensors[self._key(local, name)] for name in part.param_specs()})
+        for q in (1, 2) if self.ffn is not None else (1,):
+            self.hc[q] = tuple(tensors[t].contiguous() for t in self._stream_tensors(q))
+
+    def weight_bytes(self):
+        return sum(p.weight_bytes() for _, p in self.children())
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def first_norm(self):
+        return _StreamEntry(self)
+
+    def _join(self, x, y, q, entry):
+        """X <- mixed X + out y; returns the next sublayer's input where `entry` = (in weights, norm) is given."""
+        _, out_w, mix = self.hc[q]
+        if entry is None:
+            ops.streams_join(x, y, mix, out_w)
+            return None
+        h = self.rt.workspace.take(y.shape, self.rt.dtype)
+        ops.streams_join(x, y, mix, out_w, in_w=entry[0], norm=entry[1], h=h)
+        return h
+
+    def forward(self, x, batch, cache, normed=None, next_norm=None):
+        ws = self.rt.workspace
+        shape = (x.shape[0], x.shape[2])
+        h = normed
+        if h is None:
+            h = ws.take(shape, self.rt.dtype)
+            ops.streams_join(x, in_w=self.hc[1][0], norm=self.norm1.as_stream_norm(), h=h)
+        y = ws.take(shape, torch.float32)
+        self.mixer.forward(h, y, batch, cache, accumulate=False)
+        if self.ffn is None:
+            return self._join(x, y, 1, next_norm)
+        h = self._join(x, y, 1, (self.hc[2][0], self.norm2.as_stream_norm()))
+        y = ws.take(shape, torch.float32)
+        self.ffn.forward(h, y, batch, accumulate=False)
+        return self._join(x, y, 2, next_norm)
+
+
+register_part("block", "streams", StreamsBlock)
 register_part("block", "sandwich", SandwichBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "prenorm", PreNormBlock)

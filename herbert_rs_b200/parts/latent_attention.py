@@ -100,13 +100,14 @@ class LatentAttentionMixer(Mixer):
         pages, pos = batch.pages[cache.kv_group], self.position
         freq = pos.freq if pos is not None else self.kv_norm      # unread when nothing is rotated
         mscale = pos.mscale if pos is not None else 1.0
+        halves = pos.halves if pos is not None else True
         if cache.writes_kv:
             ops.latent_kv_store(kvg, self.kv_norm, s.norm_eps, freq, mscale, rk, dr, batch.tok_seq, batch.tok_pos, pages,
-                                cache.k, cache.page_size)
+                                cache.k, cache.page_size, halves=halves)
         qa = ws.take((T, H * (rk + dr)), f32)
         ops.headwise_gemm(q, dn + dr, self.w_kup, qa, rk + dr, scale=s.scale)
         if dr:
-            ops.rotate_heads(q, dn + dr, dn, qa, rk + dr, rk, freq, mscale, batch.tok_pos, H, dr, scale=s.scale)
+            ops.rotate_heads(q, dn + dr, dn, qa, rk + dr, rk, freq, mscale, batch.tok_pos, H, dr, scale=s.scale, halves=halves)
         lat = ws.take((T, H * rk), f32)
         ops.latent_attention(qa, lat, cache.k, self.sink, batch.tok_seq, batch.tok_pos, pages, H, rk, dr, cache.page_size,
                              s.window, batch=batch, scratch=ws.take)

@@ -1,5 +1,5 @@
 """RMSNorm: y = (x / sqrt(mean(x^2) + eps)) * w, in float
-(crates/backends/backend_common/src/kernels.rs:54-64), and the layer norm with a weight and no bias.
+(crates/backends/backend_common/src/kernels.rs:54-64), and the layer norm with a weight and, if the spec asks, a bias.
 A spec with `weight_offset` c stores w - c (weights around zero with c = 1); the offset is added once,
 in float, when the tensor is loaded, so every kernel and the norm shared between two products see w."""
 
@@ -43,17 +43,42 @@ class RMSNorm(Norm):
     def shareable(self):
         return (self.weight, self.eps) if self.groups == 1 else None
 
+    def as_stream_norm(self):
+        return (self.weight, None, self.eps, True) if self.groups == 1 else None
+
 
 class LayerNorm(RMSNorm):
-    """y = (x - mean(x)) / sqrt(var(x) + eps) * w, no bias, in float (var: mean of squared deviations)."""
+    """y = (x - mean(x)) / sqrt(var(x) + eps) * w (+ b), in float (var: mean of squared deviations)."""
 
     kind = "layernorm"
 
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        self.bias_name = self.name + spec.bias_suffix if getattr(spec, "bias", False) else None
+        self.bias = None
+
+    def param_specs(self):
+        p = super().param_specs()
+        if self.bias_name:
+            p[self.bias_name] = ParamSpec((self.dim,), role="vector", init="zeros_noise")
+        return p
+
+    def load(self, tensors):
+        super().load(tensors)
+        if self.bias_name:
+            self.bias = tensors[self.bias_name].contiguous()
+
+    def weight_bytes(self):
+        return self.dim * (8 if self.bias_name else 4)
+
     def forward(self, x, out, rows=None):
-        ops.layernorm(x, self.weight, out, self.eps, rows)
+        ops.layernorm(x, self.weight, out, self.eps, rows, bias=self.bias)
 
     def shareable(self):
         return None         # the products' shared norm is the RMS form only
+
+    def as_stream_norm(self):
+        return self.weight, self.bias, self.eps, False
 
 
 register_part("norm", "rmsnorm", RMSNorm)

@@ -66,6 +66,7 @@ class ScaledRotary(Part):
 
     def __init__(self, spec, rt):
         self.rotary_dim = spec.rotary_dim
+        self.halves = True               # pair i is channels (i, i + rotary_dim / 2)
         f, self.mscale = scaled_frequencies(spec)
         self.freq = f.to(torch.float32).to(rt.device)
 
@@ -105,6 +106,7 @@ class RotaryPairs(Part):
             raise ConfigError(f"unknown layout of rotated pairs {spec.layout!r}: interleaved, halves")
         self.rotary_dim = spec.rotary_dim
         self.halves = spec.layout == "halves"
+        self.mscale = 1.0
         self.freq = pair_frequencies(spec.rotary_dim, spec.theta, spec.linear_factor,
                                      getattr(spec, "band_scaling", None)).to(rt.device) if spec.rotary_dim else None
 

@@ -1,7 +1,8 @@
 """The dense gated feed-forward: down( act(gate(h)) * up(h) ), added to the residual stream
 (crates/backends/backend_common/src/generic_mlp.rs:83-96; silu(x) = x / (1 + exp(-x)),
-kernels.rs:677-687).  act is silu unless the spec names another (gelu in its tanh or erf form, relu); the
-product's fused epilogue serves silu, the others take the product and then the activation kernel.
+kernels.rs:677-687).  act is silu unless the spec names another (gelu in its tanh or erf form, relu,
+or "swish_clamp", min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1) with a limit L); the product's fused epilogue
+serves silu and the clamped form, the others take the product and then the activation kernel.
 With `bias` every projection adds a stored vector: gate and up leave float sums, one kernel adds their
 biases, applies the activation and rounds once; the down projection's bias is added to the float result,
 or handed to a block that norms that result (`take_output_bias`), which adds it while it reads.
@@ -43,6 +44,9 @@ class SwiGLU(FeedForward):
         if act not in ops.ACTIVATIONS:
             raise ConfigError(f"unknown activation {act!r}: {', '.join(ops.ACTIVATIONS)}")
         self.act = ops.ACTIVATIONS[act]
+        self.limit = float(getattr(spec, "act_limit", 0.0))
+        if (self.act == ops.ACT_SWISH_CLAMP) != (self.limit > 0.0):
+            raise ConfigError("the clamped activation takes a limit > 0, and no other activation does")
         self.bias = bool(getattr(spec, "bias", False))
         self.bias_suffix = getattr(spec, "bias_suffix", ".b")
         self.bgu = self.bd = None
@@ -87,7 +91,7 @@ class SwiGLU(FeedForward):
         gu = ws.take((T, 2 * inter), torch.float32)
         ops.gemm(h, self.wgu, gu, ops.EPI_STORE_F32, scratch=ws.take)
         act = ws.take((T, inter), self.rt.dtype)
-        ops.bias_glu(gu, self.bgu, act, self.interleave, self.act)
+        ops.bias_glu(gu, self.bgu, act, self.interleave, self.act, self.limit)
         if accumulate:
             ops.gemm(act, self.wd, residual, ops.EPI_RESIDUAL, scratch=ws.take)
         else:
@@ -101,8 +105,8 @@ class SwiGLU(FeedForward):
             return self._forward_bias(h, residual, accumulate, with_output_bias)
         ws, T, inter = self.rt.workspace, h.shape[0], self.spec.intermediate_size
         act = ws.take((T, inter), self.rt.dtype)
-        if self.act == ops.ACT_SILU:
-            ops.gemm_swiglu(h, self.wgu, act, self.interleave, ws.take)
+        if self.act in (ops.ACT_SILU, ops.ACT_SWISH_CLAMP):
+            ops.gemm_swiglu(h, self.wgu, act, self.interleave, ws.take, self.limit)
         else:
             gu = ws.take((T, 2 * inter), self.rt.dtype)
             ops.gemm(h, self.wgu, gu, scratch=ws.take)
