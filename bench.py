@@ -245,6 +245,31 @@ def _nefivik_config(width, heads, kv_heads, dim, vdim, window, delta_heads, delt
             "layers": layers}
 
 
+def _putazen_config(width, heads, kv_heads, dim, vdim, latent_heads, latent_dim, rot_dim, latent_vdim, kv_rank, scan_heads, scan_vdim,
+                    state, groups, streams, ff, vocab, taps=4):
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "diff": 0.35,
+           "rot": {"base": 10000.0, "dims": dim, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    latent = {"heads": latent_heads, "dim": latent_dim, "rot_dim": rot_dim, "vdim": latent_vdim, "kv_rank": kv_rank,
+              "scale": (latent_dim + rot_dim) ** -0.5, "rot": {"base": 10000.0, "dims": rot_dim}}
+    scan = {"heads": scan_heads, "vdim": scan_vdim, "state": state, "groups": groups, "norm_groups": groups, "conv": taps}
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    layers = [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "mamba2", "mixer": scan, "mlp": dense},
+              {"type": "latent_attention", "mixer": latent, "mlp": dense}, {"type": "mamba2", "mixer": scan, "mlp": dense}]
+    return {"architecture": "Putazen", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "streams": streams, "layers": layers}
+
+
+PUTAZEN_SIZES = {
+    # Putazen layer sizes (differential attention, a state-space mixer of twice the width, latent attention, the state-space mixer
+    # again; four copies of the stream); beside them Begupel (the closest in its recurrence, convolution, gated norm and the
+    # norm that joins a result to the stream), Kebisun (the closest in its latent attention) and the dense decoder (attention,
+    # gated feed-forward), each of the same width and depth.  A head of 128 value channels holds two maps of 64.
+    "1k": (dict(width=1024, heads=8, kv_heads=4, dim=64, vdim=128, latent_heads=8, latent_dim=64, rot_dim=32, latent_vdim=64, kv_rank=256,
+                scan_heads=32, scan_vdim=64, state=128, groups=2, streams=4, ff=3072, vocab=32000), "1k"),
+    "2k": (dict(width=2048, heads=16, kv_heads=8, dim=64, vdim=128, latent_heads=16, latent_dim=128, rot_dim=64, latent_vdim=128,
+                kv_rank=512, scan_heads=64, scan_vdim=64, state=128, groups=4, streams=4, ff=8192, vocab=32000), "2k"),
+}
+
 NEFIVIK_SIZES = {
     # Nefivik layer sizes (two layers of windowed sigmoid attention, the second reading the first one's keys and values, two of
     # the generalised delta rule, routed experts in every layer); beside them Begupel (the closest design in its mixers:
@@ -384,6 +409,34 @@ def _launcher_work(name, n, ctx):
             return n * 6.0 * T * top * F * D, n * (min(E, T * top) * 3 * F * D * es + T * D * (es + 4))
         if name == "hb_moe_route":
             return n * 2.0 * T * ctx["experts"] * D, n * (T * D * es + ctx["experts"] * D * es)
+    elif ctx["kind"] == "putazen":
+        H, KV, dk, dv, D, S = ctx["heads"], ctx["kv_heads"], ctx["dim"], ctx["vdim"], ctx["width"], ctx["streams"]
+        sh, sv, N, G = ctx["scan_heads"], ctx["scan_vdim"], ctx["state"], ctx["groups"]
+        lh, dn, dr, lv, rk = ctx["latent_heads"], ctx["latent_dim"], ctx["rot_dim"], ctx["latent_vdim"], ctx["kv_rank"]
+        conv = sh * sv + 2 * G * N
+        if name in ("hb_attention_prefill_tc_bf16", "hb_attention_prefill_bf16", "hb_attention_decode_bf16", "hb_attention_simt"):
+            # two maps per head over one value; the zero channels of a map's query are not counted
+            return n * 2.0 * pairs * H * 2 * (dk + dv), n * (B * L * KV * (2 * dk + dv) * es + T * H * (2 * dk + dv) * es)
+        if name in ("hb_latent_attention", "hb_latent_attention_mma_bf16"):
+            return n * 2.0 * pairs * lh * (2 * rk + dr), n * (B * L * (rk + dr) * es + T * lh * (2 * rk + dr) * 4)
+        if name == "hb_headwise_gemm":
+            per = n / 2.0
+            return per * 2.0 * T * lh * rk * (dn + lv), per * (lh * rk * (dn + lv) * es + T * lh * (rk + dn + dr + rk + lv) * 4)
+        if name in ("hb_ssd_chunked_bf16", "hb_ssd_scan"):
+            # decay, update and read-out: 5 operations a state entry and token; reads x, B, C and the step sizes, writes y
+            # as floats, reads and writes every sequence's state
+            return n * 5.0 * T * sh * N * sv, n * (T * (conv * es + sh * sv * 4 + sh * 4) + 2 * B * sh * N * sv * 4)
+        if name == "hb_streams_join":     # two per layer update every copy; the first and the last only read
+            return n * 2.0 * T * D * S * (S + 2), (n - 2) * T * D * (2 * S * 4 + 4 + es) + T * D * (S * 4 + es)
+        if name == "hb_short_conv":
+            return n * 8.0 * T * conv, n * T * conv * (4 + es)
+        if name == "hb_gated_rmsnorm":
+            return n * 8.0 * T * sh * sv, n * T * sh * sv * (4 + 4 + es)
+        if name == "hb_qkv_rotary_cache":
+            rows = 2 * H * dk + KV * (2 * dk + dv)
+            return n * 6.0 * T * rows, n * T * rows * (4 + es)
+        if name == "hb_difference_heads":
+            return n * 6.0 * T * H * dv, n * T * H * dv * (8 + es)
     else:
         H, KV, hd, D = ctx["heads"], ctx["kv_heads"], ctx["head_dim"], ctx["width"]
         if name in ("hb_attention_prefill_tc_bf16", "hb_attention_prefill_bf16", "hb_attention_decode_bf16",
@@ -461,10 +514,10 @@ def _design_point(hb, ops, torch, np, cfg, ctx, pk, prompt_len, batch, steps, wa
 
 
 def run_design(args) -> int:
-    """`--design begupel|kebisun|nefivik|votapel`: prefill and decode of that design at layer sizes that resemble a
+    """`--design begupel|kebisun|nefivik|putazen|votapel`: prefill and decode of that design at layer sizes that resemble a
     real model's, beside the dense decoder of equal width, depth and feed-forward width (random weights,
     bfloat16, four layers each); Begupel also beside Kebisun with recurrent heads of equal sizes, Nefivik also beside
-    Begupel and Votapel."""
+    Begupel and Votapel, Putazen also beside Begupel and Kebisun."""
     import numpy as np
     import torch
 
@@ -476,13 +529,14 @@ def run_design(args) -> int:
     sampler.start()
     result = {}
     table, make = {"kebisun": (DESIGN_SIZES, _kebisun_config), "votapel": (VOTAPEL_SIZES, _votapel_config),
-                   "begupel": (BEGUPEL_SIZES, _begupel_config), "nefivik": (NEFIVIK_SIZES, _nefivik_config)}[args.design]
+                   "begupel": (BEGUPEL_SIZES, _begupel_config), "nefivik": (NEFIVIK_SIZES, _nefivik_config),
+                   "putazen": (PUTAZEN_SIZES, _putazen_config)}[args.design]
     for size in (sorted(table) if args.design_size == "all" else [args.design_size]):
         closest = None
         beside = None
         if args.design == "begupel":
             kb, closest, dense = table[size]
-        elif args.design == "nefivik":
+        elif args.design in ("nefivik", "putazen"):
             kb, beside = table[size]
             dense = BEGUPEL_SIZES[beside][2]
         else:
@@ -501,7 +555,9 @@ def run_design(args) -> int:
             result[size]["kebisun"] = _design_point(hb, ops, torch, np, _kebisun_config(**closest), dict(closest, kind="kebisun"), pk,
                                                     args.prompt_len, args.batch, args.steps, args.warmup, windows)
         if beside is not None:
-            for other, sizes, maker in (("begupel", BEGUPEL_SIZES, _begupel_config), ("votapel", VOTAPEL_SIZES, _votapel_config)):
+            others = {"nefivik": (("begupel", BEGUPEL_SIZES, _begupel_config), ("votapel", VOTAPEL_SIZES, _votapel_config)),
+                      "putazen": (("begupel", BEGUPEL_SIZES, _begupel_config), ("kebisun", DESIGN_SIZES, _kebisun_config))}[args.design]
+            for other, sizes, maker in others:
                 ob = sizes[beside][0]
                 result[size][other] = _design_point(hb, ops, torch, np, maker(**ob), dict(ob, kind=other), pk, args.prompt_len,
                                                     args.batch, args.steps, args.warmup, windows)
@@ -534,7 +590,7 @@ def main() -> int:
     ap.add_argument("--pdl-graph", type=int, default=None, help="programmatic dependent launch inside recorded decode steps (0, 1, 2)")
     ap.add_argument("--workload", default=None, choices=["0.6b", "32b"],
                     help="run only this workload of the baseline and print its line")
-    ap.add_argument("--design", default=None, choices=["begupel", "kebisun", "nefivik", "votapel"],
+    ap.add_argument("--design", default=None, choices=["begupel", "kebisun", "nefivik", "putazen", "votapel"],
                     help="measure this design beside the dense decoder at equal sizes instead of the headline workload")
     ap.add_argument("--design-size", default="all", choices=["all"] + sorted(DESIGN_SIZES))
     args = ap.parse_args()
