@@ -49,8 +49,8 @@ int hb_attention_prefill_bf16(const void* q, int ldq, void* out, int ldo, const 
 int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens, void* out, int ldo, const void* kcache, const
     void* vcache, int n_pages, const int* seq_start, const int* seq_pos0, const int* seq_pages, int pages_stride, int
     n_seqs, int max_q_len, int nh, int nkv, int hd, int page_size, float scale, int window, float softcap, const
-    float* sink, const float* gate_bias, const float* out_gate, int ldg, int out_f32, int* error_flag, int*
-    work_counter, void* stream);
+    float* sink, const float* gate_bias, const float* out_gate, int ldg, float diff_lambda, float diff_factor, float
+    diff_eps, int diff_dv, int* error_flag, int* work_counter, void* stream);
 
 // attention_simt.cu: attention of any shape on the CUDA cores (the 32-bit path)
 int hb_attention_simt(int dtype, const void* q, int ldq, void* out, int ldo, const void* kcache, const void* vcache,

@@ -26,6 +26,7 @@
 // query head (the row starts at m = sink, l = 1: a first key without a value).  With `gate_bias` (a number per query
 // head) there is no softmax: P = sigmoid(s * scale + gate_bias[h]) for a visible key, 0 for a masked one, O = sum P V as it
 // is; no maximum, no sum, and O is never rescaled.
+// With `diff_dv` the two heads of an item are two maps of one head, subtracted and normed in the epilogue.
 // A head pair whose second head does not exist (an odd number of query heads per key/value head)
 // runs the first head alone.  CTAs are persistent and take items from a counter, longest first.
 // Every wait on an mbarrier is bounded; a wait that runs out sets *error_flag and the CTA winds down.
@@ -57,7 +58,10 @@ struct PrefillTcArgs {
   const float* gate_bias;  // [nh] or null.  Not null: sigmoid weights (see the head of this file)
   const float* out_gate;   // [tokens, ldg] or null: head h's result of a token is multiplied by sigmoid(out_gate[token * ldg + h])
   int ldg;
-  int out_f32;             // the output is float (something follows before it is rounded)
+  // > 0: query heads 2h and 2h + 1 are two attention maps of one head: out [tokens][nh / 2][diff_dv] receives
+  // (o1 - diff_lambda o2) / sqrt(mean(.^2) + diff_eps) * diff_factor over their first diff_dv channels
+  float diff_lambda, diff_factor, diff_eps;
+  int diff_dv;
 };
 
 // One unit of work: 128 consecutive queries of two heads (or one) of one key/value head of one sequence.
@@ -157,16 +161,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   const unsigned q_s = base, k_s = q_s + 2 * TILE_BYTES, v_s = k_s + 2 * TILE_BYTES;
   const unsigned bars = v_s + 2 * TILE_BYTES;
   // barriers: 0 q_full | 1 q_empty | 2,3 k_full | 4,5 k_empty | 6,7 v_full | 8,9 v_empty | 10,11 s_full (per head)
-  //           14,15 p_ready | 17,18 o_full | 19,20 o_empty | 21,22 item_full | 23,24 item_empty
+  //           12 second map's factors | 14,15 p_ready | 17,18 o_full | 19,20 o_empty | 21,22 item_full | 23,24 item_empty
   constexpr int N_BARS = 25;
   auto bar = [&](int i) { return bars + i * 8; };
   volatile unsigned* tmem_slot = reinterpret_cast<volatile unsigned*>(gen + (bars - base) + N_BARS * 8);
   volatile int* item_ring = reinterpret_cast<volatile int*>(gen + (bars - base) + N_BARS * 8 + 8);      // [2]
+  volatile float* row_factor = reinterpret_cast<volatile float*>(gen + (bars - base) + N_BARS * 8 + 16);   // [PT_Q] (two maps subtracted)
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < N_BARS; ++i) {
-      const bool from_rows = (i == 14 || i == 15 || i == 19 || i == 20);   // the four row warps of a head
+      const bool from_rows = (i == 12 || i == 14 || i == 15 || i == 19 || i == 20);   // the four row warps of a head
       const bool from_consumers = (i == 23 || i == 24);                                          // the MMA lane and all row warps
       mbar_init(bar(i), from_rows ? 4 : (from_consumers ? 9 : 1));
     }
@@ -325,6 +330,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int r = quad * 32 + lane;              // row of the tile
     const unsigned lane_off = (unsigned)(quad * 32) << 16;
     int c_t = 0;                                 // this head's key tiles so far
+    int items_t = 0;                             // ... and items, where two maps are subtracted
     bool ok = true;
     for (int n = 0; ok; ++n) {
       const int slot = n & 1;
@@ -455,9 +461,67 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (!mbar_wait(bar(17 + t), ct & 1)) { if (lane == 0) atomicExch(a.error_flag, 36); ok = false; break; }
         tc_fence_after();
         float inv = gated ? 1.0f : (l > 0.0f ? 1.0f / l : 0.0f);
+        if (a.diff_dv > 0) {
+          // Two maps of one head: both heads of the item have the same rows, and a row's two O lie in the same lane of tensor
+          // memory.  The second map's threads leave their factor in shared memory and are done with the item; the first
+          // map's threads read both O and hand both buffers back.
+          if (t == 1) {
+            row_factor[r] = inv * a.diff_lambda;
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive_cta(bar(12));
+          } else {
+            if (!mbar_wait(bar(12), items_t & 1)) { if (lane == 0) atomicExch(a.error_flag, 37); ok = false; break; }
+            tc_fence_after();
+            const float inv2 = row_factor[r];
+            float d[HD], ss = 0.0f;
+#pragma unroll
+            for (int cc = 0; cc < HD / 32; ++cc) {
+              float o2[32];
+              tc_ld32_issue(tm_o[0] + lane_off + cc * 32, d + cc * 32);
+              tc_ld32_issue(tm_o[1] + lane_off + cc * 32, o2);
+              tc_wait_ld();
+#pragma unroll
+              for (int i = 0; i < 32; ++i) {
+                const float v = d[cc * 32 + i] * inv - o2[i] * inv2;
+                d[cc * 32 + i] = v;
+                if (cc * 32 + i < a.diff_dv) ss = fmaf(v, v, ss);
+              }
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) {
+              mbar_arrive_cta(bar(19));
+              mbar_arrive_cta(bar(20));
+            }
+            if (valid) {
+              const float k = a.diff_factor / sqrtf(ss / (float)a.diff_dv + a.diff_eps);
+              bf16* dst = a.out + (size_t)(it.row0 + qi) * a.ldo + (size_t)(it.h0 >> 1) * a.diff_dv;
+              const bool wide = ((a.diff_dv | a.ldo) & 7) == 0;      // 16-byte stores
+#pragma unroll
+              for (int i = 0; i < HD; i += 8) {
+                if (wide && i + 8 <= a.diff_dv) {
+                  unsigned w[4];
+#pragma unroll
+                  for (int u = 0; u < 4; ++u) {
+                    __nv_bfloat162 v = __floats2bfloat162_rn(d[i + 2 * u] * k, d[i + 2 * u + 1] * k);
+                    w[u] = *reinterpret_cast<unsigned*>(&v);
+                  }
+                  *reinterpret_cast<uint4*>(dst + i) = make_uint4(w[0], w[1], w[2], w[3]);
+                } else {
+#pragma unroll
+                  for (int u = 0; u < 8; ++u)
+                    if (i + u < a.diff_dv) dst[i + u] = __float2bfloat16_rn(d[i + u] * k);
+                }
+              }
+            }
+          }
+          ++items_t;
+          c_t += n_tiles;
+          continue;
+        }
         if (a.out_gate != nullptr && valid) inv *= 1.0f / (1.0f + expf(-a.out_gate[(size_t)(it.row0 + qi) * a.ldg + it.h0 + t]));
         bf16* dst = a.out + (size_t)(it.row0 + qi) * a.ldo + (size_t)(it.h0 + t) * HD;
-        float* dst_f = reinterpret_cast<float*>(a.out) + (size_t)(it.row0 + qi) * a.ldo + (size_t)(it.h0 + t) * HD;
 #pragma unroll
         for (int cc = 0; cc < HD / 32; ++cc) {
           float o[32];
@@ -469,11 +533,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             __syncwarp();
             if (lane == 0) mbar_arrive_cta(bar(19 + t));
           }
-          if (valid && a.out_f32) {
-#pragma unroll
-            for (int i = 0; i < 32; i += 4)
-              *reinterpret_cast<float4*>(dst_f + cc * 32 + i) = make_float4(o[i] * inv, o[i + 1] * inv, o[i + 2] * inv, o[i + 3] * inv);
-          } else if (valid) {
+          if (valid) {
 #pragma unroll
             for (int i = 0; i < 32; i += 8) {
               unsigned w[4];
@@ -503,7 +563,8 @@ extern "C" int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens
                                             const void* vcache, int n_pages, const int* seq_start, const int* seq_pos0,
                                             const int* seq_pages, int pages_stride, int n_seqs, int max_q_len, int nh,
                                             int nkv, int hd, int page_size, float scale, int window, float softcap,
-                                            const float* sink, const float* gate_bias, const float* out_gate, int ldg, int out_f32,
+                                            const float* sink, const float* gate_bias, const float* out_gate, int ldg, float diff_lambda,
+                                            float diff_factor, float diff_eps, int diff_dv,
                                             int* error_flag, int* work_counter, void* stream) {
   HB_REQUIRE(n_seqs > 0 && max_q_len > 0 && nh > 0 && nkv > 0 && n_tokens > 0 && n_pages > 0, "attention_prefill_tc: sizes must be positive");
   HB_REQUIRE(hd == 64 || hd == 128, "attention_prefill_tc: head size %d is not 64 or 128", hd);
@@ -517,6 +578,8 @@ extern "C" int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens
   HB_REQUIRE(scale > 0.0f, "attention_prefill_tc: the score scale must be positive");
   HB_REQUIRE(softcap >= 0.0f, "attention_prefill_tc: the cap on the scores must be >= 0 (0: none)");
   HB_REQUIRE(gate_bias == nullptr || (sink == nullptr && softcap == 0.0f), "attention_prefill_tc: sigmoid weights have no sink and no cap");
+  HB_REQUIRE(diff_dv == 0 || (diff_dv > 0 && diff_dv <= hd && (nh / nkv) % 2 == 0 && sink == nullptr && gate_bias == nullptr && out_gate == nullptr),
+             "attention_prefill_tc: the difference of two maps takes pairs of query heads of one key/value head, no sink, no gate, no sigmoid weights");
   CUtensorMap mq, mk, mv;
   int rc = make_map_cols(&mq, q, n_tokens, nh * hd, ldq, PT_Q);
   if (rc) return rc;
@@ -527,7 +590,8 @@ extern "C" int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens
   if (rc) return rc;
   const int q_tiles = ceil_div(max_q_len, PT_Q);
   PrefillTcArgs a{(bf16*)out, ldo, seq_start, seq_pos0, seq_pages, pages_stride, nh, nkv, page_size,
-                  scale * 1.4426950408889634f, window, error_flag, n_seqs, q_tiles, work_counter, softcap, sink, gate_bias, out_gate, ldg, out_f32};
+                  scale * 1.4426950408889634f, window, error_flag, n_seqs, q_tiles, work_counter, softcap, sink, gate_bias, out_gate, ldg,
+                  diff_lambda, diff_factor, diff_eps, diff_dv};
   cudaStream_t s = (cudaStream_t)stream;
   const int pairs = (nh / nkv + 1) / 2;
   const long long items = (long long)q_tiles * n_seqs * nkv * pairs;
@@ -540,8 +604,8 @@ extern "C" int hb_attention_prefill_tc_bf16(const void* q, int ldq, int n_tokens
   }
   dim3 grid((unsigned)(items < sms ? items : sms));
   cudaError_t e;
-  // two Q tiles, two stages of K and of V; slack for the 1024-byte alignment; barriers and the item ring
-  const int smem = 6 * (hd / 64) * PT_SUB + 1024 + 512;
+  // two Q tiles, two stages of K and of V; slack for the 1024-byte alignment; barriers, the item ring, a float per row
+  const int smem = 6 * (hd / 64) * PT_SUB + 1024 + 1024;
   if (hd == 128) {
     e = cudaFuncSetAttribute(attention_prefill_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) HB_FAIL(3, "attention_prefill_tc: cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(e));

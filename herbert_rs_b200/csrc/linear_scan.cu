@@ -566,6 +566,75 @@ gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restri
     const float gv = g[i], sg = 1.0f / (1.0f + expf(-gv));
     return act == 0 ? gv * sg : sg;
   };
+  w += (size_t)u * w_stride;
+  // bfloat16 results: the fast exponential and division (errors far below the rounding that follows)
+  auto fast_gate = [&](float gv) {
+    const float sg = sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(-gv)) : 1.0f / (1.0f + expf(-gv));
+    return act == 0 ? gv * sg : sg;
+  };
+  if (n % 4 == 0 && n <= 8 * (int)blockDim.x && ((ldo | ldg | ldy) & 3) == 0 &&
+      (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)y | (uintptr_t)w) & 15) == 0) {      // the same, four columns at once
+    float4 v[2], ga[2];
+    float s = 0.0f;
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int i = (threadIdx.x + q * blockDim.x) * 4;
+      if (i >= n) continue;
+      v[q] = *reinterpret_cast<const float4*>(orow + i);
+      ga[q] = *reinterpret_cast<const float4*>(g + i);
+    }
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      if ((int)(threadIdx.x + q * blockDim.x) * 4 >= n) continue;
+      ga[q] = make_float4(fast_gate(ga[q].x), fast_gate(ga[q].y), fast_gate(ga[q].z), fast_gate(ga[q].w));
+      if (gate_first) {
+        v[q] = make_float4(v[q].x * ga[q].x, v[q].y * ga[q].y, v[q].z * ga[q].z, v[q].w * ga[q].w);
+        ga[q] = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+      }
+      s += (v[q].x * v[q].x + v[q].y * v[q].y) + (v[q].z * v[q].z + v[q].w * v[q].w);
+    }
+    const float k = 1.0f / sqrtf(block_sum(s, red) / (float)n + eps);
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int i = (threadIdx.x + q * blockDim.x) * 4;
+      if (i >= n) continue;
+      const float4 w4 = *reinterpret_cast<const float4*>(w + i);
+      T* p = y + (size_t)t * ldy + (size_t)u * n + i;
+      const float r0 = ((v[q].x * k) * w4.x) * ga[q].x, r1 = ((v[q].y * k) * w4.y) * ga[q].y;
+      const float r2 = ((v[q].z * k) * w4.z) * ga[q].z, r3 = ((v[q].w * k) * w4.w) * ga[q].w;
+      if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(p) = make_float4(r0, r1, r2, r3);
+      } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(r0, r1), hi = __floats2bfloat162_rn(r2, r3);
+        uint2 pk;
+        pk.x = *reinterpret_cast<const unsigned*>(&lo);
+        pk.y = *reinterpret_cast<const unsigned*>(&hi);
+        *reinterpret_cast<uint2*>(p) = pk;
+      }
+    }
+    return;
+  }
+  if (n <= 8 * (int)blockDim.x) {            // a thread keeps its numbers (and their gates) between the sum and the result
+    float v[8], ga[8], s = 0.0f;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      const int i = threadIdx.x + q * blockDim.x;
+      v[q] = ga[q] = 0.0f;
+      if (i < n) { v[q] = orow[i]; ga[q] = gate_of(i); }
+    }
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      if (gate_first) { v[q] *= ga[q]; ga[q] = 1.0f; }
+      s = fmaf(v[q], v[q], s);
+    }
+    const float k = 1.0f / sqrtf(block_sum(s, red) / (float)n + eps);
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      const int i = threadIdx.x + q * blockDim.x;
+      if (i < n) y[(size_t)t * ldy + (size_t)u * n + i] = from_f32<T>(((v[q] * k) * w[i]) * ga[q]);
+    }
+    return;
+  }
   float ss = 0.0f;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
     const float v = gate_first ? orow[i] * gate_of(i) : orow[i];
@@ -574,7 +643,6 @@ gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restri
   ss = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(ss / (float)n + eps);
   T* yr = y + (size_t)t * ldy + (size_t)u * n;
-  w += (size_t)u * w_stride;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
     const float ga = gate_of(i);
     yr[i] = from_f32<T>(gate_first ? ((orow[i] * ga) * inv) * w[i] : ((orow[i] * inv) * w[i]) * ga);

@@ -60,9 +60,52 @@ __device__ __forceinline__ float turn_channel(const float* head, const float* bi
   return first ? own * c - other * s : own * c + other * s;
 }
 
-template <typename T>
+// The same for channels j .. j + 3 of a head at once: every size involved is a multiple of 4 (with halves, the half too).
+__device__ __forceinline__ float4 turn_channels4(const float* head, const float* bias, const float* w, float inv, int j, int rot,
+                                                 int halves, const float* cs) {
+  auto value = [&](int i) {
+    float4 x = *reinterpret_cast<const float4*>(head + i);
+    if (bias) {
+      const float4 b = *reinterpret_cast<const float4*>(bias + i);
+      x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w;
+    }
+    x.x *= inv; x.y *= inv; x.z *= inv; x.w *= inv;
+    if (w) {
+      const float4 k = *reinterpret_cast<const float4*>(w + i);
+      x.x *= k.x; x.y *= k.y; x.z *= k.z; x.w *= k.w;
+    }
+    return x;
+  };
+  const float4 own = value(j);
+  if (j >= rot) return own;
+  const int half = rot >> 1;
+  if (halves) {
+    const bool first = j < half;
+    const int m = first ? j : j - half;
+    const float4 other = value(first ? j + half : m);
+    const float4 c = *reinterpret_cast<const float4*>(cs + m);
+    float4 s = *reinterpret_cast<const float4*>(cs + half + m);
+    if (first) { s.x = -s.x; s.y = -s.y; s.z = -s.z; s.w = -s.w; }
+    return make_float4(own.x * c.x + other.x * s.x, own.y * c.y + other.y * s.y, own.z * c.z + other.z * s.z, own.w * c.w + other.w * s.w);
+  }
+  const int m = j >> 1;
+  const float2 c = *reinterpret_cast<const float2*>(cs + m), s = *reinterpret_cast<const float2*>(cs + half + m);
+  return make_float4(own.x * c.x - own.y * s.x, own.y * c.x + own.x * s.x, own.z * c.y - own.w * s.y, own.w * c.y + own.z * s.y);
+}
+template <typename T> __device__ __forceinline__ void rot_store4(T* p, float4 v);
+template <> __device__ __forceinline__ void rot_store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void rot_store4<bf16>(bf16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<const unsigned*>(&lo);
+  u.y = *reinterpret_cast<const unsigned*>(&hi);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
+// V4: four channels a lane (see turn_channels4).
+template <typename T, bool V4>
 __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
-  extern __shared__ float tab[];          // cos and sin of the token's angles: [rot] for q and k, [dv] for values
+  extern __shared__ __align__(16) float tab[];          // cos and sin of the token's angles: [rot] for q and k, [dv] for values
   __shared__ float red[32];
   pdl_wait();
   pdl_launch();
@@ -107,29 +150,76 @@ __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
     inv_k = 1.0f / sqrtf(sk / (float)kn + a.eps);
   }
   // map m of a head lies in channels m * dk ..: a query of map m is zero elsewhere, a key holds all maps side by side
-  T* qo = (T*)a.q_out + (size_t)t * a.ldq;
-  for (int i = threadIdx.x; i < a.nh * a.maps * a.hd; i += blockDim.x) {
-    const int h = i / a.hd, j = i - h * a.hd - (h % a.maps) * a.dk;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
+  for (int h = warp; h < a.nh * a.maps; h += nwarp) {      // a warp per head: nothing is divided channel by channel
     const size_t at = (size_t)h * a.dk;
-    float r = 0.0f;
-    if (j >= 0 && j < a.dk) r = turn_channel(q + at, bq ? bq + at : nullptr, a.wq ? a.wq + at : nullptr, inv_q, j, a.rot, a.halves, tab);
-    qo[i] = from_f32<T>(r);
+    const float* hb = bq ? bq + at : nullptr;
+    const float* hw = a.wq ? a.wq + at : nullptr;
+    const int off = (h % a.maps) * a.dk;
+    T* qo = (T*)a.q_out + (size_t)t * a.ldq + (size_t)h * a.hd;
+    if constexpr (V4) {
+      for (int i = lane * 4; i < a.hd; i += 128) {
+        const int j = i - off;
+        float4 r = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (j >= 0 && j < a.dk) r = turn_channels4(q + at, hb, hw, inv_q, j, a.rot, a.halves, tab);
+        rot_store4<T>(qo + i, r);
+      }
+      continue;
+    }
+#pragma unroll 4
+    for (int i = lane; i < a.hd; i += 32) {
+      const int j = i - off;
+      float r = 0.0f;
+      if (j >= 0 && j < a.dk) r = turn_channel(q + at, hb, hw, inv_q, j, a.rot, a.halves, tab);
+      qo[i] = from_f32<T>(r);
+    }
   }
   if (!a.write_cache) return;
   const int page = a.seq_pages[(size_t)a.tok_seq[t] * a.pages_stride + p / a.page_size];
   const size_t in_page = (size_t)(p % a.page_size);
-  for (int i = threadIdx.x; i < a.nkv * a.hd; i += blockDim.x) {
-    const int g = i / a.hd, j = i - g * a.hd;
-    const size_t at = (((size_t)page * a.nkv + g) * a.page_size + in_page) * a.hd + j;
-    float rk = 0.0f, rv = 0.0f;
-    if (j < a.maps * a.dk) {
-      const int m = j / a.dk;
-      const size_t head = (size_t)(g * a.maps + m) * a.dk;
-      rk = turn_channel(k + head, bk ? bk + head : nullptr, a.wk ? a.wk + head : nullptr, inv_k, j - m * a.dk, a.rot, a.halves, tab);
+  for (int u = warp; u < 2 * a.nkv; u += nwarp) {          // key heads and value heads
+    const int g = u >> 1;
+    const size_t at = (((size_t)page * a.nkv + g) * a.page_size + in_page) * a.hd;
+    if (u & 1) {
+      T* vo = (T*)a.vcache + at;
+      const float* hv = v + (size_t)g * a.dv;
+      const float* hb = bv ? bv + (size_t)g * a.dv : nullptr;
+      if constexpr (V4) {
+        for (int j = lane * 4; j < a.hd; j += 128) {
+          float4 r = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+          if (j < a.dv) r = turn_channels4(hv, hb, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, tab_v);
+          rot_store4<T>(vo + j, r);
+        }
+        continue;
+      }
+#pragma unroll 4
+      for (int j = lane; j < a.hd; j += 32) {
+        float r = 0.0f;
+        if (j < a.dv) r = turn_channel(hv, hb, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, tab_v);
+        vo[j] = from_f32<T>(r);
+      }
+      continue;
     }
-    if (j < a.dv) rv = turn_channel(v + (size_t)g * a.dv, bv ? bv + (size_t)g * a.dv : nullptr, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, tab_v);
-    ((T*)a.kcache)[at] = from_f32<T>(rk);
-    ((T*)a.vcache)[at] = from_f32<T>(rv);
+    T* ko = (T*)a.kcache + at;
+    int m = 0, first = 0;                                   // the map that channel j belongs to
+    if constexpr (V4) {
+      for (int j = lane * 4; j < a.hd; j += 128) {
+        while (m < a.maps && j - first >= a.dk) { ++m; first += a.dk; }
+        const size_t head = (size_t)(g * a.maps + m) * a.dk;
+        float4 r = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (m < a.maps)
+          r = turn_channels4(k + head, bk ? bk + head : nullptr, a.wk ? a.wk + head : nullptr, inv_k, j - first, a.rot, a.halves, tab);
+        rot_store4<T>(ko + j, r);
+      }
+      continue;
+    }
+    for (int j = lane; j < a.hd; j += 32) {
+      float r = 0.0f;
+      while (m < a.maps && j - first >= a.dk) { ++m; first += a.dk; }
+      const size_t head = (size_t)(g * a.maps + m) * a.dk;
+      if (m < a.maps) r = turn_channel(k + head, bk ? bk + head : nullptr, a.wk ? a.wk + head : nullptr, inv_k, j - first, a.rot, a.halves, tab);
+      ko[j] = from_f32<T>(r);
+    }
   }
 }
 
@@ -149,10 +239,18 @@ extern "C" int hb_qkv_rotary_cache(int dtype, const float* rows, int ld, const f
   HB_REQUIRE(smem <= 48 * 1024, "qkv_rotary_cache: %d rotated channels exceed a block's shared memory", rot);
   RotPrepArgs a{rows, ld, bias, wq, wk, eps, whole_norm, fqk, rot, halves, mscale, fv, tok_seq, tok_pos, seq_pages, pages_stride, q_out, ldq,
                 kcache, vcache, nh, nkv, maps, dk, dv, hd, page_size, write_cache};
-  if (dtype == HB_F32)
-    hb_launch(qkv_rotary_cache_kernel<float>, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, a);
-  else
-    hb_launch(qkv_rotary_cache_kernel<bf16>, dim3(n_tokens), dim3(256), smem, (cudaStream_t)stream, a);
+  const uintptr_t in_ptrs = (uintptr_t)rows | (uintptr_t)bias | (uintptr_t)wq | (uintptr_t)wk;
+  const uintptr_t out_ptrs = (uintptr_t)q_out | (uintptr_t)kcache | (uintptr_t)vcache;
+  const bool v4 = ((dk | dv | hd | ld | ldq) & 3) == 0 && (in_ptrs & 15) == 0 && (out_ptrs & 15) == 0 && rot % (halves ? 8 : 4) == 0 &&
+                  (fv == nullptr || dv % (halves ? 8 : 4) == 0);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == HB_F32) {
+    if (v4) hb_launch(qkv_rotary_cache_kernel<float, true>, dim3(n_tokens), dim3(256), smem, s, a);
+    else hb_launch(qkv_rotary_cache_kernel<float, false>, dim3(n_tokens), dim3(256), smem, s, a);
+  } else {
+    if (v4) hb_launch(qkv_rotary_cache_kernel<bf16, true>, dim3(n_tokens), dim3(256), smem, s, a);
+    else hb_launch(qkv_rotary_cache_kernel<bf16, false>, dim3(n_tokens), dim3(256), smem, s, a);
+  }
   HB_CHECK_LAUNCH("qkv_rotary_cache");
   return 0;
 }

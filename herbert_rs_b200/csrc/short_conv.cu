@@ -16,7 +16,9 @@
 #define SC_THREADS 128
 #define SC_TOKENS 64   // most tokens per CTA; a CTA takes at least taps - 1, so that only a sequence's first CTA reads its state
 
-template <typename TO>
+// TAPS > 0: that many taps, a channel's last inputs and weights in registers (each input is read once, four tokens ahead of
+// their sums); 0: any number of them.
+template <typename TO, int TAPS>
 __global__ void __launch_bounds__(SC_THREADS)
 short_conv_kernel(const float* __restrict__ in, int ld_in, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
                   const int* __restrict__ seq_slot, const int* __restrict__ seq_start, const int* __restrict__ seq_pos0,
@@ -34,6 +36,34 @@ short_conv_kernel(const float* __restrict__ in, int ld_in, const float* __restri
   float* st = state ? state + (size_t)seq_slot[b] * back * C + c : nullptr;
   const float* wr = w + (size_t)c * taps;
   const float b0 = bias ? bias[c] : 0.0f;
+  if constexpr (TAPS > 0) {
+    constexpr int BACK = TAPS - 1;
+    float wv[TAPS], win[BACK + 4];                 // win[0 .. BACK - 1]: the inputs before token i, then four of the step's
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wv[j] = wr[j];
+#pragma unroll
+    for (int j = 0; j < BACK; ++j) {
+      const int s = lo - BACK + j;
+      win[j] = s >= 0 ? in[(size_t)(t0 + s) * ld_in + c] : (pos0 + s >= 0 ? st[(size_t)(s + BACK) * C] : 0.0f);
+    }
+    const float* src = in + (size_t)t0 * ld_in + c;
+    TO* dst = out + (size_t)t0 * ldo + c;
+    for (int i = lo; i < hi; i += 4) {
+#pragma unroll
+      for (int q = 0; q < 4; ++q) win[BACK + q] = i + q < hi ? src[(size_t)(i + q) * ld_in] : 0.0f;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        float acc = b0;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) acc = fmaf(wv[j], win[q + j], acc);
+        if (add_input) acc += win[BACK + q];
+        if (act_silu) acc = acc / (1.0f + expf(-acc));
+        if (i + q < hi) dst[(size_t)(i + q) * ldo] = from_f32<TO>(acc);
+      }
+#pragma unroll
+      for (int j = 0; j < BACK; ++j) win[j] = win[j + 4];
+    }
+  } else
   for (int i = lo; i < hi; ++i) {
     float acc = b0;
     for (int j = 0; j < taps; ++j) {
@@ -74,12 +104,17 @@ extern "C" int hb_short_conv(int out_dtype, const float* in, int ld_in, const fl
          (long long)ceil_div(channels, SC_THREADS) * ceil_div(max_q_len, span) * n_seqs < 8LL * sms)
     span /= 2;
   dim3 grid(ceil_div(channels, SC_THREADS), ceil_div(max_q_len, span), n_seqs);
-  if (out_dtype == HB_F32)
-    hb_launch(short_conv_kernel<float>, grid, dim3(SC_THREADS), 0, (cudaStream_t)stream, in, ld_in, w, bias, state, seq_slot, seq_start,
-              seq_pos0, (float*)out, ldo, channels, taps, add_input, act_silu, span);
-  else
-    hb_launch(short_conv_kernel<bf16>, grid, dim3(SC_THREADS), 0, (cudaStream_t)stream, in, ld_in, w, bias, state, seq_slot, seq_start,
-              seq_pos0, (bf16*)out, ldo, channels, taps, add_input, act_silu, span);
+#define SC_GO(TO, TAPS)                                                                                                        \
+  hb_launch(short_conv_kernel<TO, TAPS>, grid, dim3(SC_THREADS), 0, (cudaStream_t)stream, in, ld_in, w, bias, state, seq_slot, seq_start, \
+            seq_pos0, (TO*)out, ldo, channels, taps, add_input, act_silu, span)
+#define SC_GO_TAPS(TO)                                                                                                         \
+  do {                                                                                                                         \
+    if (taps == 2) SC_GO(TO, 2); else if (taps == 3) SC_GO(TO, 3); else if (taps == 4) SC_GO(TO, 4);                            \
+    else if (taps == 5) SC_GO(TO, 5); else SC_GO(TO, 0);                                                                       \
+  } while (0)
+  if (out_dtype == HB_F32) SC_GO_TAPS(float); else SC_GO_TAPS(bf16);
+#undef SC_GO_TAPS
+#undef SC_GO
   HB_CHECK_LAUNCH("short_conv");
   return 0;
 }

@@ -190,15 +190,38 @@ extern "C" int hb_ssd_scan(int dtype, const void* xbc, int ld, int b_off, int c_
 
 // ---------------------------------------------------------------------------------------------
 // Chunked form.  Chunk c of sequence b has index seq_start[b] / 64 + b + c in the scratch arrays: sequences' ranges do
-// not meet, and floor(tokens / 64) + sequences bounds them all.
+// not meet, and floor(tokens / 64) + sequences bounds them all.  A CTA works on one chunk and up to SC_HEADS heads of one
+// group, one after another: B (and C, and the scores) are the group's, what belongs to the next head is fetched while
+// this one is computed.
 #define SC_Q 64
-#define SC_T 128
+#define SC_T 256
+#define SC_HEADS 4
 __device__ __forceinline__ int ssd_chunk_index(const SsdArgs& a, int b, int c) { return a.seq_start[b] / SC_Q + b + c; }
 
-// Warp 0: the chunk's step sizes and L_t (inclusive sums of log decays); tokens past the end get dt 0 and decay 1.
+struct SsdTile {      // what a CTA of the chunked kernels works on
+  int c, b, grp, h0, nh, v0, cols, tok0, n;
+};
+__device__ __forceinline__ bool ssd_tile(const SsdArgs& a, int vblocks, int hpc, int dvm, SsdTile& w) {
+  const int per = a.H / a.G, parts = (per + hpc - 1) / hpc;
+  int y = blockIdx.y;
+  w.c = blockIdx.x; w.b = blockIdx.z;
+  w.v0 = (y % vblocks) * dvm; y /= vblocks;
+  w.grp = y / parts;
+  const int part = y % parts;
+  w.h0 = w.grp * per + part * hpc;
+  w.nh = per - part * hpc < hpc ? per - part * hpc : hpc;
+  w.cols = a.dv - w.v0 < dvm ? a.dv - w.v0 : dvm;
+  const int t0 = a.seq_start[w.b], len = a.seq_start[w.b + 1] - t0;
+  w.tok0 = t0 + w.c * SC_Q;
+  w.n = len - w.c * SC_Q < SC_Q ? len - w.c * SC_Q : SC_Q;
+  return w.n > 0;
+}
+
+// One warp: a chunk's step sizes and L_t (inclusive sums of log decays, to the base 2); tokens past the end get dt 0 and
+// decay 1.
 __device__ __forceinline__ void ssd_prepare(const SsdArgs& a, int h, int tok0, int n, float* dts, float* cum) {
   const int lane = threadIdx.x & 31;
-  const float neg_a = -expf(a.a_log[h]), bias = a.dt_bias[h];
+  const float neg_a = -expf(a.a_log[h]) * 1.4426950408889634f, bias = a.dt_bias[h];
   float d0 = 0.0f, d1 = 0.0f;
   if (2 * lane < n) d0 = ssd_softplus(a.dt[(size_t)(tok0 + 2 * lane) * a.lddt + h] + bias);
   if (2 * lane + 1 < n) d1 = ssd_softplus(a.dt[(size_t)(tok0 + 2 * lane + 1) * a.lddt + h] + bias);
@@ -213,8 +236,8 @@ __device__ __forceinline__ void ssd_prepare(const SsdArgs& a, int h, int tok0, i
   cum[2 * lane] = run - l1; cum[2 * lane + 1] = run;
 }
 
-// rows [64][cols] of bfloat16 from the token rows at column `off` into shared memory [64][stride]; rows from n on and
-// columns from `cols` to `padded` become zero.  vec: 16-byte pieces (cols, off and the row length multiples of 8).
+// rows [64][cols] of bfloat16 from the token rows into shared memory [64][stride]; rows from n on and columns from
+// `cols` to `padded` become zero.  vec: 16-byte pieces (columns and the row length multiples of 8, rows on 16 bytes).
 __device__ __forceinline__ void ssd_load_rows(bf16* dst, int stride, const bf16* src, int ld, int n, int cols, int padded, bool vec) {
   const int per = padded >> 3;
   for (int i = threadIdx.x; i < SC_Q * per; i += SC_T) {
@@ -230,95 +253,140 @@ __device__ __forceinline__ void ssd_load_rows(bf16* dst, int stride, const bf16*
   }
 }
 
-__device__ __forceinline__ void ssd_split(float v, bf16& hi, bf16& lo) {
-  hi = __float2bfloat16_rn(v);
-  lo = __float2bfloat16_rn(v - __bfloat162float(hi));
+__device__ __forceinline__ float ssd_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void ssd_split2(float x, float y, unsigned& hi, unsigned& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  const float2 f = __bfloat1622float2(h);
+  hi = *reinterpret_cast<const unsigned*>(&h);
+  lo = pack_bf16(x - f.x, y - f.y);
 }
 
-// A chunk's own contribution to the state: sum_s e^{L_last - L_s} dt_s B_s x_s^T, and its total decay.
+// A chunk's own contribution to the state: sum_s e^{L_last - L_s} dt_s B_s x_s^T, and its total decay.  A warp takes
+// every eighth tile of 16 state rows.
 template <int DVM>
-__global__ void __launch_bounds__(SC_T) ssd_chunk_state_kernel(SsdArgs a, int vblocks, int vec) {
+__global__ void __launch_bounds__(SC_T) ssd_chunk_state_kernel(SsdArgs a, int vblocks, int vec, int hpc) {
   extern __shared__ __align__(16) unsigned char smem[];
-  __shared__ float dts[SC_Q], cum[SC_Q];
-  constexpr int XS = DVM + 8;
+  __shared__ __align__(16) float dts[SC_HEADS][SC_Q], cum[SC_HEADS][SC_Q];
+  constexpr int XS = DVM + 8, PER = DVM / 8, PIECES = (SC_Q * PER + SC_T - 1) / SC_T;
   const int NP = (a.N + 15) & ~15, BS = NP + 8;
   bf16* Bs = reinterpret_cast<bf16*>(smem);          // [64][BS]
-  bf16* Xh = Bs + SC_Q * BS;                         // [64][XS]
-  bf16* Xl = Xh + SC_Q * XS;
+  bf16* Xh = Bs + SC_Q * BS;                         // [2][64][XS] weighted x, high parts
+  bf16* Xl = Xh + 2 * SC_Q * XS;                     // low parts
   pdl_wait();
   pdl_launch();
-  const int c = blockIdx.x, b = blockIdx.z, h = blockIdx.y / vblocks, v0 = (blockIdx.y % vblocks) * DVM;
-  const int t0 = a.seq_start[b], len = a.seq_start[b + 1] - t0;
-  if (c * SC_Q >= len) return;
-  const int tok0 = t0 + c * SC_Q, n = len - c * SC_Q < SC_Q ? len - c * SC_Q : SC_Q;
+  SsdTile w;
+  if (!ssd_tile(a, vblocks, hpc, DVM, w)) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int grp = h / (a.H / a.G), cols = a.dv - v0 < DVM ? a.dv - v0 : DVM;
-  const bf16* rows = (const bf16*)a.xbc + (size_t)tok0 * a.ld;
-  ssd_load_rows(Bs, BS, rows + a.b_off + (size_t)grp * a.N, a.ld, n, a.N, NP, vec);
+  const bf16* rows = (const bf16*)a.xbc + (size_t)w.tok0 * a.ld;
+  ssd_load_rows(Bs, BS, rows + a.b_off + (size_t)w.grp * a.N, a.ld, w.n, a.N, NP, vec);
   cp_async_commit();
-  if (warp == 0) ssd_prepare(a, h, tok0, n, dts, cum);
-  __syncthreads();
-  const float last = cum[SC_Q - 1];
-  const bf16* xr = rows + (size_t)h * a.dv + v0;
-  for (int i = threadIdx.x; i < SC_Q * DVM; i += SC_T) {
-    const int r = i / DVM, cc = i - r * DVM;
-    const float x = (r < n && cc < cols) ? __bfloat162float(xr[(size_t)r * a.ld + cc]) : 0.0f;
-    ssd_split(x * (__expf(last - cum[r]) * dts[r]), Xh[r * XS + cc], Xl[r * XS + cc]);
-  }
-  cp_async_wait<0>();
-  __syncthreads();
-  const size_t ci = ssd_chunk_index(a, b, c);
-  float* out = a.chunk_state + ((ci * a.H + h) * a.N) * (size_t)a.dv + v0;
-  if (threadIdx.x == 0 && v0 == 0) a.chunk_decay[ci * a.H + h] = __expf(last);
-  const int mi = lane >> 3, l8 = lane & 7, g = lane >> 2, t = lane & 3;
-  const bool pair = a.dv % 2 == 0;
-  for (int mt = warp; mt < NP / 16; mt += SC_T / 32) {
-    float acc[DVM / 8][4];
+  uint4 raw[PIECES];                                 // the next head's x, eight channels of a token a piece
+  auto fetch = [&](int h) {
+    const bf16* xr = rows + (size_t)h * a.dv + w.v0;
 #pragma unroll
-    for (int i = 0; i < DVM / 8; ++i)
+    for (int q = 0; q < PIECES; ++q) {
+      const int i = threadIdx.x + q * SC_T, r = i / PER, c = (i % PER) * 8;
+      raw[q] = make_uint4(0, 0, 0, 0);
+      if (i >= SC_Q * PER || r >= w.n || c >= w.cols) continue;
+      if (vec) {
+        raw[q] = *reinterpret_cast<const uint4*>(xr + (size_t)r * a.ld + c);
+      } else {
+        bf16 v[8];
+        for (int j = 0; j < 8; ++j) v[j] = c + j < w.cols ? xr[(size_t)r * a.ld + c + j] : __float2bfloat16_rn(0.0f);
+        unsigned u[4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) acc[i][j] = 0.0f;
-#pragma unroll
-    for (int k = 0; k < SC_Q / 16; ++k) {
-      unsigned a0, a1, a2, a3;
-      ldmatrix_x4_trans(a0, a1, a2, a3, Bs + (k * 16 + (mi >> 1) * 8 + l8) * BS + mt * 16 + (mi & 1) * 8);
-#pragma unroll
-      for (int nd = 0; nd < DVM / 16; ++nd) {
-        if (nd * 16 >= cols) continue;
-        const int off = (k * 16 + (mi & 1) * 8 + l8) * XS + nd * 16 + (mi >> 1) * 8;
-        unsigned b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, Xh + off);
-        mma16816(acc[2 * nd], a0, a1, a2, a3, b0, b1);
-        mma16816(acc[2 * nd + 1], a0, a1, a2, a3, b2, b3);
-        ldmatrix_x4_trans(b0, b1, b2, b3, Xl + off);
-        mma16816(acc[2 * nd], a0, a1, a2, a3, b0, b1);
-        mma16816(acc[2 * nd + 1], a0, a1, a2, a3, b2, b3);
+        for (int j = 0; j < 4; ++j) {
+          const __nv_bfloat162 p = __halves2bfloat162(v[2 * j], v[2 * j + 1]);
+          u[j] = *reinterpret_cast<const unsigned*>(&p);
+        }
+        raw[q] = make_uint4(u[0], u[1], u[2], u[3]);
       }
     }
+  };
+  fetch(w.h0);
+  if (warp < w.nh) ssd_prepare(a, w.h0 + warp, w.tok0, w.n, dts[warp], cum[warp]);
+  cp_async_wait<0>();
+  __syncthreads();
+  const size_t ci = ssd_chunk_index(a, w.b, w.c);
+  const int mi = lane >> 3, l8 = lane & 7, g = lane >> 2, t = lane & 3;
+  const bool pair = a.dv % 2 == 0;
+  for (int ih = 0; ih < w.nh; ++ih) {
+    const int h = w.h0 + ih;
+    bf16* xh = Xh + (ih & 1) * SC_Q * XS;
+    bf16* xl = Xl + (ih & 1) * SC_Q * XS;
+    const float last = cum[ih][SC_Q - 1];
 #pragma unroll
-    for (int nd = 0; nd < DVM / 8; ++nd)
+    for (int q = 0; q < PIECES; ++q) {
+      const int i = threadIdx.x + q * SC_T, r = i / PER, c = (i % PER) * 8;
+      if (i >= SC_Q * PER) continue;
+      const float k = ssd_exp2(last - cum[ih][r]) * dts[ih][r];
+      const unsigned u[4] = {raw[q].x, raw[q].y, raw[q].z, raw[q].w};
+      unsigned hi[4], lo[4];
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int r = mt * 16 + g + half * 8, v = nd * 8 + 2 * t;
-        if (r >= a.N || v >= cols) continue;
-        float* p = out + (size_t)r * a.dv + v;
-        if (pair) *reinterpret_cast<float2*>(p) = make_float2(acc[nd][2 * half], acc[nd][2 * half + 1]);
-        else {
-          p[0] = acc[nd][2 * half];
-          if (v + 1 < cols) p[1] = acc[nd][2 * half + 1];
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u[j]));
+        ssd_split2(f.x * k, f.y * k, hi[j], lo[j]);
+      }
+      *reinterpret_cast<uint4*>(xh + r * XS + c) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(xl + r * XS + c) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    if (ih + 1 < w.nh) fetch(h + 1);
+    __syncthreads();      // also: the buffer written next was last read before the previous head's barrier
+    float* out = a.chunk_state + ((ci * a.H + h) * a.N) * (size_t)a.dv + w.v0;
+    if (threadIdx.x == 0 && w.v0 == 0) a.chunk_decay[ci * a.H + h] = ssd_exp2(last);
+    for (int mt = warp; mt < NP / 16; mt += SC_T / 32) {
+      float acc[DVM / 8][4];
+#pragma unroll
+      for (int i = 0; i < DVM / 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0.0f;
+#pragma unroll
+      for (int k = 0; k < SC_Q / 16; ++k) {
+        unsigned a0, a1, a2, a3;
+        ldmatrix_x4_trans(a0, a1, a2, a3, Bs + (k * 16 + (mi >> 1) * 8 + l8) * BS + mt * 16 + (mi & 1) * 8);
+#pragma unroll
+        for (int nd = 0; nd < DVM / 16; ++nd) {
+          if (nd * 16 >= w.cols) continue;
+          const int off = (k * 16 + (mi & 1) * 8 + l8) * XS + nd * 16 + (mi >> 1) * 8;
+          unsigned b0, b1, b2, b3;
+          ldmatrix_x4_trans(b0, b1, b2, b3, xh + off);
+          mma16816(acc[2 * nd], a0, a1, a2, a3, b0, b1);
+          mma16816(acc[2 * nd + 1], a0, a1, a2, a3, b2, b3);
+          ldmatrix_x4_trans(b0, b1, b2, b3, xl + off);
+          mma16816(acc[2 * nd], a0, a1, a2, a3, b0, b1);
+          mma16816(acc[2 * nd + 1], a0, a1, a2, a3, b2, b3);
         }
       }
+#pragma unroll
+      for (int nd = 0; nd < DVM / 8; ++nd)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int r = mt * 16 + g + half * 8, v = nd * 8 + 2 * t;
+          if (r >= a.N || v >= w.cols) continue;
+          float* p = out + (size_t)r * a.dv + v;
+          if (pair) *reinterpret_cast<float2*>(p) = make_float2(acc[nd][2 * half], acc[nd][2 * half + 1]);
+          else {
+            p[0] = acc[nd][2 * half];
+            if (v + 1 < w.cols) p[1] = acc[nd][2 * half + 1];
+          }
+        }
+    }
   }
 }
 
 // The states handed from chunk to chunk: what a chunk contributed is replaced by the state before it; the slot's state
-// becomes the one after the step.  V neighbouring entries of a head's state per thread.
+// becomes the one after the step.  V neighbouring entries of a head's state per thread.  V = 8: the state before a chunk
+// leaves as eight high and then eight low bfloat16 parts in the place of its eight floats, ready to be an operand.
 template <int V>
-__global__ void __launch_bounds__(256) ssd_state_pass_kernel(SsdArgs a) {
+__global__ void __launch_bounds__(128) ssd_state_pass_kernel(SsdArgs a) {
   pdl_wait();
   pdl_launch();
   const int b = blockIdx.z, h = blockIdx.y, per = a.N * a.dv;
-  const int e = (blockIdx.x * 256 + threadIdx.x) * V;
+  const int e = (blockIdx.x * 128 + threadIdx.x) * V;
   const int len = a.seq_start[b + 1] - a.seq_start[b], nc = (len + SC_Q - 1) / SC_Q;
   if (e >= per) return;
   float* S = a.state + ((size_t)a.seq_slot[b] * a.H + h) * per + e;
@@ -328,14 +396,19 @@ __global__ void __launch_bounds__(256) ssd_state_pass_kernel(SsdArgs a) {
   const size_t step = (size_t)a.H * per;
   float s[V];
   auto load = [&](float* v, const float* p) {
-    if constexpr (V == 4) {
-      const float4 f = *reinterpret_cast<const float4*>(p);
-      v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    if constexpr (V == 8) {
+      const float4 f = *reinterpret_cast<const float4*>(p), k = *reinterpret_cast<const float4*>(p + 4);
+      v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; v[4] = k.x; v[5] = k.y; v[6] = k.z; v[7] = k.w;
     } else v[0] = p[0];
   };
-  auto put = [&](float* p, const float* v) {
-    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-    else p[0] = v[0];
+  auto hand_on = [&](float* p, const float* v) {
+    if constexpr (V == 8) {
+      unsigned hi[4], lo[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ssd_split2(v[2 * j], v[2 * j + 1], hi[j], lo[j]);
+      reinterpret_cast<uint4*>(p)[0] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      reinterpret_cast<uint4*>(p)[1] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    } else p[0] = v[0];
   };
   load(s, S);
   for (int c = 0; c < nc; c += 4) {      // the loads of four chunks go ahead of their stores
@@ -346,151 +419,182 @@ __global__ void __launch_bounds__(256) ssd_state_pass_kernel(SsdArgs a) {
 #pragma unroll
     for (int q = 0; q < 4; ++q)
       if (c + q < nc) {
-        put(cs + (size_t)(c + q) * step, s);
+        hand_on(cs + (size_t)(c + q) * step, s);
 #pragma unroll
         for (int j = 0; j < V; ++j) s[j] = fmaf(d[q], s[j], x[q][j]);
       }
   }
-  put(S, s);
+  if constexpr (V == 8) {
+    reinterpret_cast<float4*>(S)[0] = make_float4(s[0], s[1], s[2], s[3]);
+    reinterpret_cast<float4*>(S)[1] = make_float4(s[4], s[5], s[6], s[7]);
+  } else S[0] = s[0];
 }
 
-// The outputs of a chunk.  A warp owns 16 tokens.
+// The outputs of a chunk.  Warp w owns tokens 16 (w mod 4) .. and one half of the value channels.
 template <int DVM>
-__global__ void __launch_bounds__(SC_T) ssd_chunk_out_kernel(SsdArgs a, int vblocks, int vec) {
+__global__ void __launch_bounds__(SC_T) ssd_chunk_out_kernel(SsdArgs a, int vblocks, int vec, int hpc, int stages) {
   extern __shared__ __align__(16) unsigned char smem[];
-  __shared__ float dts[SC_Q], cum[SC_Q];
-  constexpr int XS = DVM + 8;
+  __shared__ __align__(16) float dts[SC_HEADS][SC_Q], cum[SC_HEADS][SC_Q];
+  constexpr int XS = DVM + 8, HALF = DVM / 2;
   const int NP = (a.N + 15) & ~15, BS = NP + 8;
   bf16* Cs = reinterpret_cast<bf16*>(smem);          // [64][BS]
   bf16* Bs = Cs + SC_Q * BS;                         // [64][BS]
-  bf16* Xs = Bs + SC_Q * BS;                         // [64][XS]
-  bf16* Sh = Xs + SC_Q * XS;                         // [NP][XS]
-  bf16* Sl = Sh + NP * XS;
+  bf16* ring = Bs + SC_Q * BS;                       // per stage: x [64][XS], the state's high and low parts [NP][XS] each
+  const int stage_len = (SC_Q + 2 * NP) * XS;
   pdl_wait();
   pdl_launch();
-  const int c = blockIdx.x, b = blockIdx.z, h = blockIdx.y / vblocks, v0 = (blockIdx.y % vblocks) * DVM;
-  const int t0 = a.seq_start[b], len = a.seq_start[b + 1] - t0;
-  if (c * SC_Q >= len) return;
-  const int tok0 = t0 + c * SC_Q, n = len - c * SC_Q < SC_Q ? len - c * SC_Q : SC_Q;
+  SsdTile w;
+  if (!ssd_tile(a, vblocks, hpc, DVM, w)) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int grp = h / (a.H / a.G), cols = a.dv - v0 < DVM ? a.dv - v0 : DVM;
-  const bf16* rows = (const bf16*)a.xbc + (size_t)tok0 * a.ld;
-  ssd_load_rows(Cs, BS, rows + a.c_off + (size_t)grp * a.N, a.ld, n, a.N, NP, vec);
-  ssd_load_rows(Bs, BS, rows + a.b_off + (size_t)grp * a.N, a.ld, n, a.N, NP, vec);
-  ssd_load_rows(Xs, XS, rows + (size_t)h * a.dv + v0, a.ld, n, cols, DVM, vec);
-  cp_async_commit();
-  const float* S0 = a.chunk_state + (((size_t)ssd_chunk_index(a, b, c) * a.H + h) * a.N) * (size_t)a.dv + v0;
-  if (a.dv % 4 == 0) {
-    for (int i = threadIdx.x; i < NP * (DVM / 4); i += SC_T) {
-      const int r = i / (DVM / 4), v = (i - r * (DVM / 4)) * 4;
-      float4 f = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-      if (r < a.N && v < cols) f = *reinterpret_cast<const float4*>(S0 + (size_t)r * a.dv + v);
-      __nv_bfloat162 h0 = __floats2bfloat162_rn(f.x, f.y), h1 = __floats2bfloat162_rn(f.z, f.w);
-      const float2 g0 = __bfloat1622float2(h0), g1 = __bfloat1622float2(h1);
-      __nv_bfloat162 l0 = __floats2bfloat162_rn(f.x - g0.x, f.y - g0.y), l1 = __floats2bfloat162_rn(f.z - g1.x, f.w - g1.y);
-      *reinterpret_cast<__nv_bfloat162*>(Sh + r * XS + v) = h0; *reinterpret_cast<__nv_bfloat162*>(Sh + r * XS + v + 2) = h1;
-      *reinterpret_cast<__nv_bfloat162*>(Sl + r * XS + v) = l0; *reinterpret_cast<__nv_bfloat162*>(Sl + r * XS + v + 2) = l1;
+  const bf16* rows = (const bf16*)a.xbc + (size_t)w.tok0 * a.ld;
+  const size_t ci = ssd_chunk_index(a, w.b, w.c);
+  const bool packed = a.dv % 8 == 0;                 // the states lie as high and low parts already
+  auto stage = [&](int ih) {
+    bf16* Xs = ring + (ih % stages) * stage_len;
+    bf16* Sh = Xs + SC_Q * XS;
+    bf16* Sl = Sh + NP * XS;
+    const int h = w.h0 + ih;
+    ssd_load_rows(Xs, XS, rows + (size_t)h * a.dv + w.v0, a.ld, w.n, w.cols, DVM, vec);
+    const float* S0 = a.chunk_state + ((ci * a.H + h) * a.N) * (size_t)a.dv + w.v0;
+    constexpr int PER = DVM / 8;
+    for (int i = threadIdx.x; i < NP * PER; i += SC_T) {
+      const int r = i / PER, v = (i % PER) * 8;
+      bf16* dh = Sh + r * XS + v;
+      bf16* dl = Sl + r * XS + v;
+      const float* src = S0 + (size_t)r * a.dv + v;
+      if (r >= a.N || v >= w.cols) {
+        *reinterpret_cast<uint4*>(dh) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(dl) = make_uint4(0, 0, 0, 0);
+      } else if (packed) {
+        cp_async16(dh, src);
+        cp_async16(dl, src + 4);
+      } else {
+        for (int j = 0; j < 8; j += 2) {
+          const float f0 = v + j < w.cols ? src[j] : 0.0f, f1 = v + j + 1 < w.cols ? src[j + 1] : 0.0f;
+          unsigned hi, lo;
+          ssd_split2(f0, f1, hi, lo);
+          *reinterpret_cast<unsigned*>(dh + j) = hi;
+          *reinterpret_cast<unsigned*>(dl + j) = lo;
+        }
+      }
     }
-  } else {
-    for (int i = threadIdx.x; i < NP * DVM; i += SC_T) {
-      const int r = i / DVM, v = i - r * DVM;
-      const float f = (r < a.N && v < cols) ? S0[(size_t)r * a.dv + v] : 0.0f;
-      ssd_split(f, Sh[r * XS + v], Sl[r * XS + v]);
-    }
-  }
-  if (warp == 0) ssd_prepare(a, h, tok0, n, dts, cum);
-  cp_async_wait<0>();
-  __syncthreads();
-  if (warp * 16 >= n) return;                        // nothing of this chunk is left for these 16 tokens
+    cp_async_commit();
+  };
+  ssd_load_rows(Cs, BS, rows + a.c_off + (size_t)w.grp * a.N, a.ld, w.n, a.N, NP, vec);
+  ssd_load_rows(Bs, BS, rows + a.b_off + (size_t)w.grp * a.N, a.ld, w.n, a.N, NP, vec);
+  stage(0);
+  if (warp < w.nh) ssd_prepare(a, w.h0 + warp, w.tok0, w.n, dts[warp], cum[warp]);
+  const int rb = warp & 3, cb = (warp >> 2) * HALF;
   const int mi = lane >> 3, l8 = lane & 7, g = lane >> 2, t = lane & 3;
-  float acc[DVM / 8][4], sc[8][4];
-#pragma unroll
-  for (int i = 0; i < DVM / 8; ++i)
-#pragma unroll
-    for (int j = 0; j < 4; ++j) acc[i][j] = 0.0f;
-#pragma unroll
-  for (int i = 0; i < 8; ++i)
-#pragma unroll
-    for (int j = 0; j < 4; ++j) sc[i][j] = 0.0f;
-  // C S0 and C B^T over the state rows
-  for (int ks = 0; ks < NP / 16; ++ks) {
-    unsigned a0, a1, a2, a3;
-    ldmatrix_x4(a0, a1, a2, a3, Cs + (warp * 16 + (lane & 15)) * BS + ks * 16 + (lane >> 4) * 8);
-#pragma unroll
-    for (int np = 0; np < 4; ++np) {
-      if (np > warp) continue;                       // keys after the warp's tokens
-      unsigned b0, b1, b2, b3;
-      ldmatrix_x4(b0, b1, b2, b3, Bs + (np * 16 + l8 + ((lane >> 4) << 3)) * BS + ks * 16 + ((lane >> 3) & 1) * 8);
-      mma16816(sc[2 * np], a0, a1, a2, a3, b0, b1);
-      mma16816(sc[2 * np + 1], a0, a1, a2, a3, b2, b3);
-    }
-#pragma unroll
-    for (int nd = 0; nd < DVM / 16; ++nd) {
-      if (nd * 16 >= cols) continue;
-      const int off = (ks * 16 + (mi & 1) * 8 + l8) * XS + nd * 16 + (mi >> 1) * 8;
-      unsigned b0, b1, b2, b3;
-      ldmatrix_x4_trans(b0, b1, b2, b3, Sh + off);
-      mma16816(acc[2 * nd], a0, a1, a2, a3, b0, b1);
-      mma16816(acc[2 * nd + 1], a0, a1, a2, a3, b2, b3);
-      ldmatrix_x4_trans(b0, b1, b2, b3, Sl + off);
-      mma16816(acc[2 * nd], a0, a1, a2, a3, b0, b1);
-      mma16816(acc[2 * nd + 1], a0, a1, a2, a3, b2, b3);
-    }
-  }
-  const int tr0 = warp * 16 + g, tr1 = tr0 + 8;
-  const float L0 = cum[tr0], L1 = cum[tr1], e0 = __expf(L0), e1 = __expf(L1);
-#pragma unroll
-  for (int nd = 0; nd < DVM / 8; ++nd) {
-    acc[nd][0] *= e0; acc[nd][1] *= e0; acc[nd][2] *= e1; acc[nd][3] *= e1;
-  }
-  // the scores, weighted and masked, times x
-#pragma unroll
-  for (int kc = 0; kc < 4; ++kc) {
-    if (kc > warp) continue;
-    unsigned hi[4], lo[4];
-#pragma unroll
-    for (int q = 0; q < 4; ++q) {                    // (key tile, token half): a0 (0, 0), a1 (0, 1), a2 (1, 0), a3 (1, 1)
-      const int nt = 2 * kc + (q >> 1), half = q & 1, tr = half ? tr1 : tr0;
-      const float L = half ? L1 : L0;
-      float w[2];
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int s = nt * 8 + 2 * t + j;
-        w[j] = s <= tr ? sc[nt][2 * half + j] * (__expf(L - cum[s]) * dts[s]) : 0.0f;
-      }
-      const __nv_bfloat162 h2 = __floats2bfloat162_rn(w[0], w[1]);
-      const float2 back = __bfloat1622float2(h2);
-      hi[q] = *reinterpret_cast<const unsigned*>(&h2);
-      lo[q] = pack_bf16(w[0] - back.x, w[1] - back.y);
-    }
-#pragma unroll
-    for (int nd = 0; nd < DVM / 16; ++nd) {
-      if (nd * 16 >= cols) continue;
-      unsigned b0, b1, b2, b3;
-      ldmatrix_x4_trans(b0, b1, b2, b3, Xs + (kc * 16 + (mi & 1) * 8 + l8) * XS + nd * 16 + (mi >> 1) * 8);
-      mma16816(acc[2 * nd], hi[0], hi[1], hi[2], hi[3], b0, b1);
-      mma16816(acc[2 * nd + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
-      mma16816(acc[2 * nd], lo[0], lo[1], lo[2], lo[3], b0, b1);
-      mma16816(acc[2 * nd + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
-    }
-  }
-  const float dskip = a.dskip[h];
+  const int tr0 = rb * 16 + g, tr1 = tr0 + 8;
+  const bool live = rb * 16 < w.n && cb < w.cols;    // a warp without tokens or channels keeps the barriers company
   const bool pair = a.dv % 2 == 0 && a.ldo % 2 == 0;
-#pragma unroll
-  for (int nd = 0; nd < DVM / 8; ++nd)
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int tr = half ? tr1 : tr0, v = nd * 8 + 2 * t;
-      if (tr >= n || v >= cols) continue;
-      const float y0 = fmaf(dskip, __bfloat162float(Xs[tr * XS + v]), acc[nd][2 * half]);
-      const float y1 = fmaf(dskip, __bfloat162float(Xs[tr * XS + v + 1]), acc[nd][2 * half + 1]);
-      float* p = a.out + (size_t)(tok0 + tr) * a.ldo + (size_t)h * a.dv + v0 + v;
-      if (pair) *reinterpret_cast<float2*>(p) = make_float2(y0, y1);
-      else {
-        p[0] = y0;
-        if (v + 1 < cols) p[1] = y1;
-      }
+  float sc[8][4];                                    // C B^T of the warp's tokens: the group's, kept for all heads
+  for (int ih = 0; ih < w.nh; ++ih) {
+    if (stages > 1 && ih + 1 < w.nh) {
+      stage(ih + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
     }
+    __syncthreads();
+    if (live) {
+      if (ih == 0) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) sc[i][j] = 0.0f;
+        for (int ks = 0; ks < NP / 16; ++ks) {
+          unsigned a0, a1, a2, a3;
+          ldmatrix_x4(a0, a1, a2, a3, Cs + (rb * 16 + (lane & 15)) * BS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+          for (int np = 0; np < 4; ++np) {
+            if (np > rb) continue;                   // keys after the warp's tokens
+            unsigned b0, b1, b2, b3;
+            ldmatrix_x4(b0, b1, b2, b3, Bs + (np * 16 + l8 + ((lane >> 4) << 3)) * BS + ks * 16 + ((lane >> 3) & 1) * 8);
+            mma16816(sc[2 * np], a0, a1, a2, a3, b0, b1);
+            mma16816(sc[2 * np + 1], a0, a1, a2, a3, b2, b3);
+          }
+        }
+      }
+      const int h = w.h0 + ih;
+      const bf16* Xs = ring + (ih % stages) * stage_len;
+      const bf16* Sh = Xs + SC_Q * XS;
+      const bf16* Sl = Sh + NP * XS;
+      float acc[HALF / 8][4];
+#pragma unroll
+      for (int i = 0; i < HALF / 8; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0.0f;
+#pragma unroll 2
+      for (int ks = 0; ks < NP / 16; ++ks) {         // C S0
+        unsigned a0, a1, a2, a3;
+        ldmatrix_x4(a0, a1, a2, a3, Cs + (rb * 16 + (lane & 15)) * BS + ks * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int nd = 0; nd < HALF / 16; ++nd) {
+          const int off = (ks * 16 + (mi & 1) * 8 + l8) * XS + cb + nd * 16 + (mi >> 1) * 8;
+          unsigned b0, b1, b2, b3;
+          ldmatrix_x4_trans(b0, b1, b2, b3, Sh + off);
+          mma16816(acc[2 * nd], a0, a1, a2, a3, b0, b1);
+          mma16816(acc[2 * nd + 1], a0, a1, a2, a3, b2, b3);
+          ldmatrix_x4_trans(b0, b1, b2, b3, Sl + off);
+          mma16816(acc[2 * nd], a0, a1, a2, a3, b0, b1);
+          mma16816(acc[2 * nd + 1], a0, a1, a2, a3, b2, b3);
+        }
+      }
+      const float L0 = cum[ih][tr0], L1 = cum[ih][tr1], e0 = ssd_exp2(L0), e1 = ssd_exp2(L1);
+#pragma unroll
+      for (int nd = 0; nd < HALF / 8; ++nd) {
+        acc[nd][0] *= e0; acc[nd][1] *= e0; acc[nd][2] *= e1; acc[nd][3] *= e1;
+      }
+      // the scores, weighted and masked, times x
+#pragma unroll
+      for (int kc = 0; kc < 4; ++kc) {
+        if (kc > rb) continue;
+        unsigned hi[4], lo[4];
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {                // key tile q: a0, a2 the first eight tokens, a1, a3 the others
+          const int nt = 2 * kc + q, s = nt * 8 + 2 * t;
+          const float2 Ls = *reinterpret_cast<const float2*>(&cum[ih][s]), ds = *reinterpret_cast<const float2*>(&dts[ih][s]);
+          float v0 = sc[nt][0] * (ssd_exp2(L0 - Ls.x) * ds.x), v1 = sc[nt][1] * (ssd_exp2(L0 - Ls.y) * ds.y);
+          float v2 = sc[nt][2] * (ssd_exp2(L1 - Ls.x) * ds.x), v3 = sc[nt][3] * (ssd_exp2(L1 - Ls.y) * ds.y);
+          if (kc == rb) {                            // the tile on the diagonal: nothing from later tokens
+            v0 = s <= tr0 ? v0 : 0.0f; v1 = s < tr0 ? v1 : 0.0f;
+            v2 = s <= tr1 ? v2 : 0.0f; v3 = s < tr1 ? v3 : 0.0f;
+          }
+          ssd_split2(v0, v1, hi[2 * q], lo[2 * q]);
+          ssd_split2(v2, v3, hi[2 * q + 1], lo[2 * q + 1]);
+        }
+#pragma unroll
+        for (int nd = 0; nd < HALF / 16; ++nd) {
+          unsigned b0, b1, b2, b3;
+          ldmatrix_x4_trans(b0, b1, b2, b3, Xs + (kc * 16 + (mi & 1) * 8 + l8) * XS + cb + nd * 16 + (mi >> 1) * 8);
+          mma16816(acc[2 * nd], hi[0], hi[1], hi[2], hi[3], b0, b1);
+          mma16816(acc[2 * nd + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
+          mma16816(acc[2 * nd], lo[0], lo[1], lo[2], lo[3], b0, b1);
+          mma16816(acc[2 * nd + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
+        }
+      }
+      const float dskip = a.dskip[h];
+#pragma unroll
+      for (int nd = 0; nd < HALF / 8; ++nd)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int tr = half ? tr1 : tr0, v = cb + nd * 8 + 2 * t;
+          if (tr >= w.n || v >= w.cols) continue;
+          const float y0 = fmaf(dskip, __bfloat162float(Xs[tr * XS + v]), acc[nd][2 * half]);
+          const float y1 = fmaf(dskip, __bfloat162float(Xs[tr * XS + v + 1]), acc[nd][2 * half + 1]);
+          float* p = a.out + (size_t)(w.tok0 + tr) * a.ldo + (size_t)h * a.dv + w.v0 + v;
+          if (pair) *reinterpret_cast<float2*>(p) = make_float2(y0, y1);
+          else {
+            p[0] = y0;
+            if (v + 1 < w.cols) p[1] = y1;
+          }
+        }
+    }
+    __syncthreads();                                 // this head's stage may be overwritten
+    if (stages == 1 && ih + 1 < w.nh) stage(ih + 1);
+  }
 }
 
 // Chunks that a step of n_tokens tokens in n_seqs sequences can have (rows of the scratch arrays); 0: these sizes go
@@ -514,30 +618,38 @@ extern "C" int hb_ssd_chunked_bf16(const void* xbc, int ld, int b_off, int c_off
                   0, chunk_state, chunk_decay};
   const int dvm = dv <= 32 ? 32 : dv <= 64 ? 64 : 128, vb = ceil_div(dv, dvm), chunks = ceil_div(max_q_len, SC_Q);
   const int vec = ld % 8 == 0 && b_off % 8 == 0 && c_off % 8 == 0 && N % 8 == 0 && dv % 8 == 0 && ((uintptr_t)xbc & 15) == 0;
-  HB_REQUIRE((long long)heads * vb <= 65535, "ssd_chunked: too many heads or value channels");
+  // heads of a group per CTA: as many as still leave every SM a CTA or two
+  const int per = heads / groups;
+  int hpc = per < SC_HEADS ? per : SC_HEADS;
+  while (hpc > 1 && (long long)chunks * n_seqs * groups * ceil_div(per, hpc) * vb < 2LL * ssd_sms()) --hpc;
+  const long long gy = (long long)groups * ceil_div(per, hpc) * vb;
+  HB_REQUIRE(gy <= 65535, "ssd_chunked: too many heads or value channels");
   const int NP = (N + 15) / 16 * 16;
-  const size_t row = (size_t)SC_Q * (NP + 8) * 2, xrow = (size_t)SC_Q * (dvm + 8) * 2;
-  const size_t sm1 = row + 2 * xrow, sm3 = 2 * row + xrow + 2 * (size_t)NP * (dvm + 8) * 2;
-  const dim3 grid(chunks, heads * vb, n_seqs);
+  const size_t row = (size_t)SC_Q * (NP + 8) * 2, xrow = (size_t)SC_Q * (dvm + 8) * 2, st = xrow + 2 * (size_t)NP * (dvm + 8) * 2;
+  const size_t sm1 = row + 4 * xrow;
+  // two CTAs an SM hide each other's loads; where only one fits, it fetches the next head's ahead
+  const int stages = hpc > 1 && 2 * row + st > 110 * 1024 && 2 * row + 2 * st <= 220 * 1024 ? 2 : 1;
+  const size_t sm3 = 2 * row + stages * st;
+  const dim3 grid(chunks, (unsigned)gy, n_seqs);
   cudaStream_t s = (cudaStream_t)stream;
-#define SC_GO(KERNEL, SM)                                                                                          \
+#define SC_GO(KERNEL, SM, ...)                                                                                     \
   do {                                                                                                             \
     cudaError_t e = cudaFuncSetAttribute(KERNEL, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(SM));          \
     if (e != cudaSuccess) HB_FAIL(3, "ssd_chunked: cannot reserve %d bytes of shared memory: %s", (int)(SM), cudaGetErrorString(e)); \
-    hb_launch(KERNEL, grid, dim3(SC_T), SM, s, a, vb, vec);                                                        \
+    hb_launch(KERNEL, grid, dim3(SC_T), SM, s, a, vb, vec, __VA_ARGS__);                                           \
   } while (0)
-  if (dvm == 32) SC_GO(ssd_chunk_state_kernel<32>, sm1);
-  else if (dvm == 64) SC_GO(ssd_chunk_state_kernel<64>, sm1);
-  else SC_GO(ssd_chunk_state_kernel<128>, sm1);
+  if (dvm == 32) SC_GO(ssd_chunk_state_kernel<32>, sm1, hpc);
+  else if (dvm == 64) SC_GO(ssd_chunk_state_kernel<64>, sm1, hpc);
+  else SC_GO(ssd_chunk_state_kernel<128>, sm1, hpc);
   HB_CHECK_LAUNCH("ssd_chunk_state");
-  if (N * dv % 4 == 0)
-    hb_launch(ssd_state_pass_kernel<4>, dim3(ceil_div(N * dv / 4, 256), heads, n_seqs), dim3(256), 0, s, a);
+  if (dv % 8 == 0)
+    hb_launch(ssd_state_pass_kernel<8>, dim3(ceil_div(N * dv / 8, 128), heads, n_seqs), dim3(128), 0, s, a);
   else
-    hb_launch(ssd_state_pass_kernel<1>, dim3(ceil_div(N * dv, 256), heads, n_seqs), dim3(256), 0, s, a);
+    hb_launch(ssd_state_pass_kernel<1>, dim3(ceil_div(N * dv, 128), heads, n_seqs), dim3(128), 0, s, a);
   HB_CHECK_LAUNCH("ssd_state_pass");
-  if (dvm == 32) SC_GO(ssd_chunk_out_kernel<32>, sm3);
-  else if (dvm == 64) SC_GO(ssd_chunk_out_kernel<64>, sm3);
-  else SC_GO(ssd_chunk_out_kernel<128>, sm3);
+  if (dvm == 32) SC_GO(ssd_chunk_out_kernel<32>, sm3, hpc, stages);
+  else if (dvm == 64) SC_GO(ssd_chunk_out_kernel<64>, sm3, hpc, stages);
+  else SC_GO(ssd_chunk_out_kernel<128>, sm3, hpc, stages);
 #undef SC_GO
   HB_CHECK_LAUNCH("ssd_chunk_out");
   return 0;

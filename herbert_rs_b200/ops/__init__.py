@@ -68,7 +68,7 @@ _SIGS = {
                                   c_void_p, c_int, c_int, c_void_p],
     "hb_attention_prefill_tc_bf16": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                      c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p,
-                                     c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
+                                     c_void_p, c_void_p, c_int, c_float, c_float, c_float, c_int, c_void_p, c_void_p, c_void_p],
     "hb_argmax": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, ctypes.c_longlong, c_void_p],
     "hb_gemm_skinny_norm_parts": [c_int, c_int],
     "hb_sample": [c_void_p, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
@@ -1391,9 +1391,9 @@ def attention_prefill(q, ldq, out, k_cache, v_cache, seq_start, seq_pos0, seq_pa
 
 def attention_prefill_tc(q, ldq, out, k_cache, v_cache, seq_start, seq_pos0, seq_pages, n_seqs, max_q_len,
                          num_heads, num_kv_heads, head_dim, page_size, scale, window, softcap=None, sink=None,
-                         gate_bias=None, out_gate=None) -> None:
-    """The same on tcgen05 tensor cores (head sizes 64 and 128): S and O in tensor memory."""
-    _check(out, None, "out")
+                         gate_bias=None, out_gate=None, difference=None) -> None:
+    """The same on tcgen05 tensor cores (head sizes 64 and 128): S and O in tensor memory.  `difference` as in `attention`."""
+    _check(out, torch.bfloat16, "out")
     if sink is not None:
         _check(sink, torch.float32, "sink")
     if gate_bias is not None:
@@ -1402,7 +1402,7 @@ def attention_prefill_tc(q, ldq, out, k_cache, v_cache, seq_start, seq_pos0, seq
          k_cache.data_ptr(), v_cache.data_ptr(), k_cache.shape[0], seq_start.data_ptr(), seq_pos0.data_ptr(),
          seq_pages.data_ptr(), seq_pages.stride(0), int(n_seqs), int(max_q_len), num_heads, num_kv_heads, head_dim,
          page_size, float(scale), int(window or 0), float(softcap or 0.0), _ptr(sink), _ptr(gate_bias),
-         *_out_gate(out_gate, out.shape[0], num_heads), 1 if out.dtype == torch.float32 else 0, _error_flag(out.device).data_ptr(), _work_counter(out.device).data_ptr(),
+         *_out_gate(out_gate, out.shape[0], num_heads), *_difference(difference), _error_flag(out.device).data_ptr(), _work_counter(out.device).data_ptr(),
          _stream())
 
 
@@ -1419,7 +1419,7 @@ def _work_counter(device) -> torch.Tensor:
 
 
 def _prefill_tc_ok(q, ldq, out, head_dim, page_size) -> bool:
-    return (options.prefill_attention == "tcgen05" and q.dtype == torch.bfloat16 and head_dim in (64, 128) and page_size % 64 == 0
+    return (options.prefill_attention == "tcgen05" and q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and head_dim in (64, 128) and page_size % 64 == 0
             and ldq % 8 == 0 and out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0)
 
 
@@ -1445,9 +1445,11 @@ def attention(q, ldq, out, k_cache, v_cache, batch, num_heads, num_kv_heads, hea
 
     `difference` = (lambda, factor, eps, dv): query heads 2h and 2h + 1 are two attention maps over the same values; out
     [tokens, num_heads / 2 * dv] receives (a1 - lambda a2) / sqrt(mean(.^2) + eps) * factor of their first dv channels,
-    taken from the float results: where the key ranges of a decode step are combined, by a kernel of its own otherwise."""
-    if difference is not None and not (options.attention != "simt" and batch.is_decode
-                                       and _decode_kernel_ok(out, num_heads, num_kv_heads, head_dim, page_size)):
+    taken from the float results: where the key ranges of a decode step are combined, in the epilogue of the tcgen05 prompt
+    kernel, by a kernel of its own otherwise."""
+    if difference is not None and not (options.attention != "simt" and (
+            (batch.is_decode and scratch is not None and _decode_kernel_ok(out, num_heads, num_kv_heads, head_dim, page_size))
+            or (not batch.is_decode and _prefill_tc_ok(q, ldq, out, head_dim, page_size)))):
         lam, factor, eps, dv = difference
         maps = scratch((out.shape[0], num_heads * head_dim), torch.float32)
         _attention_rows(q, ldq, maps, k_cache, v_cache, batch, num_heads, num_kv_heads, head_dim, page_size, scale, window, seq_pages,
@@ -1474,7 +1476,7 @@ def _attention_rows(q, ldq, out, k_cache, v_cache, batch, num_heads, num_kv_head
     if _prefill_tc_ok(q, ldq, out, head_dim, page_size):
         attention_prefill_tc(q, ldq, out, k_cache, v_cache, batch.seq_start, batch.seq_pos0, seq_pages, batch.n_seqs,
                              batch.max_q_len, num_heads, num_kv_heads, head_dim, page_size, scale, window, softcap, sink, gate_bias,
-                             out_gate)
+                             out_gate, difference)
         return
     if _prefill_kernel_ok(q, head_dim, page_size):
         attention_prefill(q, ldq, out, k_cache, v_cache, batch.seq_start, batch.seq_pos0, seq_pages, batch.n_seqs,

@@ -168,7 +168,7 @@ def test_the_gate_before_the_norm_in_parts(dtype, parts, n):
     assert_close(to_np(out), P.gated_group_norm(y.double(), z.double()[:, :W], w.double(), parts, 1e-5).numpy(), dtype, "gate, norm")
 
 
-SSD_SIZES = [(4, 2, 24, 16), (6, 2, 48, 32), (2, 1, 128, 64), (8, 4, 16, 8), (3, 3, 7, 5), (2, 2, 130, 12), (1, 1, 256, 128), (2, 1, 40, 150), (4, 4, 5, 100)]
+SSD_SIZES = [(4, 2, 24, 16), (6, 3, 56, 24), (2, 1, 128, 64), (8, 4, 16, 8), (3, 3, 7, 5), (2, 2, 130, 12), (1, 1, 256, 128), (2, 1, 40, 150), (4, 4, 5, 100)]
 
 
 def _ssd_inputs(g, T, H, G, N, dv, dtype, extreme):
@@ -308,7 +308,7 @@ def test_latent_rows_rotated_in_either_layout(dtype, halves):
     assert_close(to_np(out.view(T, H, rank + rot)[:, :, rank:]), want.numpy(), "float32", "rotated parts of the queries")
 
 
-@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 32, 64), (2, 1, 8, 16), (8, 2, 64, 128), (2, 2, 24, 40), (6, 3, 48, 96), (2, 1, 64, 100), (4, 1, 20, 50), (4, 2, 120, 200)])
+@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 32, 64), (2, 1, 8, 16), (8, 2, 64, 128), (2, 2, 24, 40), (6, 3, 40, 80), (2, 1, 64, 100), (4, 1, 20, 50), (4, 2, 120, 200)])
 def test_difference_of_two_maps_in_every_attention_kernel(H, G, dk, dv):
     """One sequence of 300 cached keys in pages that are not in order; the queries of the last 150 positions as a prompt's
     portion and the last one alone.  Scaled queries make one far key, keys at page borders and the query's own key stand
