@@ -88,7 +88,7 @@ def mixed(tmp_path_factory):
               (U.mamba(heads=4, vdim=16, state=24, groups=2, norm_groups=2, conv=3), U.dense(ff=72)),
               (U.latent(heads=2, dim=16, rot_dim=8, vdim=24, kv_rank=32), None),
               (U.attention(heads=2, kv_heads=2, dim=8, vdim=16), U.dense())]
-    return U.make(tmp_path_factory.mktemp("putazen_mixed"), layers, seed=3, loop=(1, 3, 3))
+    return U.make(tmp_path_factory.mktemp("putazen_mixed"), layers, seed=13, loop=(1, 3, 3))
 
 
 # ---- each mechanism alone -------------------------------------------------------------------------

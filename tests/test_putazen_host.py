@@ -227,7 +227,7 @@ def test_order_of_layers():
 
 def test_leaving_out_a_mechanism_moves_the_logits(tmp_path):
     layers = [(U.attention(rot_dims=8), U.dense()), (U.mamba(), U.dense()), (U.latent(), None)]
-    d, pm = U.make(tmp_path / "m", layers, seed=5, loop=(1, 3, 2))
+    d, pm = U.make(tmp_path / "m", layers, seed=8, loop=(1, 3, 2))
     ids = np.random.default_rng(5).integers(0, 131, 40).tolist()
     ref = pm.logits(ids)
     low = float((pm.logits(ids, F64, P.bf16_storage) - ref).abs().max())
@@ -254,7 +254,7 @@ def test_leaving_out_a_mechanism_moves_the_logits(tmp_path):
     for name in ("l0.hc1.mix", "l1.hc2.mix"):
         assert moved(W=dict(pm.W, **{name: pm.W[name].T.contiguous()})) > 3 * low, name
     for name in ("l0.hc2.in", "l1.hc1.in", "l2.hc1.out"):
-        assert moved(W=dict(pm.W, **{name: pm.W[name].flip(0)})) > 3 * low, name
+        assert moved(W=dict(pm.W, **{name: pm.W[name].roll(1) * 1.5})) > 3 * low, name
     # the rows of B and C belong to groups of neighbouring heads, the maps of a head lie side by side
     m = pm.cfg["layers"][1]["mixer"]
     inner, gn = m["heads"] * m["vdim"], m["groups"] * m["state"]
