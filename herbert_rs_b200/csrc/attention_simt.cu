@@ -19,7 +19,7 @@
 #include "api.h"
 #include "common.cuh"
 
-#define ATT_MAX_HD 256
+#define ATT_MAX_HD 512      // heads of up to 256 channels take an instance with half the registers for a result
 #define ATT_WARPS 4
 
 struct AttnArgs {
@@ -44,9 +44,9 @@ struct AttnArgs {
   int out_f32;              // the output is float whatever the activation type (something follows before it is rounded)
 };
 
-template <typename T>
+template <typename T, int MAX_HD>
 __global__ void __launch_bounds__(ATT_WARPS * 32) attention_simt_kernel(AttnArgs a) {
-  __shared__ float qs[ATT_WARPS][ATT_MAX_HD];
+  __shared__ float qs[ATT_WARPS][MAX_HD];
   pdl_wait();
   pdl_launch();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -66,9 +66,9 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attention_simt_kernel(AttnArgs
   if (a.sink != nullptr) { m = a.sink[h]; l = 1.0f; }
   const bool gated = a.gate_bias != nullptr;
   const float gb = gated ? a.gate_bias[h] : 0.0f;
-  float o[ATT_MAX_HD / 32];
+  float o[MAX_HD / 32];
 #pragma unroll
-  for (int i = 0; i < ATT_MAX_HD / 32; ++i) o[i] = 0.0f;
+  for (int i = 0; i < MAX_HD / 32; ++i) o[i] = 0.0f;
 
   for (int j0 = lo; j0 <= p; j0 += 32) {
     const int j = j0 + lane;
@@ -91,7 +91,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attention_simt_kernel(AttnArgs
       l = l * corr + warp_sum(pj);
       m = m_new;
 #pragma unroll
-      for (int i = 0; i < ATT_MAX_HD / 32; ++i) o[i] *= corr;
+      for (int i = 0; i < MAX_HD / 32; ++i) o[i] *= corr;
     }
     const int nk = (p - j0 + 1 < 32) ? p - j0 + 1 : 32;
     for (int k = 0; k < nk; ++k) {
@@ -100,7 +100,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attention_simt_kernel(AttnArgs
       const int page = pages[jk / a.page_size];
       const T* vr = (const T*)a.vcache + ((size_t)page * a.nkv + kvh) * head_stride + (size_t)(jk % a.page_size) * a.hd;
 #pragma unroll
-      for (int i = 0; i < ATT_MAX_HD / 32; ++i) {
+      for (int i = 0; i < MAX_HD / 32; ++i) {
         const int d = lane + 32 * i;
         if (d < a.hd) o[i] = fmaf(pk, to_f32(vr[d]), o[i]);
       }
@@ -111,7 +111,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attention_simt_kernel(AttnArgs
   T* op = (T*)a.out + (size_t)t * a.ldo + (size_t)h * a.hd;
   float* of = (float*)a.out + (size_t)t * a.ldo + (size_t)h * a.hd;
 #pragma unroll
-  for (int i = 0; i < ATT_MAX_HD / 32; ++i) {
+  for (int i = 0; i < MAX_HD / 32; ++i) {
     const int d = lane + 32 * i;
     if (d >= a.hd) continue;
     if (a.out_f32) of[d] = o[i] * inv;
@@ -134,10 +134,13 @@ extern "C" int hb_attention_simt(int dtype, const void* q, int ldq, void* out, i
              n_tokens, nh, nkv, hd, page_size, scale, window, softcap, sink, gate_bias, out_gate, ldg, out_f32};
   const long long blocks = ceil_div_ll((long long)n_tokens * nh, ATT_WARPS);
   HB_REQUIRE(blocks < 2147483647LL, "attention: too many (token, head) pairs");
-  if (dtype == HB_F32)
-    hb_launch(attention_simt_kernel<float>, dim3((unsigned)blocks), dim3(ATT_WARPS * 32), 0, (cudaStream_t)stream, a);
-  else
-    hb_launch(attention_simt_kernel<bf16>, dim3((unsigned)blocks), dim3(ATT_WARPS * 32), 0, (cudaStream_t)stream, a);
+#define AS_GO(T, MAX_HD) hb_launch(attention_simt_kernel<T, MAX_HD>, dim3((unsigned)blocks), dim3(ATT_WARPS * 32), 0, (cudaStream_t)stream, a)
+  if (dtype == HB_F32) {
+    if (hd <= 256) AS_GO(float, 256); else AS_GO(float, 512);
+  } else {
+    if (hd <= 256) AS_GO(bf16, 256); else AS_GO(bf16, 512);
+  }
+#undef AS_GO
   HB_CHECK_LAUNCH("attention_simt");
   return 0;
 }

@@ -198,7 +198,7 @@ def _attention_case(dtype, nh, nkv, hd, lens, qlens, window, page=16, seed=5, sh
 
 
 @pytest.mark.parametrize("dtype", DT)
-@pytest.mark.parametrize("nh,nkv,hd", [(4, 2, 16), (6, 3, 48), (8, 1, 128), (5, 5, 80), (12, 4, 64), (2, 1, 256), (3, 1, 112)])
+@pytest.mark.parametrize("nh,nkv,hd", [(4, 2, 16), (6, 3, 48), (8, 1, 128), (5, 5, 80), (12, 4, 64), (2, 1, 256), (3, 1, 112), (2, 1, 400)])
 @pytest.mark.parametrize("window", [None, 21])
 def test_attention_simt_prefill_and_decode_shapes(dtype, nh, nkv, hd, window):
     for lens, qlens in [([1, 70, 33], [1, 70, 33]), ([200, 17, 64, 65], [1, 1, 1, 1]), ([90, 50], [7, 50])]:
@@ -357,8 +357,11 @@ def test_sample_refuses_bad_options():
     x = dev(torch.zeros(1, 8)); u = dev(torch.zeros(1)); o = torch.empty(1, dtype=torch.int32, device="cuda")
     with pytest.raises(BackendError, match="temperature must be > 0"):
         ops.sample(x, 0.0, 0, 1.0, u, o)
-    with pytest.raises(BackendError, match="head size 272 exceeds"):
-        ops.attention_simt(x, 8, x, x, x, o, o, o, 1, 1, 272, 16, 1.0, None)
+    # operands of the size they are said to have: were the size allowed, nothing would be read out of bounds
+    q, out = dev(torch.zeros(1, 528)), dev(torch.zeros(1, 528))
+    cache, zero = dev(torch.zeros(1, 1, 16, 528)), torch.zeros(1, dtype=torch.int32, device="cuda")
+    with pytest.raises(BackendError, match="head size 528 exceeds"):
+        ops.attention_simt(q, 528, out, cache, cache, zero, zero, zero.view(1, 1), 1, 1, 528, 16, 1.0, None)
     with pytest.raises(BackendError, match="CUDA tensor"):
         ops.argmax(torch.zeros(1, 8), o)
 

@@ -308,7 +308,7 @@ def test_latent_rows_rotated_in_either_layout(dtype, halves):
     assert_close(to_np(out.view(T, H, rank + rot)[:, :, rank:]), want.numpy(), "float32", "rotated parts of the queries")
 
 
-@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 32, 64), (2, 1, 8, 16), (8, 2, 64, 128), (2, 2, 24, 40), (6, 3, 40, 80), (2, 1, 64, 100), (4, 1, 20, 50), (4, 2, 120, 200)])
+@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 32, 64), (2, 1, 8, 16), (8, 2, 64, 128), (2, 2, 24, 40), (6, 3, 40, 80), (2, 1, 64, 100), (4, 1, 20, 50), (4, 2, 120, 200), (2, 1, 150, 40)])
 def test_difference_of_two_maps_in_every_attention_kernel(H, G, dk, dv):
     """One sequence of 300 cached keys in pages that are not in order; the queries of the last 150 positions as a prompt's
     portion and the last one alone.  Scaled queries make one far key, keys at page borders and the query's own key stand
@@ -601,6 +601,7 @@ OTHER = {
     "wide_states_and_heads": ([(U.mamba(heads=2, vdim=160, state=264, groups=1, norm_groups=5), None), (U.mamba(heads=2, vdim=96, state=160, groups=2), None),
                                (U.latent(heads=2, dim=40, rot_dim=24, vdim=96, kv_rank=200), None)], {"streams": 2}),
     "everything_looped": ([(U.latent(), U.dense(limit=0.4)), (U.mamba(), U.dense()), (U.attention(), None)], {"loop": (0, 3, 2), "streams": 9}),
+    "heads_of_320": ([(U.attention(heads=2, kv_heads=1, dim=160, vdim=48, rot_dims=32), None)], {"streams": 2}),
     "heads_of_256": ([(U.attention(heads=2, kv_heads=1, dim=128, vdim=256, rot_dims=64), None)], {"streams": 2}),
 }
 
