@@ -21,7 +21,8 @@ from typing import Optional, Sequence
 class NormSpec:
     """A normalisation over the last axis.  kind "rmsnorm": y = x / sqrt(mean(x^2) + eps) * w;
     kind "layernorm": y = (x - mean(x)) / sqrt(var(x) + eps) * w (+ b with `bias`, a tensor named as the weight with
-    `bias_suffix` added).  `weight_offset` c: the
+    `bias_suffix` added); kind "dynamic_tanh": y = tanh(alpha * x) * w + b, no statistics and no use of eps, alpha one number in a
+    tensor named as the weight with `alpha_suffix` added, b always there.  `weight_offset` c: the
     stored tensor is w - c (a weight kept around zero with c = 1), so the factor is c + stored."""
 
     dim: int
@@ -34,6 +35,7 @@ class NormSpec:
     groups: int = 1
     bias: bool = False              # layernorm only
     bias_suffix: str = ".b"
+    alpha_suffix: str = ".alpha"    # dynamic_tanh only
 
 
 @dataclass(frozen=True)
@@ -177,10 +179,20 @@ class AttentionSpec:
     # `reads_kv`: the mixer has no key and value tensors: its schedule step reads what another step stored;
     # `cache_window`: how many of the last keys the cache must keep, where that differs from the mixer's own window
     #     (another step with a longer window reads this one's keys); -1: the mixer's window, None: every key.
+    # `head_qk_norm`: every head of q and of k is divided by its own root mean square and multiplied by a weight of head_dim
+    #     that all heads share (tensors `norm_names`, eps of `qk_norm`), before the rotation;
+    # `output_bias`: the output projection adds a vector, named as its matrix with `bias_suffix`;
+    # `value_blend`: "keep": the mixer's values of the step's tokens are kept for later layers of the same step; "blend":
+    #     v <- (1 - lambda) v + lambda v_kept before v is stored, lambda the one number of tensor `value_blend_name` (which
+    #     a mixer that keeps has too, without using it).
     # `difference` c: two softmax maps per head over the same values, subtracted.  q and k have twice the rows (head by head
     #     map 1, map 2, each of `head_dim` and rotated alike); with lambda = exp(a1 . b1) - exp(a2 . b2) + c (four vectors of
     #     head_dim, tensors `difference_names`) a head's result is o = map1 - lambda map2, divided by sqrt(mean(o^2) +
     #     difference_eps) over its value channels and multiplied by 1 - c.
+    head_qk_norm: bool = False
+    output_bias: bool = False
+    value_blend: Optional[str] = None
+    value_blend_name: str = "vmix"
     difference: Optional[float] = None
     difference_eps: float = 0.0
     difference_names: tuple = ("lq1", "lk1", "lq2", "lk2")
@@ -247,6 +259,45 @@ class GeneralDeltaSpec:
     decay_constant: float
     unit_eps: float = 1e-6
     kind: str = "general_delta"
+    names: tuple = ()          # pairs (role, tensor name) that replace the mixer's defaults
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """A matrix memory with exponential gates (mLSTM): per head i = c tanh((I h + bi) / c), f = log sigmoid(c tanh((F h + bf) / c))
+    with c = `gate_cap`; m <- max(f + m, i) from m = 0; S <- e^(f + m_old - m) S + e^(i - m) k v^T, n likewise with k alone;
+    o = S^T q / (max(|n . q|, e^(-m)) + read_eps), q also times key_dim^-1/2.  Each head's o is divided by its root mean square,
+    the heads side by side are multiplied by a weight (one number per head and channel) and by sigmoid(G h), then projected."""
+
+    hidden_size: int
+    num_heads: int
+    key_dim: int
+    value_dim: int
+    gate_cap: float
+    norm_eps: float
+    read_eps: float = 1e-6
+    kind: str = "matrix_memory"
+    names: tuple = ()          # pairs (role, tensor name) that replace the mixer's defaults
+
+
+@dataclass(frozen=True)
+class ChannelDeltaSpec:
+    """The gated delta rule with a decay per key channel: per head S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q,
+    with q, k of `qk_heads` heads, each of q, k, v through a short causal convolution and silu, unit q and k per head (q also times
+    key_dim^-1/2), beta = sigmoid(B h), g = exp(-exp(A_log) softplus(A2 A1 h + dt_bias)) with one A_log per head; per-head RMS norm
+    of o (weight of value_dim, shared), gate sigmoid(G2 G1 h), output product.  The inner widths of A and G are the stored
+    tensors'; random weights take `low_rank`."""
+
+    hidden_size: int
+    num_heads: int
+    qk_heads: int
+    key_dim: int
+    value_dim: int
+    conv_taps: int
+    norm_eps: float
+    unit_eps: float = 1e-6
+    low_rank: int = 16
+    kind: str = "channel_delta"
     names: tuple = ()          # pairs (role, tensor name) that replace the mixer's defaults
 
 
@@ -336,7 +387,8 @@ class RoutedFFSpec:
     `group_top` largest scores, and only experts of the `keep_groups` best groups can be chosen;
     `weight_scale`: a factor on every chosen weight; `shared`: a dense gated feed-forward (its own
     spec, which also names its tensors) that runs for every token and is added.  activation "swish_clamp" (gated
-    experts only) takes `act_limit` L: g = min(gate, L), u = clamp(up, -L, L), hidden = g sigmoid(1.702 g) (u + 1)."""
+    experts only) takes `act_limit` L: g = min(gate, L), u = clamp(up, -L, L), hidden = g sigmoid(1.702 g) (u + 1).
+    `weigh_input` (gated experts only): a weight multiplies the expert's input instead of its output."""
 
     hidden_size: int
     num_experts: int
@@ -355,6 +407,7 @@ class RoutedFFSpec:
     weight_scale: float = 1.0
     shared: Optional[SwiGLUSpec] = None
     act_limit: float = 0.0
+    weigh_input: bool = False
 
 
 @dataclass(frozen=True)
@@ -368,7 +421,8 @@ class BlockSpec:
     `input_conv_taps` the mixer reads x + conv(x) instead, a causal convolution over time on each
     channel (tensor `input_conv_name`, [width, taps], the last column weighs the token itself).
     kind "parallel": h = norm1(x); out = x + residual_mult * (mixer(h) + ffn(h)): one norm, both
-    sublayers read its result; `ffn` may be None; norm2 is unused (None).
+    sublayers read its result; with norm2 given the feed-forward reads norm2(x) instead; `ffn` may be None (then norm2 is
+    unused).
     kind "sandwich": a norm before and after each sublayer, h = norm1(x); x <- x + post1(mixer(h) * gate1);
     h = norm2(x); x <- x + post2(ffn(h) * gate2): `post_norms` are the two norms of the results, `residual_gates`
     (None: no gates) names two matrices R with biases (R's name + `residual_gate_bias`): gate = sigmoid(R h + b), a
@@ -448,6 +502,10 @@ class ModelSpec:
     logit_softcap: Optional[float] = None
     # (tensor name, columns): a second table [vocab, columns] of which blocks with a `token_side` read their columns
     token_side_table: Optional[tuple] = None
+    # the logits are multiplied by this
+    logit_scale: float = 1.0
+    # tensors that a file may hold without being used
+    unused_names: tuple = ()
     # n: the residual is n copies of the stream, all equal to the embedding at the start and summed before the final norm
     # (blocks of kind "streams"); None: one stream
     streams: Optional[int] = None

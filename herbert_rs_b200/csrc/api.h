@@ -111,9 +111,9 @@ long long hb_gemm_tcgen05_workspace_floats(int ctas);
 int hb_gemm_tcgen05_set_workspace(float* floats, int* counters, int ctas);
 int hb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N, int K, int
     epi, float glu_limit, int* error_flag, void* stream);
-int hb_gemm_tcgen05_grouped_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M_max, int
-    N, int K, int E, int epi, float glu_limit, const int* rows_used, const int* tile_expert, int* error_flag, void*
-    stream);
+int hb_gemm_tcgen05_grouped_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M_max,
+    int N, int K, int E, int epi, float glu_limit, const float* row_scale, const int* rows_used, const int*
+    tile_expert, int* error_flag, void* stream);
 int hb_gemm_tcgen05_qkv_ok(int M, int N);
 int hb_gemm_tcgen05_qkv_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M, int N,
     int K, const float* in_sumsq, int in_parts, int in_stride, float in_eps, const float* qw, const float* kw,
@@ -164,16 +164,16 @@ int hb_layernorm_residual(int dtype, const float* y, int ldy, const float* w, co
 int hb_moe_route(int dtype, const void* h, int ld, const void* w_router, int* ids, float* weights, int n_tokens,
     int D, int E, int top, int renorm, int sigmoid, int groups, int keep, int group_top, float wscale, void* stream);
 int hb_moe_experts(int dtype, const void* h, int ld, const void* up, const void* down, const int* ids, const
-    float* weights, void* mid, float* y, int ldy, int n_tokens, int D, int F, int top, int act, int gated, float
-    act_limit, int accumulate, void* stream);
+    float* weights, void* mid, float* y, int ldy, int n_tokens, int D, int F, int top, int act, int gated,
+    float act_limit, int weigh_input, int accumulate, void* stream);
 long long hb_moe_grouped_scratch_ints(int n_tokens, int E, int top);
 int hb_moe_experts_tc_rows(int n_tokens, int E, int top);
-int hb_moe_experts_tc_bf16(const void* h, int ld, const void* up, const void* down, const int* ids, const float*
-    weights, int* ints, void* sorted, void* mid, float* part, float* y, int ldy, int n_tokens, int D, int E, int F,
-    int top, float act_limit, int accumulate, int* error_flag, void* stream);
+int hb_moe_experts_tc_bf16(const void* h, int ld, const void* up, const void* down, const int* ids, const
+    float* weights, int* ints, void* sorted, void* mid, float* part, float* y, int ldy, int n_tokens, int D,
+    int E, int F, int top, float act_limit, float* row_scale, int accumulate, int* error_flag, void* stream);
 int hb_moe_experts_grouped_bf16(const void* h, int ld, const void* up, const void* down, const int* ids, const
-    float* weights, int* scratch, void* mid, float* part, float* y, int ldy, int n_tokens, int D, int E, int F, int
-    top, int act, int gated, float act_limit, int accumulate, void* stream);
+    float* weights, int* scratch, void* mid, float* part, float* y, int ldy, int n_tokens, int D, int E, int
+    F, int top, int act, int gated, float act_limit, int weigh_input, int accumulate, void* stream);
 
 // qk_prepare.cu: biases, query temperature and cache write for a mixer that neither norms nor rotates its heads
 int hb_qk_prepare_cache(int dtype, const float* qkv, int ld, const float* bias, void* q_out, int ldq, float
@@ -217,15 +217,16 @@ int hb_delta_prepare(float* qk, int ld, int q_off, int k_off, int qk_heads, int 
 int hb_linear_scan(int delta, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const
     float* gates, const float* decay, float* state, const int* seq_slot, const int* seq_start, float* out, int ldo,
     int n_seqs, int max_q_len, int heads, int qk_heads, int dk, int dv, void* stream);
-int hb_gated_rmsnorm(int dtype, const float* o, int ldo, const float* w, float eps, const float* gate, int ldg, void*
-    y, int ldy, int n_tokens, int units, int n, int act, int w_stride, int gate_first, void* stream);
+int hb_gated_rmsnorm(int dtype, const float* o, int ldo, int o_stride, const float* w, float eps, const float*
+    gate, int ldg, void* y, int ldy, int n_tokens, int units, int n, int act, int w_stride, int gate_first,
+    const float* floor_, float div_scale, float div_eps, void* stream);
 
 // rotary_pairs.cu: whole-projection q/k norm, rotation of pairs by position (q, k and v), cache write; the turn back of the results
-int hb_qkv_rotary_cache(int dtype, const float* rows, int ld, const float* bias, const float* wq, const float* wk,
-    float eps, int whole_norm, const float* fqk, int rot, int halves, float mscale, const float* fv, const int*
-    tok_seq, const int* tok_pos, const int* seq_pages, int pages_stride, void* q_out, int ldq, void* kcache, void*
-    vcache, int n_tokens, int nh, int nkv, int maps, int dk, int dv, int hd, int page_size, int write_cache, void*
-    stream);
+int hb_qkv_rotary_cache(int dtype, const float* rows, int ld, const float* bias, const float* wq, const float*
+    wk, float eps, int norm, const float* fqk, int rot, int halves, float mscale, const float* fv, const int*
+    tok_seq, const int* tok_pos, const int* seq_pages, int pages_stride, void* q_out, int ldq, void* kcache,
+    void* vcache, int n_tokens, int nh, int nkv, int maps, int dk, int dv, int hd, int page_size, int
+    write_cache, const float* blend, float lambda, float* keep, void* stream);
 int hb_rotate_heads_back(int dtype, const void* att, int ld, int hd, const float* fv, int halves, const int*
     tok_pos, void* y, int ldy, int n_tokens, int nh, int dv, void* stream);
 int hb_difference_heads(int dtype, const float* att, int ld, int hd, float lambda, float factor, float eps, void* y,
@@ -233,10 +234,14 @@ int hb_difference_heads(int dtype, const float* att, int ld, int hd, float lambd
 int hb_head_gate(int dtype, const void* att, int ld, int hd, const float* gate, int ldg, void* y, int ldy, int
     n_tokens, int nh, int dv, void* stream);
 
-// general_delta.cu: the generalised delta rule (decay per key channel, removal along the unit key): its vectors, its recurrence
+// general_delta.cu: the generalised delta rule (decay per key channel, removal along the unit key): its vectors (also those of the delta rule with a decay per key channel), its recurrence
 int hb_general_delta_prepare(int dtype, const float* rows, int ld, int r_off, int k_off, int a_off, int low_off,
     const void* w2, const float* w0, const float* a0, float decay_c, float unit_eps, float* prep, int n_tokens, int
     heads, int dk, int rank, void* stream);
+int hb_channel_delta_prepare(int dtype, const float* qk, int ldqk, int q_off, int k_off, const float* rows,
+    int ld, int b_off, int low_off, const void* w2, const float* dt_bias, const float* a_log, float unit_eps,
+    float qscale, float* prep, int gate_off, int gate_rank, void* gate_low, int ldgl, int n_tokens, int heads,
+    int qk_heads, int dk, int rank, void* stream);
 int hb_general_delta_scan(const float* prep, const float* v, int ldv, float* state, const int* seq_slot, const int*
     seq_start, float* out, int ldo, int n_seqs, int heads, int dk, int dv, void* stream);
 
@@ -252,14 +257,26 @@ int hb_streams_join(int dtype, float* x, int n, const float* y, int ldy, const f
     void* stream);
 
 // state_space.cu: a state-space recurrence with one decay and step size per token and head
-int hb_ssd_scan(int dtype, const void* xbc, int ld, int b_off, int c_off, const float* dt, int lddt, const float*
-    dt_bias, const float* a_log, const float* dskip, float* state, const int* seq_slot, const int* seq_start, float*
-    out, int ldo, int n_seqs, int heads, int groups, int N, int dv, void* stream);
+int hb_ssd_scan(int dtype, const void* xbc, int ld, int b_off, int c_off, const float* dt, int lddt, const
+    float* logd, const float* dt_bias, const float* a_log, const float* dskip, float* state, const int*
+    seq_slot, const int* seq_start, float* out, int ldo, int n_seqs, int heads, int groups, int N, int dv,
+    void* stream);
 int hb_ssd_chunks(int n_tokens, int n_seqs, int N, int dv);
 int hb_ssd_chunked_bf16(const void* xbc, int ld, int b_off, int c_off, const float* dt, int lddt, const float*
-    dt_bias, const float* a_log, const float* dskip, float* state, const int* seq_slot, const int* seq_start, float*
-    out, int ldo, int n_seqs, int max_q_len, int heads, int groups, int N, int dv, float* chunk_state, float*
-    chunk_decay, void* stream);
+    logd, const float* dt_bias, const float* a_log, const float* dskip, float* state, const int* seq_slot,
+    const int* seq_start, float* out, int ldo, int n_seqs, int max_q_len, int heads, int groups, int N, int
+    dv, float* chunk_state, float* chunk_decay, void* stream);
+
+// matrix_memory.cu: a matrix-memory mixer's gates with their running maximum, its values, keys and queries packed for the recurrence
+int hb_matrix_memory_prepare(int dtype, const float* rows, int ld, int q_off, int k_off, int v_off, int i_off,
+    int f_off, const float* i_bias, const float* f_bias, float cap, float* m_state, const int* seq_slot, const
+    int* seq_start, void* packed, int ldp, float* logd, float* weight, float* floor_, int n_tokens, int
+    n_seqs, int max_q_len, int heads, int dk, int dv, int dvp, void* stream);
+
+// dynamic_tanh.cu: a norm without statistics, alone and behind the residual sum of a block
+int hb_residual_tanh(int dtype, const float* y, int ldy, const float* yb, float mult, float* x, const int*
+    rows, float alpha1, const float* w1, const float* b1, void* h1, float alpha2, const float* w2, const
+    float* b2, void* h2, int n_rows, int dim, void* stream);
 
 #ifdef __cplusplus
 }

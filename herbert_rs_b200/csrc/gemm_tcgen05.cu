@@ -238,6 +238,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         for (int i = 0; i < nm.in_parts; ++i) sum += nm.in_sumsq[(size_t)i * nm.in_stride + m];
         inv_rms = rsqrtf(sum / (float)K + nm.in_eps);
       }
+      if (NORM && nm.row_scale != nullptr && m < M) inv_rms = nm.row_scale[m];
       if (!mbar_wait(acc_full(buf), (local >> 1) & 1)) {
         if (lane == 0) atomicExch(error_flag, 3);
         ok = false;
@@ -793,9 +794,10 @@ extern "C" int hb_gemm_tcgen05_bf16(const void* A, int lda, const void* W, int l
 // 128 rows; W [E * N, K] stacks the experts' matrices; tile i of A (128 rows) is multiplied by the matrix of expert
 // tile_expert[i]; only the first *rows_used rows are computed (both written on the device before this launch).
 // C [M_max, N] (EPI_STORE, EPI_STORE_F32) or [M_max, N / 2] (EPI_SWIGLU; with glu_limit > 0 the clamped form of the gated
-// activation).  Rows of padding are computed and mean nothing.
+// activation).  row_scale [M_max]: a factor per row on the results, before the activation; or null.  Rows of padding are
+// computed and mean nothing.
 extern "C" int hb_gemm_tcgen05_grouped_bf16(const void* A, int lda, const void* W, int ldw, void* C, int ldc, int M_max,
-                                            int N, int K, int E, int epi, float glu_limit, const int* rows_used,
+                                            int N, int K, int E, int epi, float glu_limit, const float* row_scale, const int* rows_used,
                                             const int* tile_expert, int* error_flag, void* stream) {
   HB_REQUIRE(M_max > 0 && N > 0 && K > 0 && E > 0, "gemm_tcgen05_grouped: sizes must be positive");
   HB_REQUIRE(M_max % TG_BM == 0, "gemm_tcgen05_grouped: %d rows are not whole tiles of %d", M_max, TG_BM);
@@ -814,10 +816,15 @@ extern "C" int hb_gemm_tcgen05_grouped_bf16(const void* A, int lda, const void* 
   cudaStream_t s = (cudaStream_t)stream;
   TgNorm none{};
   none.glu_limit = epi == HB_EPI_SWIGLU ? glu_limit : 0.0f;
+  none.row_scale = row_scale;
+  HB_REQUIRE(row_scale == nullptr || epi == HB_EPI_SWIGLU, "gemm_tcgen05_grouped: a factor per row goes with the gated epilogue");
   TgGrouped grp;
   grp.rows_used = rows_used;
   grp.tile_expert = tile_expert;
   grp.expert_rows = N;
+  if (row_scale != nullptr)
+    return BN == 256 ? tg_launch<256, HB_EPI_SWIGLU, true>(ma, mw, C, ldc, M_max, N, K, error_flag, s, none, grp)
+                     : tg_launch<128, HB_EPI_SWIGLU, true>(ma, mw, C, ldc, M_max, N, K, error_flag, s, none, grp);
   if (BN == 256) {
     if (epi == HB_EPI_SWIGLU) return tg_launch<256, HB_EPI_SWIGLU, false>(ma, mw, C, ldc, M_max, N, K, error_flag, s, none, grp);
     if (epi == HB_EPI_STORE) return tg_launch<256, HB_EPI_STORE, false>(ma, mw, C, ldc, M_max, N, K, error_flag, s, none, grp);

@@ -34,6 +34,8 @@ struct TgNorm {
   // SwiGLU epilogue only.  > 0: the clamped form with this limit L, min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1),
   // in place of silu(g) u
   float glu_limit;
+  // A factor per row of A by which the results are multiplied, in place of 1 / rms (the product grouped by expert); or null
+  const float* row_scale;
 };
 
 // The q/k/v product whose epilogue also does what follows it in an attention layer with heads of

@@ -14,6 +14,11 @@
 // pieces or token by token performs the same float operations in the same order.  Everything here is float on both
 // paths; only W2 arrives in the compute type (its products are exact, the sums float).
 //
+// The delta rule with a decay per key channel, S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T with unit keys, is the
+// case w = g, u = g * k, a * u -> beta k, k -> beta k.
+//
+//   hb_channel_delta_prepare   that form's vectors, in the same packing, from convolved q and k rows: unit vectors per head
+//                              (q also times a scale), beta = sigmoid(b), g = exp(-exp(A_log) softplus(W2 low + dt_bias))
 //   hb_general_delta_prepare   from the projection's float rows: the five key-side vectors of every (token, head),
 //                              packed as [T][H][5][dk]: r, k, w, u, a * u
 //   hb_general_delta_scan      the recurrence
@@ -121,6 +126,121 @@ extern "C" int hb_general_delta_prepare(int dtype, const float* rows, int ld, in
   else
     hb_launch(general_delta_prepare_kernel<bf16>, grid, dim3(threads), smem, (cudaStream_t)stream, a);
   HB_CHECK_LAUNCH("general_delta_prepare");
+  return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// The same for the delta rule with a decay per key channel.  Value head h reads query/key head h / (H / G).  The CTAs of
+// head 0 also round the inner row of a low-rank output gate to the compute type, for the product that widens it.
+struct CdPrepArgs {
+  const float* qk; int ldqk; int q_off, k_off;      // convolved rows: [G dk] each
+  const float* rows; int ld; int b_off, low_off;    // the projection's rows: [H] and [rank]
+  const void* w2;                                   // [H dk][rank], compute type
+  const float* dt_bias;                             // [H dk]
+  const float* a_log;                               // [H]
+  float unit_eps, qscale;
+  float* prep;                                      // [T][H][5][dk]
+  int gate_off, gate_rank; void* gate_low; int ldgl;      // rows[:, gate_off ..] -> gate_low [T][ldgl]; gate_rank 0: none
+  int n_tokens, H, G, dk, rank;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(GP_MAX_THREADS) channel_delta_prepare_kernel(CdPrepArgs a) {
+  extern __shared__ float lows[];   // [GP_TOK][rank]
+  __shared__ float red[2][GP_TOK][GP_MAX_THREADS / 32];
+  __shared__ float coef[3][GP_TOK];           // q's factor, k's factor, beta
+  pdl_wait();
+  pdl_launch();
+  const int t0 = blockIdx.x * GP_TOK, h = blockIdx.y;
+  const int nt = a.n_tokens - t0 < GP_TOK ? a.n_tokens - t0 : GP_TOK;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
+  const size_t qh = (size_t)(h / (a.H / a.G)) * a.dk;
+  const float* q = a.qk + (size_t)t0 * a.ldqk + a.q_off + qh;
+  const float* k = a.qk + (size_t)t0 * a.ldqk + a.k_off + qh;
+  for (int i = threadIdx.x; i < nt * a.rank; i += blockDim.x) {
+    const int tt = i / a.rank, j = i - tt * a.rank;
+    lows[i] = a.rows[(size_t)(t0 + tt) * a.ld + a.low_off + j];
+  }
+  if (h == 0)
+    for (int i = threadIdx.x; i < nt * a.gate_rank; i += blockDim.x) {
+      const int tt = i / a.gate_rank, j = i - tt * a.gate_rank;
+      ((T*)a.gate_low)[(size_t)(t0 + tt) * a.ldgl + j] = from_f32<T>(a.rows[(size_t)(t0 + tt) * a.ld + a.gate_off + j]);
+    }
+  float sq[GP_TOK], sk[GP_TOK];
+#pragma unroll
+  for (int tt = 0; tt < GP_TOK; ++tt) sq[tt] = sk[tt] = 0.0f;
+  for (int i = threadIdx.x; i < a.dk; i += blockDim.x) {
+#pragma unroll
+    for (int tt = 0; tt < GP_TOK; ++tt)
+      if (tt < nt) {
+        const float x = q[(size_t)tt * a.ldqk + i], y = k[(size_t)tt * a.ldqk + i];
+        sq[tt] = fmaf(x, x, sq[tt]);
+        sk[tt] = fmaf(y, y, sk[tt]);
+      }
+  }
+#pragma unroll
+  for (int tt = 0; tt < GP_TOK; ++tt) {
+    const float x = warp_sum(sq[tt]), y = warp_sum(sk[tt]);
+    if (lane == 0) { red[0][tt][warp] = x; red[1][tt][warp] = y; }
+  }
+  __syncthreads();
+  if (threadIdx.x < 2 * GP_TOK) {
+    const int which = threadIdx.x / GP_TOK, tt = threadIdx.x % GP_TOK;
+    float v = 0.0f;
+    for (int w = 0; w < nwarp; ++w) v += red[which][tt][w];
+    coef[which][tt] = (which == 0 ? a.qscale : 1.0f) / sqrtf(v + a.unit_eps);
+    if (which == 0 && tt < nt) coef[2][tt] = 1.0f / (1.0f + expf(-a.rows[(size_t)(t0 + tt) * a.ld + a.b_off + h]));
+  }
+  __syncthreads();
+  const T* w2 = (const T*)a.w2;
+  const float rate = expf(a.a_log[h]);
+  for (int i = threadIdx.x; i < a.dk; i += blockDim.x) {
+    const int c = h * a.dk + i;
+    const T* wr = w2 + (size_t)c * a.rank;
+    float z[GP_TOK];
+    const float z0 = a.dt_bias[c];
+#pragma unroll
+    for (int tt = 0; tt < GP_TOK; ++tt) z[tt] = z0;
+    for (int j = 0; j < a.rank; ++j) {
+      const float w = to_f32(wr[j]);
+#pragma unroll
+      for (int tt = 0; tt < GP_TOK; ++tt)
+        if (tt < nt) z[tt] = fmaf(lows[tt * a.rank + j], w, z[tt]);
+    }
+#pragma unroll
+    for (int tt = 0; tt < GP_TOK; ++tt)
+      if (tt < nt) {
+        float* out = a.prep + ((size_t)(t0 + tt) * a.H + h) * 5 * a.dk;
+        const float g = expf(-rate * (fmaxf(z[tt], 0.0f) + log1pf(expf(-fabsf(z[tt])))));
+        const float ku = k[(size_t)tt * a.ldqk + i] * coef[1][tt], bk = coef[2][tt] * ku;
+        out[i] = q[(size_t)tt * a.ldqk + i] * coef[0][tt];
+        out[a.dk + i] = bk;
+        out[2 * a.dk + i] = g;
+        out[3 * a.dk + i] = g * ku;
+        out[4 * a.dk + i] = bk;
+      }
+  }
+}
+
+extern "C" int hb_channel_delta_prepare(int dtype, const float* qk, int ldqk, int q_off, int k_off, const float* rows, int ld,
+                                        int b_off, int low_off, const void* w2, const float* dt_bias, const float* a_log,
+                                        float unit_eps, float qscale, float* prep, int gate_off, int gate_rank, void* gate_low,
+                                        int ldgl, int n_tokens, int heads, int qk_heads, int dk, int rank, void* stream) {
+  HB_REQUIRE(n_tokens > 0 && heads > 0 && qk_heads > 0 && dk > 0 && rank > 0, "channel_delta_prepare: sizes must be positive");
+  HB_REQUIRE(heads % qk_heads == 0, "channel_delta_prepare: %d heads are not a multiple of %d query/key heads", heads, qk_heads);
+  const size_t smem = (size_t)GP_TOK * rank * sizeof(float);
+  HB_REQUIRE(smem <= 40 * 1024, "channel_delta_prepare: the decay's inner width %d exceeds what a block keeps in shared memory", rank);
+  HB_REQUIRE(heads <= 65535, "channel_delta_prepare: too many heads");
+  HB_REQUIRE(gate_rank == 0 || (gate_rank > 0 && gate_low != nullptr && ldgl >= gate_rank), "channel_delta_prepare: the gate's inner row needs a place");
+  const CdPrepArgs a{qk, ldqk, q_off, k_off, rows, ld, b_off, low_off, w2, dt_bias, a_log, unit_eps, qscale, prep,
+                     gate_off, gate_rank, gate_low, ldgl, n_tokens, heads, qk_heads, dk, rank};
+  dim3 grid(ceil_div(n_tokens, GP_TOK), heads);
+  const int threads = dk >= GP_MAX_THREADS ? GP_MAX_THREADS : ceil_div(dk, 32) * 32;
+  if (dtype == HB_F32)
+    hb_launch(channel_delta_prepare_kernel<float>, grid, dim3(threads), smem, (cudaStream_t)stream, a);
+  else
+    hb_launch(channel_delta_prepare_kernel<bf16>, grid, dim3(threads), smem, (cudaStream_t)stream, a);
+  HB_CHECK_LAUNCH("channel_delta_prepare");
   return 0;
 }
 

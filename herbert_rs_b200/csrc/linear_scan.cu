@@ -17,7 +17,9 @@
 //   hb_linear_scan      the recurrence: token by token (decode, short steps, several sequences), or for one long
 //                       prompt alone the delta rule sixteen tokens at a time
 //   hb_gated_rmsnorm    y = o / rms(o) * w * gate-activation(g), the norm per head (w [dv]) or over all heads (w [H dv]);
-//                       with gate_first the gate comes before the norm: v = o * gate-activation(g), y = v / rms(v) * w
+//                       with gate_first the gate comes before the norm: v = o * gate-activation(g), y = v / rms(v) * w;
+//                       with a floor per (token, head) the head's numbers are first divided: o[i] = s o[i] / (max(|s o[n]|, floor)
+//                       + eps'), where o[n], the column behind the head's n, is a normaliser's read-out
 #include "api.h"
 #include "common.cuh"
 
@@ -552,15 +554,20 @@ extern "C" int hb_linear_scan(int delta, const float* q, int ldq, const float* k
 // y[t, u, :] = o / sqrt(mean(o^2) + eps) * w * act(gate): a unit u is one head (w [n] shared by the heads, or with
 // w_stride = n a weight [units * n] with a part for every head) or the whole row of all heads (one unit).
 // act: 0 silu, 1 sigmoid.  gate_first: the gate multiplies o before the norm instead of its result.  One CTA per (token, unit).
+struct HeadDivide {
+  const float* floor_;      // [tokens][units]; null: no division
+  float scale, eps;
+};
 template <typename T>
 __global__ void __launch_bounds__(256)
-gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ w, float eps, const float* __restrict__ gate,
-                     int ldg, T* __restrict__ y, int ldy, int units, int n, int act, int w_stride, int gate_first) {
+gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, int o_stride, const float* __restrict__ w, float eps, const float* __restrict__ gate,
+                     int ldg, T* __restrict__ y, int ldy, int units, int n, int act, int w_stride, int gate_first, HeadDivide hd) {
   __shared__ float red[32];
   pdl_wait();
   pdl_launch();
   const int t = blockIdx.x / units, u = blockIdx.x % units;
-  const float* orow = o + (size_t)t * ldo + (size_t)u * n;
+  const float* orow = o + (size_t)t * ldo + (size_t)u * o_stride;
+  const float pre = hd.floor_ ? hd.scale / (fmaxf(fabsf(hd.scale * orow[n]), hd.floor_[blockIdx.x]) + hd.eps) : 1.0f;
   const float* g = gate + (size_t)t * ldg + (size_t)u * n;
   auto gate_of = [&](int i) {
     const float gv = g[i], sg = 1.0f / (1.0f + expf(-gv));
@@ -572,7 +579,7 @@ gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restri
     const float sg = sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(-gv)) : 1.0f / (1.0f + expf(-gv));
     return act == 0 ? gv * sg : sg;
   };
-  if (n % 4 == 0 && n <= 8 * (int)blockDim.x && ((ldo | ldg | ldy) & 3) == 0 &&
+  if (n % 4 == 0 && n <= 8 * (int)blockDim.x && ((ldo | ldg | ldy | o_stride) & 3) == 0 &&
       (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)y | (uintptr_t)w) & 15) == 0) {      // the same, four columns at once
     float4 v[2], ga[2];
     float s = 0.0f;
@@ -581,6 +588,7 @@ gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restri
       const int i = (threadIdx.x + q * blockDim.x) * 4;
       if (i >= n) continue;
       v[q] = *reinterpret_cast<const float4*>(orow + i);
+      v[q] = make_float4(v[q].x * pre, v[q].y * pre, v[q].z * pre, v[q].w * pre);
       ga[q] = *reinterpret_cast<const float4*>(g + i);
     }
 #pragma unroll
@@ -620,7 +628,7 @@ gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restri
     for (int q = 0; q < 8; ++q) {
       const int i = threadIdx.x + q * blockDim.x;
       v[q] = ga[q] = 0.0f;
-      if (i < n) { v[q] = orow[i]; ga[q] = gate_of(i); }
+      if (i < n) { v[q] = orow[i] * pre; ga[q] = gate_of(i); }
     }
 #pragma unroll
     for (int q = 0; q < 8; ++q) {
@@ -637,7 +645,7 @@ gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restri
   }
   float ss = 0.0f;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float v = gate_first ? orow[i] * gate_of(i) : orow[i];
+    const float v = gate_first ? (orow[i] * pre) * gate_of(i) : orow[i] * pre;
     ss = fmaf(v, v, ss);
   }
   ss = block_sum(ss, red);
@@ -645,25 +653,28 @@ gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, const float* __restri
   T* yr = y + (size_t)t * ldy + (size_t)u * n;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
     const float ga = gate_of(i);
-    yr[i] = from_f32<T>(gate_first ? ((orow[i] * ga) * inv) * w[i] : ((orow[i] * inv) * w[i]) * ga);
+    const float v = orow[i] * pre;
+    yr[i] = from_f32<T>(gate_first ? ((v * ga) * inv) * w[i] : ((v * inv) * w[i]) * ga);
   }
 }
 
-extern "C" int hb_gated_rmsnorm(int dtype, const float* o, int ldo, const float* w, float eps, const float* gate, int ldg,
+extern "C" int hb_gated_rmsnorm(int dtype, const float* o, int ldo, int o_stride, const float* w, float eps, const float* gate, int ldg,
                                 void* y, int ldy, int n_tokens, int units, int n, int act, int w_stride, int gate_first,
-                                void* stream) {
+                                const float* floor_, float div_scale, float div_eps, void* stream) {
   HB_REQUIRE(n_tokens > 0 && units > 0 && n > 0, "gated_rmsnorm: sizes must be positive");
   HB_REQUIRE(act == 0 || act == 1, "gated_rmsnorm: the gate's activation is 0 (silu) or 1 (sigmoid)");
   HB_REQUIRE(w_stride == 0 || w_stride == n, "gated_rmsnorm: the weight is shared by the units (stride 0) or has a part for each (stride %d)", n);
+  HB_REQUIRE(o_stride >= (floor_ ? n + 1 : n), "gated_rmsnorm: units %d apart do not hold their %d numbers%s", o_stride, n, floor_ ? " and the normaliser" : "");
+  const HeadDivide hd{floor_, div_scale, div_eps};
   const long long blocks = (long long)n_tokens * units;
   HB_REQUIRE(blocks < 2147483647LL, "gated_rmsnorm: too many (token, unit) pairs");
   const int threads = n >= 1024 ? 256 : n >= 128 ? 128 : (n >= 64 ? 64 : 32);
   if (dtype == HB_F32)
-    hb_launch(gated_rmsnorm_kernel<float>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, o, ldo, w, eps, gate,
-              ldg, (float*)y, ldy, units, n, act, w_stride, gate_first);
+    hb_launch(gated_rmsnorm_kernel<float>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, o, ldo, o_stride, w, eps, gate,
+              ldg, (float*)y, ldy, units, n, act, w_stride, gate_first, hd);
   else
-    hb_launch(gated_rmsnorm_kernel<bf16>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, o, ldo, w, eps, gate,
-              ldg, (bf16*)y, ldy, units, n, act, w_stride, gate_first);
+    hb_launch(gated_rmsnorm_kernel<bf16>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, o, ldo, o_stride, w, eps, gate,
+              ldg, (bf16*)y, ldy, units, n, act, w_stride, gate_first, hd);
   HB_CHECK_LAUNCH("gated_rmsnorm");
   return 0;
 }

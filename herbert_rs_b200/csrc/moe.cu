@@ -10,7 +10,9 @@
 // Down_e (act(Gate_e h) * (Up_e h)) whose first matrix has 2F rows per expert: `gated` 2: the rows of
 // Gate_e and Up_e in turn in groups of 8 (8 gate rows, the 8 up rows of the same channels, ...: the layout
 // of the dense gated feed-forward, so that a thread of a tensor-core tile holds both halves of a
-// channel); `gated` 1: all gate rows, then all up rows (any F; the few-token kernel only).
+// channel); `gated` 1: all gate rows, then all up rows (any F; the few-token kernel only).  A weight may multiply a gated
+// expert's input instead of its output: then both its products are multiplied before the activation, in float, and the
+// experts' results are added as they are.
 //
 // Three launches, all reading the choice from device memory (nothing of it is known to the host, so
 // a recorded step can be replayed): the router with softmax and choice; the chosen experts' first
@@ -176,11 +178,11 @@ __device__ __forceinline__ float moe_act(float z, int act) {
 }
 
 // mid[(t*top + r), f] = act(Up_e[f, :] . h[t, :]),  e = ids[t, r]; gated: act(gate row f . h) * (up row f . h) of
-// the expert's 2F rows.  One warp per output.
+// the expert's 2F rows, both products times in_w[u] if given.  One warp per output.
 template <typename T>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
-moe_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ up, const int* __restrict__ ids, T* __restrict__ mid,
-              int D, int F, int top, int act, int gated, float limit) {
+moe_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ up, const int* __restrict__ ids, const float* __restrict__ in_w,
+              T* __restrict__ mid, int D, int F, int top, int act, int gated, float limit) {
   pdl_wait();
   pdl_launch();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -191,7 +193,8 @@ moe_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ up, const i
   if (gated) {
     const int grow = gated == 2 ? (f >> 3) * 16 + (f & 7) : f, urow = gated == 2 ? grow + 8 : F + f;
     const T* w = up + (size_t)e * 2 * F * D;
-    const float g = warp_dot(hr, w + (size_t)grow * D, D, lane), v = warp_dot(hr, w + (size_t)urow * D, D, lane);
+    float g = warp_dot(hr, w + (size_t)grow * D, D, lane), v = warp_dot(hr, w + (size_t)urow * D, D, lane);
+    if (in_w) { g *= in_w[u]; v *= in_w[u]; }
     if (lane == 0) mid[(size_t)u * F + f] = from_f32<T>(moe_glu(g, v, act, limit));
     return;
   }
@@ -200,7 +203,7 @@ moe_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ up, const i
   if (lane == 0) mid[(size_t)u * F + f] = from_f32<T>(moe_act(dot, act));
 }
 
-// y[t, d] (+)= sum_r wts[t, r] * Down_e[d, :] . mid[(t*top + r), :].  One warp per output.
+// y[t, d] (+)= sum_r wts[t, r] * Down_e[d, :] . mid[(t*top + r), :] (wts null: 1).  One warp per output.
 template <typename T>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
 moe_down_kernel(const T* __restrict__ mid, const T* __restrict__ down, const int* __restrict__ ids, const float* __restrict__ wts,
@@ -215,7 +218,7 @@ moe_down_kernel(const T* __restrict__ mid, const T* __restrict__ down, const int
     const int u = t * top + r;
     const T* w = down + ((size_t)ids[u] * D + d) * F;
     const T* m = mid + (size_t)u * F;
-    acc = fmaf(wts[u], warp_dot(m, w, F, lane), acc);
+    acc = fmaf(wts ? wts[u] : 1.0f, warp_dot(m, w, F, lane), acc);
   }
   if (lane == 0) {
     float* o = y + (size_t)t * ldy + d;
@@ -225,19 +228,22 @@ moe_down_kernel(const T* __restrict__ mid, const T* __restrict__ down, const int
 
 extern "C" int hb_moe_experts(int dtype, const void* h, int ld, const void* up, const void* down, const int* ids,
                               const float* weights, void* mid, float* y, int ldy, int n_tokens, int D, int F, int top,
-                              int act, int gated, float act_limit, int accumulate, void* stream) {
+                              int act, int gated, float act_limit, int weigh_input, int accumulate, void* stream) {
   HB_REQUIRE(n_tokens > 0 && D > 0 && F > 0 && top > 0, "moe_experts: sizes must be positive");
+  HB_REQUIRE(!weigh_input || gated, "moe_experts: the weight multiplies the input of gated experts only");
+  const float* in_w = weigh_input ? weights : nullptr;
+  const float* out_w = weigh_input ? nullptr : weights;
   HB_REQUIRE(act != HB_ACT_SWISH_CLAMP || gated, "moe_experts: the clamped activation is a gated expert's");
   HB_REQUIRE((long long)n_tokens * top < 2147483647LL && ceil_div(F, MOE_WARPS) <= 65535 && ceil_div(D, MOE_WARPS) <= 65535,
              "moe_experts: too many (token, choice) pairs or channels");
   cudaStream_t s = (cudaStream_t)stream;
   dim3 g1(n_tokens * top, ceil_div(F, MOE_WARPS)), g2(n_tokens, ceil_div(D, MOE_WARPS));
   if (dtype == HB_F32) {
-    hb_launch(moe_up_kernel<float>, g1, dim3(MOE_WARPS * 32), 0, s, (const float*)h, ld, (const float*)up, ids, (float*)mid, D, F, top, act, gated, act_limit);
-    hb_launch(moe_down_kernel<float>, g2, dim3(MOE_WARPS * 32), 0, s, (const float*)mid, (const float*)down, ids, weights, y, ldy, D, F, top, accumulate);
+    hb_launch(moe_up_kernel<float>, g1, dim3(MOE_WARPS * 32), 0, s, (const float*)h, ld, (const float*)up, ids, in_w, (float*)mid, D, F, top, act, gated, act_limit);
+    hb_launch(moe_down_kernel<float>, g2, dim3(MOE_WARPS * 32), 0, s, (const float*)mid, (const float*)down, ids, out_w, y, ldy, D, F, top, accumulate);
   } else {
-    hb_launch(moe_up_kernel<bf16>, g1, dim3(MOE_WARPS * 32), 0, s, (const bf16*)h, ld, (const bf16*)up, ids, (bf16*)mid, D, F, top, act, gated, act_limit);
-    hb_launch(moe_down_kernel<bf16>, g2, dim3(MOE_WARPS * 32), 0, s, (const bf16*)mid, (const bf16*)down, ids, weights, y, ldy, D, F, top, accumulate);
+    hb_launch(moe_up_kernel<bf16>, g1, dim3(MOE_WARPS * 32), 0, s, (const bf16*)h, ld, (const bf16*)up, ids, in_w, (bf16*)mid, D, F, top, act, gated, act_limit);
+    hb_launch(moe_down_kernel<bf16>, g2, dim3(MOE_WARPS * 32), 0, s, (const bf16*)mid, (const bf16*)down, ids, out_w, y, ldy, D, F, top, accumulate);
   }
   HB_CHECK_LAUNCH("moe_experts");
   return 0;
@@ -301,7 +307,7 @@ template <bool UP>
 __global__ void __launch_bounds__(MG_THREADS)
 moe_grouped_gemm_kernel(const bf16* __restrict__ A, int lda, const bf16* __restrict__ W, void* __restrict__ C, int ldc,
                         const int* __restrict__ pair_off, const int* __restrict__ tile_off, const int* __restrict__ list, int E,
-                        int N, int K, int top, int act, int gated, float limit) {
+                        int N, int K, int top, int act, int gated, float limit, const float* __restrict__ in_w) {
   __shared__ __align__(16) bf16 AW[2][(MG_TM + MG_TN) * (MG_TK + 8)];      // per buffer: the A tile, then the W tile
   __shared__ int rows[MG_TM];
   pdl_wait();
@@ -393,6 +399,7 @@ moe_grouped_gemm_kernel(const bf16* __restrict__ A, int lda, const bf16* __restr
       const int pair = rows[wm + m * 16 + g + half * 8];
       if (pair < 0) continue;
       if (UP && gated) {
+        const float iw = in_w ? in_w[pair] : 1.0f;
 #pragma unroll
         for (int nt = 0; nt < 8; nt += 2)
 #pragma unroll
@@ -400,7 +407,7 @@ moe_grouped_gemm_kernel(const bf16* __restrict__ A, int lda, const bf16* __restr
             const int n = n0 + wn + nt * 8 + 2 * t + c;      // a gate column; its up column is n + 8 (N is a multiple of 16)
             if (n >= N) continue;
             ((bf16*)C)[(size_t)pair * ldc + ((n0 + wn + nt * 8) >> 1) + 2 * t + c] =
-                __float2bfloat16_rn(moe_glu(acc[m][nt][half * 2 + c], acc[m][nt + 1][half * 2 + c], act, limit));
+                __float2bfloat16_rn(moe_glu(iw * acc[m][nt][half * 2 + c], iw * acc[m][nt + 1][half * 2 + c], act, limit));
           }
         continue;
       }
@@ -417,7 +424,7 @@ moe_grouped_gemm_kernel(const bf16* __restrict__ A, int lda, const bf16* __restr
     }
 }
 
-// slot: where each pair's row lies in `part` (null: at the pair's own index)
+// slot: where each pair's row lies in `part` (null: at the pair's own index); wts null: weights of 1
 __global__ void moe_combine_kernel(const float* __restrict__ part, const float* __restrict__ wts, float* __restrict__ y, int ldy,
                                    int D, int top, int accumulate, const int* __restrict__ slot) {
   pdl_wait();
@@ -427,7 +434,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ part, const float* 
   float acc = 0.0f;
   for (int r = 0; r < top; ++r) {
     const size_t u = (size_t)t * top + r;
-    acc = fmaf(wts[u], part[(slot ? (size_t)slot[u] : u) * D + d], acc);
+    acc = fmaf(wts ? wts[u] : 1.0f, part[(slot ? (size_t)slot[u] : u) * D + d], acc);
   }
   float* o = y + (size_t)t * ldy + d;
   *o = accumulate ? *o + acc : acc;
@@ -441,7 +448,8 @@ extern "C" long long hb_moe_grouped_scratch_ints(int n_tokens, int E, int top) {
 extern "C" int hb_moe_experts_grouped_bf16(const void* h, int ld, const void* up, const void* down, const int* ids,
                                            const float* weights, int* scratch, void* mid, float* part, float* y, int ldy,
                                            int n_tokens, int D, int E, int F, int top, int act, int gated,
-                                           float act_limit, int accumulate, void* stream) {
+                                           float act_limit, int weigh_input, int accumulate, void* stream) {
+  HB_REQUIRE(!weigh_input || gated, "moe_experts_grouped: the weight multiplies the input of gated experts only");
   HB_REQUIRE(n_tokens > 0 && D > 0 && E > 0 && F > 0 && top > 0, "moe_experts_grouped: sizes must be positive");
   HB_REQUIRE(E <= MG_MAX_EXPERTS, "moe_experts_grouped: at most %d experts", MG_MAX_EXPERTS);
   HB_REQUIRE(D % 8 == 0 && F % 8 == 0 && ld % 8 == 0, "moe_experts_grouped: widths must be multiples of 8");
@@ -457,10 +465,12 @@ extern "C" int hb_moe_experts_grouped_bf16(const void* h, int ld, const void* up
   const int max_tiles = ceil_div(n_pairs, MG_TM) + E;
   const int n_up = gated ? 2 * F : F;      // rows of an expert's first matrix
   hb_launch(moe_grouped_gemm_kernel<true>, dim3(max_tiles, ceil_div(n_up, MG_TN)), dim3(MG_THREADS), 0, s, (const bf16*)h, ld, (const bf16*)up,
-            mid, F, (const int*)pair_off, (const int*)tile_off, (const int*)list, E, n_up, D, top, act, gated, act_limit);
+            mid, F, (const int*)pair_off, (const int*)tile_off, (const int*)list, E, n_up, D, top, act, gated, act_limit,
+            weigh_input ? weights : (const float*)nullptr);
   hb_launch(moe_grouped_gemm_kernel<false>, dim3(max_tiles, ceil_div(D, MG_TN)), dim3(MG_THREADS), 0, s, (const bf16*)mid, F,
-            (const bf16*)down, (void*)part, D, (const int*)pair_off, (const int*)tile_off, (const int*)list, E, D, F, top, act, 0, 0.0f);
-  hb_launch(moe_combine_kernel, dim3(ceil_div(D, 256), n_tokens), dim3(256), 0, s, (const float*)part, weights, y, ldy, D, top, accumulate, (const int*)nullptr);
+            (const bf16*)down, (void*)part, D, (const int*)pair_off, (const int*)tile_off, (const int*)list, E, D, F, top, act, 0, 0.0f, (const float*)nullptr);
+  hb_launch(moe_combine_kernel, dim3(ceil_div(D, 256), n_tokens), dim3(256), 0, s, (const float*)part, weigh_input ? (const float*)nullptr : weights, y, ldy, D, top, accumulate,
+            (const int*)nullptr);
   HB_CHECK_LAUNCH("moe_experts_grouped");
   return 0;
 }
@@ -470,7 +480,8 @@ extern "C" int hb_moe_experts_grouped_bf16(const void* h, int ld, const void* up
 // products on tcgen05.  The pairs are sorted by
 // expert into a buffer in which every expert's run is padded to whole tiles of 128 rows, so that a tile of the
 // tensor-memory product (gemm_tcgen05.cu, grouped mode) belongs to one expert:
-//   sort:     counts per expert, padded offsets, slot[pair] = its row, tile_expert[tile], rows in use
+//   sort:     counts per expert, padded offsets, slot[pair] = its row, tile_expert[tile], rows in use (and, where the
+//             weights multiply the experts' inputs, the weight of every row, by which the product's epilogue multiplies)
 //   gather:   sorted[slot[pair]] = h[pair / top]
 //   product:  mid = silu(gate) * up of sorted x W1_e (the dense feed-forward's fused epilogue)
 //   product:  part = mid x W2_e (float)
@@ -478,7 +489,7 @@ extern "C" int hb_moe_experts_grouped_bf16(const void* h, int ld, const void* up
 // Rows of padding are computed and never read.  A pair's numbers do not depend on its place.
 __global__ void __launch_bounds__(1024)
 moe_sort_padded_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __restrict__ slot, int* __restrict__ tile_expert,
-                       int* __restrict__ rows_used, int max_tiles) {
+                       int* __restrict__ rows_used, int max_tiles, const float* __restrict__ wts, float* __restrict__ row_scale) {
   __shared__ int cnt[MG_MAX_EXPERTS], off[MG_MAX_EXPERTS];
   pdl_wait();
   pdl_launch();
@@ -502,6 +513,7 @@ moe_sort_padded_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __r
   for (int u = threadIdx.x; u < n_pairs; u += blockDim.x) {
     const int e = ids[u];
     slot[u] = off[e] + atomicAdd(&cnt[e], 1);
+    if (row_scale) row_scale[slot[u]] = wts[u];
   }
 }
 
@@ -521,11 +533,12 @@ extern "C" int hb_moe_experts_tc_rows(int n_tokens, int E, int top) {
   return tiles * 128 > 2147483647LL ? -1 : (int)(tiles * 128);
 }
 
-// up [E, 2F, D] with gate and up rows in groups of 8; ints: n_tokens * top + rows / 128 + 1; sorted [rows, D] and
+// up [E, 2F, D] with gate and up rows in groups of 8; row_scale: `rows` floats if the weights multiply the experts' inputs,
+// else null; ints: n_tokens * top + rows / 128 + 1; sorted [rows, D] and
 // mid [rows, F] bfloat16, part [rows, D] floats, with rows = hb_moe_experts_tc_rows(...).
 extern "C" int hb_moe_experts_tc_bf16(const void* h, int ld, const void* up, const void* down, const int* ids,
                                       const float* weights, int* ints, void* sorted, void* mid, float* part, float* y, int ldy,
-                                      int n_tokens, int D, int E, int F, int top, float act_limit, int accumulate,
+                                      int n_tokens, int D, int E, int F, int top, float act_limit, float* row_scale, int accumulate,
                                       int* error_flag, void* stream) {
   HB_REQUIRE(n_tokens > 0 && D > 0 && E > 0 && F > 0 && top > 0, "moe_experts_tc: sizes must be positive");
   HB_REQUIRE(E <= MG_MAX_EXPERTS, "moe_experts_tc: at most %d experts", MG_MAX_EXPERTS);
@@ -538,18 +551,19 @@ extern "C" int hb_moe_experts_tc_bf16(const void* h, int ld, const void* up, con
   int* tile_expert = ints + n_pairs;
   int* rows_used = tile_expert + max_tiles;
   cudaStream_t s = (cudaStream_t)stream;
-  hb_launch(moe_sort_padded_kernel, dim3(1), dim3(1024), 0, s, ids, n_pairs, E, slot, tile_expert, rows_used, max_tiles);
+  hb_launch(moe_sort_padded_kernel, dim3(1), dim3(1024), 0, s, ids, n_pairs, E, slot, tile_expert, rows_used, max_tiles, weights,
+            row_scale);
   hb_launch(moe_gather_rows_kernel, dim3(n_pairs), dim3(D / 8 >= 128 ? 128 : 64), 0, s, (const bf16*)h, ld, (const int*)slot,
             (bf16*)sorted, D / 8, top);
   HB_CHECK_LAUNCH("moe_experts_tc (sort, gather)");
-  int rc = hb_gemm_tcgen05_grouped_bf16(sorted, D, up, D, mid, F, rows, 2 * F, D, E, HB_EPI_SWIGLU, act_limit, rows_used,
+  int rc = hb_gemm_tcgen05_grouped_bf16(sorted, D, up, D, mid, F, rows, 2 * F, D, E, HB_EPI_SWIGLU, act_limit, row_scale, rows_used,
                                         tile_expert, error_flag, stream);
   if (rc) return rc;
-  rc = hb_gemm_tcgen05_grouped_bf16(mid, F, down, F, part, D, rows, D, F, E, HB_EPI_STORE_F32, 0.0f, rows_used, tile_expert,
+  rc = hb_gemm_tcgen05_grouped_bf16(mid, F, down, F, part, D, rows, D, F, E, HB_EPI_STORE_F32, 0.0f, nullptr, rows_used, tile_expert,
                                     error_flag, stream);
   if (rc) return rc;
-  hb_launch(moe_combine_kernel, dim3(ceil_div(D, 256), n_tokens), dim3(256), 0, s, (const float*)part, weights, y, ldy, D, top,
-            accumulate, (const int*)slot);
+  hb_launch(moe_combine_kernel, dim3(ceil_div(D, 256), n_tokens), dim3(256), 0, s, (const float*)part, row_scale ? (const float*)nullptr : weights, y, ldy,
+            D, top, accumulate, (const int*)slot);
   HB_CHECK_LAUNCH("moe_experts_tc (combine)");
   return 0;
 }

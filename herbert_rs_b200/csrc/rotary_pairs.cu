@@ -1,9 +1,12 @@
 // What lies between the q/k/v product and attention for a mixer that norms q and k over the whole projection,
 // rotates pairs by angles taken from the position, and keeps its values rotated too:
 //
-//   q <- q / sqrt(mean_all(q^2) + eps) * wq     over all heads of the row at once (likewise k; optional)
+//   q <- q / sqrt(mean(q^2) + eps) * wq         over all heads of the row at once, or over each head's channels with one
+//                                               weight for all heads (likewise k; optional)
 //   pair m of the first `rot` channels of every q and k head turns by  p * fqk[m]
 //   pair m of all dv channels of every v head turns by                p * fv[m]      (optional)
+//   v <- (1 - lambda) v + lambda v'              v': a row of values that another layer of the step left as floats (optional);
+//                                               a layer can leave its own rows (with their bias) for others
 //   cos and sin of q's and k's angles are multiplied by one constant (scaled frequencies); a bias vector may be added
 //   to the row before anything else
 //   (u, v) -> (u cos a - v sin a, v cos a + u sin a);  pair m is (2m, 2m + 1) ("interleaved") or (m, m + n/2) ("halves")
@@ -28,13 +31,15 @@
 struct RotPrepArgs {
   const float* rows; int ld;
   const float* bias;               // in the rows' layout, added first; null: none
-  const float* wq; const float* wk; float eps; int whole_norm;
+  const float* wq; const float* wk; float eps; int norm;      // norm: 0 none, 1 over the whole projection, 2 per head
   const float* fqk; int rot; int halves; float mscale;
   const float* fv;                 // null: values are stored as they are
   const int* tok_seq; const int* tok_pos; const int* seq_pages; int pages_stride;
   void* q_out; int ldq;
   void* kcache; void* vcache;
   int nh, nkv, maps, dk, dv, hd, page_size, write_cache;
+  const float* blend; float lambda;      // [tokens][nkv * dv]: v <- (1 - lambda) v + lambda blend; null: as they are
+  float* keep;                           // [tokens][nkv * dv]: receives v (with its bias, before any blending); or null
 };
 
 // own * cos + (-/+ partner) * sin for channel j of a head whose first `rot` channels are rotated; cs holds the
@@ -102,6 +107,16 @@ template <> __device__ __forceinline__ void rot_store4<bf16>(bf16* p, float4 v) 
   *reinterpret_cast<uint2*>(p) = u;
 }
 
+// One warp: 1 / rms of a head's n numbers (plus a bias).
+__device__ __forceinline__ float head_inv_rms(const float* head, const float* bias, int n, float eps) {
+  float s = 0.0f;
+  for (int i = threadIdx.x & 31; i < n; i += 32) {
+    const float x = head[i] + (bias ? bias[i] : 0.0f);
+    s = fmaf(x, x, s);
+  }
+  return 1.0f / sqrtf(warp_sum(s) / (float)n + eps);
+}
+
 // V4: four channels a lane (see turn_channels4).
 template <typename T, bool V4>
 __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
@@ -134,7 +149,7 @@ __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
   const float* bk = a.bias ? a.bias + qn : nullptr;
   const float* bv = a.bias ? a.bias + qn + kn : nullptr;
   float inv_q = 1.0f, inv_k = 1.0f;
-  if (a.whole_norm) {
+  if (a.norm == 1) {
     float sq = 0.0f, sk = 0.0f;
     for (int i = threadIdx.x; i < qn; i += blockDim.x) {
       const float x = q[i] + (bq ? bq[i] : 0.0f);
@@ -154,7 +169,8 @@ __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
   for (int h = warp; h < a.nh * a.maps; h += nwarp) {      // a warp per head: nothing is divided channel by channel
     const size_t at = (size_t)h * a.dk;
     const float* hb = bq ? bq + at : nullptr;
-    const float* hw = a.wq ? a.wq + at : nullptr;
+    const float* hw = a.norm == 2 ? a.wq : a.wq ? a.wq + at : nullptr;
+    if (a.norm == 2) inv_q = head_inv_rms(q + at, hb, a.dk, a.eps);
     const int off = (h % a.maps) * a.dk;
     T* qo = (T*)a.q_out + (size_t)t * a.ldq + (size_t)h * a.hd;
     if constexpr (V4) {
@@ -184,10 +200,19 @@ __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
       T* vo = (T*)a.vcache + at;
       const float* hv = v + (size_t)g * a.dv;
       const float* hb = bv ? bv + (size_t)g * a.dv : nullptr;
+      const size_t vrow = ((size_t)t * a.nkv + g) * a.dv;
       if constexpr (V4) {
         for (int j = lane * 4; j < a.hd; j += 128) {
           float4 r = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-          if (j < a.dv) r = turn_channels4(hv, hb, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, tab_v);
+          if (j < a.dv) {
+            r = turn_channels4(hv, hb, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, tab_v);
+            if (a.keep) *reinterpret_cast<float4*>(a.keep + vrow + j) = r;
+            if (a.blend) {
+              const float4 f = *reinterpret_cast<const float4*>(a.blend + vrow + j);
+              const float k = 1.0f - a.lambda;
+              r = make_float4(k * r.x + a.lambda * f.x, k * r.y + a.lambda * f.y, k * r.z + a.lambda * f.z, k * r.w + a.lambda * f.w);
+            }
+          }
           rot_store4<T>(vo + j, r);
         }
         continue;
@@ -195,12 +220,17 @@ __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
 #pragma unroll 4
       for (int j = lane; j < a.hd; j += 32) {
         float r = 0.0f;
-        if (j < a.dv) r = turn_channel(hv, hb, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, tab_v);
+        if (j < a.dv) {
+          r = turn_channel(hv, hb, nullptr, 1.0f, j, a.fv ? a.dv : 0, a.halves, tab_v);
+          if (a.keep) a.keep[vrow + j] = r;
+          if (a.blend) r = (1.0f - a.lambda) * r + a.lambda * a.blend[vrow + j];
+        }
         vo[j] = from_f32<T>(r);
       }
       continue;
     }
     T* ko = (T*)a.kcache + at;
+    if (a.norm == 2) inv_k = head_inv_rms(k + (size_t)g * a.dk, bk ? bk + (size_t)g * a.dk : nullptr, a.dk, a.eps);
     int m = 0, first = 0;                                   // the map that channel j belongs to
     if constexpr (V4) {
       for (int j = lane * 4; j < a.hd; j += 128) {
@@ -208,7 +238,7 @@ __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
         const size_t head = (size_t)(g * a.maps + m) * a.dk;
         float4 r = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (m < a.maps)
-          r = turn_channels4(k + head, bk ? bk + head : nullptr, a.wk ? a.wk + head : nullptr, inv_k, j - first, a.rot, a.halves, tab);
+          r = turn_channels4(k + head, bk ? bk + head : nullptr, a.wk ? a.wk + (a.norm == 2 ? 0 : head) : nullptr, inv_k, j - first, a.rot, a.halves, tab);
         rot_store4<T>(ko + j, r);
       }
       continue;
@@ -217,29 +247,32 @@ __global__ void __launch_bounds__(256) qkv_rotary_cache_kernel(RotPrepArgs a) {
       float r = 0.0f;
       while (m < a.maps && j - first >= a.dk) { ++m; first += a.dk; }
       const size_t head = (size_t)(g * a.maps + m) * a.dk;
-      if (m < a.maps) r = turn_channel(k + head, bk ? bk + head : nullptr, a.wk ? a.wk + head : nullptr, inv_k, j - first, a.rot, a.halves, tab);
+      if (m < a.maps) r = turn_channel(k + head, bk ? bk + head : nullptr, a.wk ? a.wk + (a.norm == 2 ? 0 : head) : nullptr, inv_k, j - first, a.rot, a.halves, tab);
       ko[j] = from_f32<T>(r);
     }
   }
 }
 
 extern "C" int hb_qkv_rotary_cache(int dtype, const float* rows, int ld, const float* bias, const float* wq, const float* wk, float eps,
-                                   int whole_norm, const float* fqk, int rot, int halves, float mscale, const float* fv, const int* tok_seq,
+                                   int norm, const float* fqk, int rot, int halves, float mscale, const float* fv, const int* tok_seq,
                                    const int* tok_pos, const int* seq_pages, int pages_stride, void* q_out, int ldq, void* kcache,
                                    void* vcache, int n_tokens, int nh, int nkv, int maps, int dk, int dv, int hd, int page_size,
-                                   int write_cache, void* stream) {
+                                   int write_cache, const float* blend, float lambda, float* keep, void* stream) {
   HB_REQUIRE(n_tokens > 0 && nh > 0 && nkv > 0 && maps > 0 && dk > 0 && dv > 0 && page_size > 0, "qkv_rotary_cache: sizes must be positive");
   HB_REQUIRE(hd >= maps * dk && hd >= dv, "qkv_rotary_cache: cache heads of %d channels cannot hold keys of %d x %d and values of %d", hd, maps, dk, dv);
   HB_REQUIRE(rot >= 0 && rot <= dk && rot % 2 == 0, "qkv_rotary_cache: %d rotated channels must be even and at most %d", rot, dk);
+  HB_REQUIRE(norm >= 0 && norm <= 2 && (norm == 0 || (wq != nullptr && wk != nullptr)), "qkv_rotary_cache: a norm needs both its weights");
+  HB_REQUIRE(norm != 2 || maps == 1, "qkv_rotary_cache: a norm per head serves one map per head");
+  HB_REQUIRE((blend == nullptr && keep == nullptr) || (fv == nullptr && write_cache), "qkv_rotary_cache: values that are blended or kept are stored and not rotated");
   HB_REQUIRE(rot == 0 || fqk != nullptr, "qkv_rotary_cache: rotated channels need their frequencies");
   HB_REQUIRE(fv == nullptr || dv % 2 == 0, "qkv_rotary_cache: rotated values need an even size, got %d", dv);
   // a step that stores nothing (it reads another layer's keys and values) brings rows of queries only
   HB_REQUIRE(ld >= nh * maps * dk + (write_cache ? nkv * (maps * dk + dv) : 0) && ldq >= nh * maps * hd, "qkv_rotary_cache: rows are shorter than their heads");
   const size_t smem = (size_t)(rot + (fv ? dv : 0)) * sizeof(float);
   HB_REQUIRE(smem <= 48 * 1024, "qkv_rotary_cache: %d rotated channels exceed a block's shared memory", rot);
-  RotPrepArgs a{rows, ld, bias, wq, wk, eps, whole_norm, fqk, rot, halves, mscale, fv, tok_seq, tok_pos, seq_pages, pages_stride, q_out, ldq,
-                kcache, vcache, nh, nkv, maps, dk, dv, hd, page_size, write_cache};
-  const uintptr_t in_ptrs = (uintptr_t)rows | (uintptr_t)bias | (uintptr_t)wq | (uintptr_t)wk;
+  RotPrepArgs a{rows, ld, bias, wq, wk, eps, norm, fqk, rot, halves, mscale, fv, tok_seq, tok_pos, seq_pages, pages_stride, q_out, ldq,
+                kcache, vcache, nh, nkv, maps, dk, dv, hd, page_size, write_cache, blend, lambda, keep};
+  const uintptr_t in_ptrs = (uintptr_t)rows | (uintptr_t)bias | (uintptr_t)wq | (uintptr_t)wk | (uintptr_t)blend | (uintptr_t)keep;
   const uintptr_t out_ptrs = (uintptr_t)q_out | (uintptr_t)kcache | (uintptr_t)vcache;
   const bool v4 = ((dk | dv | hd | ld | ldq) & 3) == 0 && (in_ptrs & 15) == 0 && (out_ptrs & 15) == 0 && rot % (halves ? 8 : 4) == 0 &&
                   (fv == nullptr || dv % (halves ? 8 : 4) == 0);

@@ -4,6 +4,9 @@
 //   dt_t = softplus(raw_t + dt_bias),   a_t = exp(-exp(A_log) dt_t)
 //   S_t  = a_t S_{t-1} + dt_t B_t x_t^T,     y_t = S_t^T C_t + D x_t
 //
+// A mixer that makes its decays and weights itself (the gates of a matrix memory) brings them: log a_t as `logd`, the
+// weight of B x^T in dt_t's place, no D.
+//
 // x, B and C arrive in the activation type as columns of one row per token (what a short convolution leaves), the raw
 // step sizes as floats; step sizes, decays, state and sums are float.  The state of a sequence is its slot of the
 // cache's state region ([slots][H][N][dv]): a step continues from it, whatever a prompt was cut into.
@@ -25,14 +28,16 @@
 
 struct SsdArgs {
   const void* xbc; int ld, b_off, c_off;      // row t: x at 0 [H][dv], B at b_off [G][N], C at c_off [G][N]
-  const float* dt; int lddt;                  // raw step sizes [tokens][H]
-  const float* dt_bias; const float* a_log; const float* dskip;      // [H] each
+  const float* dt; int lddt;                  // raw step sizes [tokens][H]; with logd: the weights as they are
+  const float* logd;                          // log decays [tokens][H] with dt's row stride, <= 0; null: from the step sizes
+  const float* dt_bias; const float* a_log; const float* dskip;      // [H] each; null with logd
   float* state;                               // [slots][H][N][dv]
   const int* seq_slot; const int* seq_start;
   float* out; int ldo;                        // [tokens][H][dv]
   int H, G, N, dv;
   int cb;                                     // token by token: value channels per CTA (a power of two, at least 4)
   float* chunk_state; float* chunk_decay;     // chunked: [chunk][H][N][dv], [chunk][H]
+  int vw;                                     // chunked: value channels per CTA, at most the kernel's DVM
 };
 
 __device__ __forceinline__ float ssd_softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
@@ -76,7 +81,8 @@ __global__ void __launch_bounds__(SS_THREADS) ssd_scan_kernel(SsdArgs a) {
     }
   }
   for (int i = tid; i < SS_CHUNK * (2 * NP + a.cb); i += SS_THREADS) sh[i] = 0.0f;      // rows past N stay zero
-  const float neg_a = -expf(a.a_log[h]), bias = a.dt_bias[h], dskip = a.dskip[h];
+  const bool given = a.logd != nullptr;
+  const float neg_a = given ? 0.0f : -expf(a.a_log[h]), bias = given ? 0.0f : a.dt_bias[h], dskip = given ? 0.0f : a.dskip[h];
   for (int c0 = t0; c0 < t1; c0 += SS_CHUNK) {
     const int n = t1 - c0 < SS_CHUNK ? t1 - c0 : SS_CHUNK;
     __syncthreads();
@@ -92,8 +98,9 @@ __global__ void __launch_bounds__(SS_THREADS) ssd_scan_kernel(SsdArgs a) {
       if (col0 + c < a.dv) xs[i] = to_f32(base[(size_t)tt * a.ld + (size_t)h * a.dv + col0 + c]);
     }
     if (tid < n) {
-      const float dt = ssd_softplus(a.dt[(size_t)(c0 + tid) * a.lddt + h] + bias);
-      coef[2 * tid] = expf(neg_a * dt);
+      const size_t at = (size_t)(c0 + tid) * a.lddt + h;
+      const float dt = given ? a.dt[at] : ssd_softplus(a.dt[at] + bias);
+      coef[2 * tid] = expf(given ? a.logd[at] : neg_a * dt);
       coef[2 * tid + 1] = dt;
     }
     __syncthreads();
@@ -150,10 +157,12 @@ static int ssd_sms() {
   HB_REQUIRE(n_seqs > 0 && heads > 0 && groups > 0 && N > 0 && dv > 0, name ": sizes must be positive");                       \
   HB_REQUIRE(heads % groups == 0, name ": %d heads are not a multiple of %d groups", heads, groups);                           \
   HB_REQUIRE(n_seqs <= 65535 && heads <= 65535, name ": too many sequences or heads");                                         \
+  HB_REQUIRE(logd != nullptr || (dt_bias != nullptr && a_log != nullptr && dskip != nullptr),                                  \
+             name ": needs log decays, or the step sizes' bias, the decay rates and D");                                       \
   HB_REQUIRE(((uintptr_t)state & 15) == 0, name ": the state must be 16-byte aligned")
 
 extern "C" int hb_ssd_scan(int dtype, const void* xbc, int ld, int b_off, int c_off, const float* dt, int lddt,
-                           const float* dt_bias, const float* a_log, const float* dskip, float* state, const int* seq_slot,
+                           const float* logd, const float* dt_bias, const float* a_log, const float* dskip, float* state, const int* seq_slot,
                            const int* seq_start, float* out, int ldo, int n_seqs, int heads, int groups, int N, int dv,
                            void* stream) {
   SS_CHECKS("ssd_scan");
@@ -167,8 +176,8 @@ extern "C" int hb_ssd_scan(int dtype, const void* xbc, int ld, int b_off, int c_
   const int rpt = need <= 1 ? 1 : need <= 2 ? 2 : need <= 4 ? 4 : need <= 8 ? 8 : 16;
   const size_t smem = (size_t)(SS_CHUNK * (2 * rgs * rpt + cb) + SS_CHUNK * SS_THREADS * 4 + 2 * SS_CHUNK) * sizeof(float);
   HB_REQUIRE(smem <= 220 * 1024 && ceil_div(dv, cb) <= 65535, "ssd_scan: %d state rows or %d value channels are too many", N, dv);
-  const SsdArgs a{xbc, ld, b_off, c_off, dt, lddt, dt_bias, a_log, dskip, state, seq_slot, seq_start, out, ldo, heads, groups, N, dv,
-                  cb, nullptr, nullptr};
+  const SsdArgs a{xbc, ld, b_off, c_off, dt, lddt, logd, dt_bias, a_log, dskip, state, seq_slot, seq_start, out, ldo, heads, groups, N, dv,
+                  cb, nullptr, nullptr, 0};
   const dim3 grid(n_seqs, heads, ceil_div(dv, cb));
   cudaStream_t s = (cudaStream_t)stream;
 #define SS_GO(T, RPT)                                                                                                          \
@@ -201,16 +210,16 @@ __device__ __forceinline__ int ssd_chunk_index(const SsdArgs& a, int b, int c) {
 struct SsdTile {      // what a CTA of the chunked kernels works on
   int c, b, grp, h0, nh, v0, cols, tok0, n;
 };
-__device__ __forceinline__ bool ssd_tile(const SsdArgs& a, int vblocks, int hpc, int dvm, SsdTile& w) {
+__device__ __forceinline__ bool ssd_tile(const SsdArgs& a, int vblocks, int hpc, SsdTile& w) {
   const int per = a.H / a.G, parts = (per + hpc - 1) / hpc;
   int y = blockIdx.y;
   w.c = blockIdx.x; w.b = blockIdx.z;
-  w.v0 = (y % vblocks) * dvm; y /= vblocks;
+  w.v0 = (y % vblocks) * a.vw; y /= vblocks;
   w.grp = y / parts;
   const int part = y % parts;
   w.h0 = w.grp * per + part * hpc;
   w.nh = per - part * hpc < hpc ? per - part * hpc : hpc;
-  w.cols = a.dv - w.v0 < dvm ? a.dv - w.v0 : dvm;
+  w.cols = a.dv - w.v0 < a.vw ? a.dv - w.v0 : a.vw;
   const int t0 = a.seq_start[w.b], len = a.seq_start[w.b + 1] - t0;
   w.tok0 = t0 + w.c * SC_Q;
   w.n = len - w.c * SC_Q < SC_Q ? len - w.c * SC_Q : SC_Q;
@@ -221,11 +230,20 @@ __device__ __forceinline__ bool ssd_tile(const SsdArgs& a, int vblocks, int hpc,
 // decay 1.
 __device__ __forceinline__ void ssd_prepare(const SsdArgs& a, int h, int tok0, int n, float* dts, float* cum) {
   const int lane = threadIdx.x & 31;
-  const float neg_a = -expf(a.a_log[h]) * 1.4426950408889634f, bias = a.dt_bias[h];
-  float d0 = 0.0f, d1 = 0.0f;
-  if (2 * lane < n) d0 = ssd_softplus(a.dt[(size_t)(tok0 + 2 * lane) * a.lddt + h] + bias);
-  if (2 * lane + 1 < n) d1 = ssd_softplus(a.dt[(size_t)(tok0 + 2 * lane + 1) * a.lddt + h] + bias);
-  const float l0 = neg_a * d0, l1 = neg_a * d1;
+  constexpr float LOG2E = 1.4426950408889634f;
+  const size_t at = (size_t)(tok0 + 2 * lane) * a.lddt + h;
+  const bool live0 = 2 * lane < n, live1 = 2 * lane + 1 < n;
+  float d0 = 0.0f, d1 = 0.0f, l0 = 0.0f, l1 = 0.0f;
+  if (a.logd != nullptr) {
+    if (live0) { d0 = a.dt[at]; l0 = a.logd[at] * LOG2E; }
+    if (live1) { d1 = a.dt[at + a.lddt]; l1 = a.logd[at + a.lddt] * LOG2E; }
+  } else {
+    const float neg_a = -expf(a.a_log[h]) * LOG2E, bias = a.dt_bias[h];
+    if (live0) d0 = ssd_softplus(a.dt[at] + bias);
+    if (live1) d1 = ssd_softplus(a.dt[at + a.lddt] + bias);
+    l0 = neg_a * d0;
+    l1 = neg_a * d1;
+  }
   float run = l0 + l1;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
@@ -279,7 +297,7 @@ __global__ void __launch_bounds__(SC_T) ssd_chunk_state_kernel(SsdArgs a, int vb
   pdl_wait();
   pdl_launch();
   SsdTile w;
-  if (!ssd_tile(a, vblocks, hpc, DVM, w)) return;
+  if (!ssd_tile(a, vblocks, hpc, w)) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const bf16* rows = (const bf16*)a.xbc + (size_t)w.tok0 * a.ld;
   ssd_load_rows(Bs, BS, rows + a.b_off + (size_t)w.grp * a.N, a.ld, w.n, a.N, NP, vec);
@@ -444,7 +462,7 @@ __global__ void __launch_bounds__(SC_T) ssd_chunk_out_kernel(SsdArgs a, int vblo
   pdl_wait();
   pdl_launch();
   SsdTile w;
-  if (!ssd_tile(a, vblocks, hpc, DVM, w)) return;
+  if (!ssd_tile(a, vblocks, hpc, w)) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const bf16* rows = (const bf16*)a.xbc + (size_t)w.tok0 * a.ld;
   const size_t ci = ssd_chunk_index(a, w.b, w.c);
@@ -575,7 +593,7 @@ __global__ void __launch_bounds__(SC_T) ssd_chunk_out_kernel(SsdArgs a, int vblo
           mma16816(acc[2 * nd + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
         }
       }
-      const float dskip = a.dskip[h];
+      const float dskip = a.dskip != nullptr ? a.dskip[h] : 0.0f;
 #pragma unroll
       for (int nd = 0; nd < HALF / 8; ++nd)
 #pragma unroll
@@ -605,8 +623,8 @@ extern "C" int hb_ssd_chunks(int n_tokens, int n_seqs, int N, int dv) {
 }
 
 // chunk_state [hb_ssd_chunks(..)][heads][N][dv], chunk_decay [hb_ssd_chunks(..)][heads]: scratch.
-extern "C" int hb_ssd_chunked_bf16(const void* xbc, int ld, int b_off, int c_off, const float* dt, int lddt, const float* dt_bias,
-                                   const float* a_log, const float* dskip, float* state, const int* seq_slot,
+extern "C" int hb_ssd_chunked_bf16(const void* xbc, int ld, int b_off, int c_off, const float* dt, int lddt, const float* logd,
+                                   const float* dt_bias, const float* a_log, const float* dskip, float* state, const int* seq_slot,
                                    const int* seq_start, float* out, int ldo, int n_seqs, int max_q_len, int heads, int groups,
                                    int N, int dv, float* chunk_state, float* chunk_decay, void* stream) {
   SS_CHECKS("ssd_chunked");
@@ -614,9 +632,10 @@ extern "C" int hb_ssd_chunked_bf16(const void* xbc, int ld, int b_off, int c_off
              "ssd_chunked: needs tokens and scratch (16-byte aligned)");
   HB_REQUIRE(N <= 256, "ssd_chunked: %d state rows per head exceed the supported maximum 256", N);
   HB_REQUIRE(((uintptr_t)out & 7) == 0, "ssd_chunked: the output must be 8-byte aligned");
-  const SsdArgs a{xbc, ld, b_off, c_off, dt, lddt, dt_bias, a_log, dskip, state, seq_slot, seq_start, out, ldo, heads, groups, N, dv,
-                  0, chunk_state, chunk_decay};
   const int dvm = dv <= 32 ? 32 : dv <= 64 ? 64 : 128, vb = ceil_div(dv, dvm), chunks = ceil_div(max_q_len, SC_Q);
+  const int vw = ceil_div(ceil_div(dv, vb), 16) * 16;      // the blocks of value channels are of one width, or nearly
+  const SsdArgs a{xbc, ld, b_off, c_off, dt, lddt, logd, dt_bias, a_log, dskip, state, seq_slot, seq_start, out, ldo, heads, groups, N, dv,
+                  0, chunk_state, chunk_decay, vw};
   const int vec = ld % 8 == 0 && b_off % 8 == 0 && c_off % 8 == 0 && N % 8 == 0 && dv % 8 == 0 && ((uintptr_t)xbc & 15) == 0;
   // heads of a group per CTA: as many as still leave every SM a CTA or two
   const int per = heads / groups;

@@ -96,6 +96,7 @@ class StepBatch:
         self.host: Optional[np.ndarray] = None
         self.dev: Optional[torch.Tensor] = None
         self.pages: List[torch.Tensor] = []
+        self.kept: dict = {}             # what a layer of the step leaves for later layers of the same step, by name
 
     def fill_host(self, buf: np.ndarray, page_rows: Sequence[np.ndarray], uniforms: Optional[np.ndarray] = None) -> None:
         """Write every array into `buf` (int32, at least layout.total long)."""

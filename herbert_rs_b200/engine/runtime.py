@@ -59,8 +59,14 @@ class Workspace:
         if lane != 0:
             self.current.offset = 0
 
+    def take_for_step(self, shape, dtype: torch.dtype) -> torch.Tensor:
+        """Scratch that lives until the step ends, whichever lane is current: what a layer leaves for a later one."""
+        return self._take(self.lanes[0], shape, dtype)
+
     def take(self, shape, dtype: torch.dtype) -> torch.Tensor:
-        lane = self.current
+        return self._take(self.current, shape, dtype)
+
+    def _take(self, lane: _Lane, shape, dtype: torch.dtype) -> torch.Tensor:
         shape = tuple(shape)
         n = 1
         for s in shape:

@@ -2,6 +2,7 @@
 
 from ..config.begupel import BegupelConfig
 from ..config.kebisun import KebisunConfig
+from ..config.muzasun import MuzasunConfig
 from ..config.nefivik import NefivikConfig
 from ..config.putazen import PutazenConfig
 from ..config.qwen3 import Qwen3Config
@@ -28,5 +29,9 @@ register_architecture("Nefivik", NefivikConfig)
 # A residual of several mixed copies; layers of differential attention, latent attention and a Mamba-2 state-space mixer,
 # a run of them several times with the same weights; clamped dense feed-forwards, layer norms with biases.
 register_architecture("Putazen", PutazenConfig)
+# Parallel blocks whose two sublayers read norms without statistics of the same stream; layers of a matrix memory with
+# exponential gates, of the delta rule with a decay per key channel, or of attention whose values are blended with the
+# first such layer's; routed experts whose weights multiply their inputs.
+register_architecture("Muzasun", MuzasunConfig)
 
 __all__ = ["DecoderModel"]

@@ -12,7 +12,7 @@ earlier step instead of storing its own.
 
 Options of the spec: a scaled embedding, a learned vector per position, a second table chosen by (previous
 token, token) whose previous token is kept per sequence in the cache's fixed-size region (the first schedule
-step's entry carries it under the name "embedding.last_id"), a tanh cap on the logits, a second table by token id
+step's entry carries it under the name "embedding.last_id"), a factor and a tanh cap on the logits, a second table by token id
 of which blocks read their own columns (`ModelSpec.token_side_table`), a residual of several copies of the stream
 (`ModelSpec.streams`): equal at the start, mixed by the blocks, summed before the final norm.
 """
@@ -47,6 +47,7 @@ class DecoderModel:
         self.pair_table = None          # [buckets + 1, hidden], if the spec has a pair embedding
         self.token_side_table = None    # [vocab, columns], if blocks add a second input chosen by the token
         self.streams = spec.streams
+        self.scale_logits = False       # the final norm cannot carry the factor on the logits
         for i, b in enumerate(self.blocks):
             if b.streams != self.streams:
                 raise ConfigError(f"layer {i} works on {b.streams or 'one'} copies of the stream, the model on {self.streams or 'one'}")
@@ -85,8 +86,8 @@ class DecoderModel:
         return self.spec.final_norm_name.rsplit(".", 1)[0] + "."
 
     def ignored_names(self) -> set:
-        """Tensors a file may hold without being used (a tied model's stored head)."""
-        return {self.spec.head_name} if self.spec.tie_word_embeddings else set()
+        """Tensors a file may hold without being used (a tied model's stored head, what the spec names)."""
+        return ({self.spec.head_name} if self.spec.tie_word_embeddings else set()) | set(self.spec.unused_names)
 
     def load_embedding(self, t: torch.Tensor) -> None:
         self.embed = t.contiguous()
@@ -116,6 +117,8 @@ class DecoderModel:
 
     def load_final_norm(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.final_norm.load(tensors)
+        # a factor on the logits is a factor on what the head reads, where the norm can carry it
+        self.scale_logits = self.spec.logit_scale != 1.0 and not self.final_norm.scale_result(self.spec.logit_scale)
 
     def weight_bytes(self, rows: int = 0) -> int:
         """Bytes of weights one step reads: every scheduled block, the final norm, the head;
@@ -165,7 +168,7 @@ class DecoderModel:
                 pending = None
                 continue
             nxt = self.blocks[sched[i + 1].layer] if i + 1 < len(sched) else None
-            nxt_norm = nxt.first_norm() if nxt is not None and nxt.chains_norms else None
+            nxt_norm = nxt.first_norm() if nxt is not None and nxt.chains_norms and nxt.chain_kind == block.chain_kind else None
             pending = block.forward(x, batch, cache.view(i), normed=pending,
                                     next_norm=nxt_norm.shareable() if nxt_norm is not None else None)
         ws.use(0)
@@ -178,6 +181,8 @@ class DecoderModel:
             ops.streams_join(x, norm=self.final_norm.as_stream_norm(), h=hn, rows=batch.want_rows)
         logits = ws.take((batch.n_want, self.spec.vocab_size), torch.float32)
         ops.gemm(hn, self.head, logits, ops.EPI_STORE_F32)
+        if self.scale_logits:
+            ops.axpby(logits, self.spec.logit_scale, logits, 0.0)
         if self.spec.logit_softcap:
             ops.tanh_cap(logits, self.spec.logit_softcap)
         return logits

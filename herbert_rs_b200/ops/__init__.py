@@ -86,10 +86,12 @@ _SIGS = {
     "hb_latent_attention": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "hb_moe_experts_grouped_bf16": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
+                                    c_void_p],
     "hb_moe_experts_tc_rows": [c_int, c_int, c_int],
-    "hb_moe_experts_tc_bf16": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                               c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p],
+    "hb_moe_experts_tc_bf16": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                               c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p,
+                               c_void_p],
     "hb_latent_attention_mma_ok": [c_int, c_int],
     "hb_latent_attention_mma_bf16": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                      c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
@@ -101,7 +103,7 @@ _SIGS = {
     "hb_moe_route": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                      c_int, c_int, c_float, c_void_p],
     "hb_moe_experts": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                       c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+                       c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
     "hb_group_rmsnorm": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     "hb_group_rmsnorm_residual": [c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
                                   c_int, c_int, c_int, c_float, c_void_p],
@@ -117,20 +119,21 @@ _SIGS = {
                          c_void_p, c_void_p, c_int, c_int, c_void_p],
     "hb_linear_scan": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "hb_gated_rmsnorm": [c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
-                         c_int, c_int, c_int, c_void_p],
-    "hb_qkv_rotary_cache": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_float,
-                            c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "hb_gated_rmsnorm": [c_int, c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
+                         c_int, c_int, c_int, c_int, c_void_p, c_float, c_float, c_void_p],
+    "hb_qkv_rotary_cache": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int,
+                            c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
+                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p],
     "hb_difference_heads": [c_int, c_void_p, c_int, c_int, c_float, c_float, c_float, c_void_p, c_int, c_int, c_int, c_int,
                             c_void_p],
     "hb_streams_join": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int,
                         c_void_p, c_void_p, c_int, c_int, c_void_p],
     "hb_ssd_scan": [c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                    c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                    c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "hb_ssd_chunks": [c_int, c_int, c_int, c_int],
-    "hb_ssd_chunked_bf16": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                            c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    "hb_ssd_chunked_bf16": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                            c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                            c_void_p, c_void_p],
     "hb_rotate_heads_back": [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                              c_void_p],
     "hb_head_gate": [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -141,6 +144,14 @@ _SIGS = {
     "hb_gated_norm_residual": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
                                c_float, c_void_p, c_int, c_int, c_void_p],
     "hb_token_gate": [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "hb_channel_delta_prepare": [c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
+                                 c_void_p, c_float, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                 c_int, c_void_p],
+    "hb_matrix_memory_prepare": [c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
+                                 c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                 c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "hb_residual_tanh": [c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
+                         c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
 }
 _fns: dict = {}
 
@@ -638,35 +649,54 @@ def linear_scan(q, k, v, state, batch, out, heads, qk_heads, dk, dv, gates=None,
          out.data_ptr(), out.stride(0), batch.n_seqs, batch.max_q_len, int(heads), int(qk_heads), int(dk), int(dv), _stream())
 
 
-def gated_rmsnorm(o, w, eps, gate, out, units, n, sigmoid_gate=False, gate_first=False) -> None:
+def gated_rmsnorm(o, w, eps, gate, out, units, n, sigmoid_gate=False, gate_first=False, unit_stride=None, divide=None) -> None:
     """out[t, u, :] = o[t, u, :] / sqrt(mean(o[t, u, :]^2) + eps) * w * act(gate[t, u, :]) for `units` runs of n columns;
     w [n] is shared by the units (units == 1: one norm over the whole row), or w [units * n] has a part for each.
-    act: silu, or the sigmoid.  With `gate_first` the gate multiplies o before the norm: v = o * act(gate), v / rms(v) * w."""
+    act: silu, or the sigmoid.  With `gate_first` the gate multiplies o before the norm: v = o * act(gate), v / rms(v) * w.
+    Units lie `unit_stride` columns apart in o (None: n).  `divide` = (floor [T, units] float, scale, eps): before anything else
+    a unit's numbers become scale * o / (max(|scale * z|, floor) + eps), z the column of o behind the unit's n."""
     _check(o, torch.float32, "o"); _check(w, torch.float32, "w"); _check(gate, torch.float32, "gate"); _check(out, None, "out")
     if w.numel() not in (n, units * n):
         raise BackendError(f"gated_rmsnorm: the weight has {w.numel()} numbers, a unit {n}, all units {units * n}")
-    _run("hb_gated_rmsnorm", dtype_code(out.dtype), o.data_ptr(), o.stride(0), w.data_ptr(), float(eps), gate.data_ptr(),
+    floor, div_scale, div_eps = divide if divide is not None else (None, 1.0, 0.0)
+    if floor is not None:
+        _check(floor, torch.float32, "floor")
+        if not floor.is_contiguous() or floor.numel() != o.shape[0] * units:
+            raise BackendError(f"gated_rmsnorm: the floor must be a contiguous [{o.shape[0]}, {units}] array")
+    _run("hb_gated_rmsnorm", dtype_code(out.dtype), o.data_ptr(), o.stride(0), int(n if unit_stride is None else unit_stride), w.data_ptr(), float(eps), gate.data_ptr(),
          gate.stride(0), out.data_ptr(), out.stride(0), o.shape[0], int(units), int(n), 1 if sigmoid_gate else 0,
-         int(n) if (units > 1 and w.numel() == units * n) else 0, 1 if gate_first else 0, _stream())
+         int(n) if (units > 1 and w.numel() == units * n) else 0, 1 if gate_first else 0, _ptr(floor), float(div_scale),
+         float(div_eps), _stream())
 
 
 def qkv_rotary_cache(rows, wq, wk, eps, fqk, rot, halves, fv, batch, seq_pages, q_out, k_cache, v_cache, num_heads,
-                     num_kv_heads, dk, dv, hd, page_size, write_cache=True, bias=None, mscale=1.0, maps=1) -> None:
+                     num_kv_heads, dk, dv, hd, page_size, write_cache=True, bias=None, mscale=1.0, maps=1, head_norm=False, blend=None,
+                     keep=None) -> None:
     """Float rows [q: heads x dk | k: kv heads x dk | v: kv heads x dv] (+ bias in the same layout): q and k normed over the whole projection
     (weights wq, wk; None: no norm), pair m of their first `rot` channels turned by p * fqk[m], pair m of all value
     channels by p * fv[m] (fv None: values as they are; q's and k's cos and sin times `mscale`); q into q_out (heads of hd
     channels), k and v into the paged cache (heads of hd channels, zeros beyond dk and dv).  With `maps` > 1 every head has
     that many queries and keys of dk channels: the query of map m is a query head of its own (heads x maps of them in q_out)
-    whose channels from m * dk are set, a key head of the cache holds its maps side by side."""
+    whose channels from m * dk are set, a key head of the cache holds its maps side by side.  With `head_norm` every head of q
+    and k is normed by itself (wq and wk [dk], shared by the heads).  `blend` = (values [T, kv heads * dv] float, lambda): the
+    stored value is (1 - lambda) v + lambda * that; `keep` (float, the same shape) receives v before that."""
+    lam = 0.0
+    if blend is not None:
+        blend, lam = blend
+    for t, n in ((blend, "blend"), (keep, "keep")):
+        if t is not None:
+            _check(t, torch.float32, n)
+            if not t.is_contiguous() or tuple(t.shape) != (rows.shape[0], num_kv_heads * dv):
+                raise BackendError(f"qkv_rotary_cache: {n} must be a contiguous [{rows.shape[0]}, {num_kv_heads * dv}] array, got {list(t.shape)}")
     _check(rows, torch.float32, "rows"); _check(q_out, k_cache.dtype, "q_out")
     for t, n in ((wq, "wq"), (wk, "wk"), (fqk, "fqk"), (fv, "fv"), (bias, "bias")):
         if t is not None:
             _check(t, torch.float32, n)
     _run("hb_qkv_rotary_cache", dtype_code(q_out.dtype), rows.data_ptr(), rows.stride(0), _ptr(bias), _ptr(wq), _ptr(wk), float(eps),
-         1 if wq is not None else 0, _ptr(fqk), int(rot), 1 if halves else 0, float(mscale), _ptr(fv), batch.tok_seq.data_ptr(),
+         0 if wq is None else 2 if head_norm else 1, _ptr(fqk), int(rot), 1 if halves else 0, float(mscale), _ptr(fv), batch.tok_seq.data_ptr(),
          batch.tok_pos.data_ptr(), seq_pages.data_ptr(), seq_pages.stride(0), q_out.data_ptr(), q_out.stride(0),
          k_cache.data_ptr(), v_cache.data_ptr(), rows.shape[0], int(num_heads), int(num_kv_heads), int(maps), int(dk), int(dv), int(hd),
-         int(page_size), 1 if write_cache else 0, _stream())
+         int(page_size), 1 if write_cache else 0, _ptr(blend), float(lam), _ptr(keep), _stream())
 
 
 def rotate_heads_back(att, hd, fv, halves, tok_pos, out, num_heads, dv) -> None:
@@ -719,18 +749,23 @@ def streams_join(x, y=None, mix=None, out_w=None, in_w=None, norm=None, h=None, 
 SSD_CHUNKED_MIN_TOKENS = 16
 
 
-def ssd_scan(xbc, b_off, c_off, dt, dt_bias, a_log, dskip, state, batch, out, heads, groups, n_state, dv, scratch) -> None:
+def ssd_scan(xbc, b_off, c_off, dt, dt_bias, a_log, dskip, state, batch, out, heads, groups, n_state, dv, scratch, logd=None) -> None:
     """S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + dskip x over every sequence's tokens of the step, in order, from and
     into state[slot] ([slots, heads, n_state, dv] float), with dt = softplus(raw + dt_bias).  xbc rows hold x (heads * dv)
     from column 0, B from b_off and C from c_off (groups * n_state each; head h reads group h / (heads / groups)); dt raw,
-    float [T, heads]; out float [T, heads * dv].  bfloat16 steps that bring many tokens run chunk by chunk on the tensor cores."""
+    float [T, heads]; out float [T, heads * dv].  bfloat16 steps that bring many tokens run chunk by chunk on the tensor cores.
+    With `logd` [T, heads] the decays are e^logd (logd <= 0) and dt holds the weights of B x^T as they are; dt_bias, a_log and
+    dskip are then None."""
     _check(xbc, None, "xbc")
-    for t, n in ((dt, "dt"), (dt_bias, "dt_bias"), (a_log, "a_log"), (dskip, "dskip"), (state, "state"), (out, "out")):
-        _check(t, torch.float32, n)
+    for t, n in ((dt, "dt"), (logd, "logd"), (dt_bias, "dt_bias"), (a_log, "a_log"), (dskip, "dskip"), (state, "state"), (out, "out")):
+        if t is not None:
+            _check(t, torch.float32, n)
+    if logd is not None and logd.stride(0) != dt.stride(0):
+        raise BackendError("ssd_scan: log decays and weights must have one row stride")
     if not state.is_contiguous() or tuple(state.shape[1:]) != (heads, n_state, dv):
         raise BackendError(f"ssd_scan: state of shape {tuple(state.shape)} is not [slots, {heads}, {n_state}, {dv}]")
-    args = (xbc.data_ptr(), xbc.stride(0), int(b_off), int(c_off), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr(), a_log.data_ptr(),
-            dskip.data_ptr(), state.data_ptr(), batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), out.data_ptr(), out.stride(0),
+    args = (xbc.data_ptr(), xbc.stride(0), int(b_off), int(c_off), dt.data_ptr(), dt.stride(0), _ptr(logd), _ptr(dt_bias), _ptr(a_log),
+            _ptr(dskip), state.data_ptr(), batch.seq_slot.data_ptr(), batch.seq_start.data_ptr(), out.data_ptr(), out.stride(0),
             batch.n_seqs)
     chunks = 0
     if options.ssd_chunked and xbc.dtype == torch.bfloat16 and batch.max_q_len >= SSD_CHUNKED_MIN_TOKENS:
@@ -777,6 +812,65 @@ def general_delta_scan(prep, v, state, batch, out, heads, dk, dv) -> None:
         raise BackendError(f"general_delta_scan: state of shape {tuple(state.shape)} is not [slots, {heads}, {dk}, {dv}]")
     _run("hb_general_delta_scan", prep.data_ptr(), v.data_ptr(), v.stride(0), state.data_ptr(), batch.seq_slot.data_ptr(),
          batch.seq_start.data_ptr(), out.data_ptr(), out.stride(0), batch.n_seqs, int(heads), int(dk), int(dv), _stream())
+
+
+def channel_delta_prepare(qk, q_off, k_off, rows, b_off, low_off, w2, dt_bias, a_log, unit_eps, qscale, prep, heads, qk_heads, dk,
+                          gate_off=0, gate_low=None) -> None:
+    """The delta rule with a decay per key channel, for `general_delta_scan`: from float rows qk (q and k, qk_heads * dk numbers
+    each) and rows (b: one number per head, low: the decay's inner row of w2.shape[1] numbers): prep [T, heads, 5, dk] = q' , beta k',
+    g, g k', beta k' with unit vectors x / sqrt(sum x^2 + unit_eps) per head, q' also times qscale, beta = sigmoid(b),
+    g = exp(-exp(a_log) softplus(w2 low + dt_bias)).  `gate_low` [T, r], if given, receives rows[:, gate_off : gate_off + r] in its dtype."""
+    for t, n in ((qk, "qk"), (rows, "rows"), (dt_bias, "dt_bias"), (a_log, "a_log"), (prep, "prep")):
+        _check(t, torch.float32, n)
+    _check(w2, None, "w2")
+    if not (w2.is_contiguous() and prep.is_contiguous()) or w2.shape[0] != heads * dk:
+        raise BackendError("channel_delta_prepare: w2 must be [heads * dk, rank] and contiguous, prep contiguous")
+    if gate_low is not None:
+        _check(gate_low, w2.dtype, "gate_low")
+    _run("hb_channel_delta_prepare", dtype_code(w2.dtype), qk.data_ptr(), qk.stride(0), int(q_off), int(k_off), rows.data_ptr(),
+         rows.stride(0), int(b_off), int(low_off), w2.data_ptr(), dt_bias.data_ptr(), a_log.data_ptr(), float(unit_eps), float(qscale),
+         prep.data_ptr(), int(gate_off), 0 if gate_low is None else gate_low.shape[1], _ptr(gate_low),
+         0 if gate_low is None else gate_low.stride(0), qk.shape[0], int(heads), int(qk_heads), int(dk), w2.shape[1], _stream())
+
+
+def matrix_memory_prepare(rows, q_off, k_off, v_off, i_off, f_off, i_bias, f_bias, cap, m_state, batch, packed, logd, weight, floor,
+                          heads, dk, dv, dvp) -> None:
+    """From a matrix memory's projection (float rows): packed [T, >= heads * (dvp + 2 dk)] in its dtype = values (heads of dvp
+    columns: dv values, a one, zeros), keys, queries; and per token and head, with i = cap tanh((zi + i_bias) / cap),
+    f = log sigmoid(cap tanh((zf + f_bias) / cap)) and the running maximum m <- max(f + m, i) (m_state [slots, heads], where the step
+    leaves its last one): logd = f + m_before - m, weight = e^(i - m), floor = e^-m."""
+    for t, n in ((rows, "rows"), (i_bias, "i_bias"), (f_bias, "f_bias"), (m_state, "m_state"), (logd, "logd"), (weight, "weight"), (floor, "floor")):
+        _check(t, torch.float32, n)
+    _check(packed, None, "packed")
+    if not all(t.is_contiguous() and tuple(t.shape) == (rows.shape[0], heads) for t in (logd, weight, floor)) or not m_state.is_contiguous():
+        raise BackendError(f"matrix_memory_prepare: the gates' arrays must be contiguous [{rows.shape[0]}, {heads}]")
+    _run("hb_matrix_memory_prepare", dtype_code(packed.dtype), rows.data_ptr(), rows.stride(0), int(q_off), int(k_off), int(v_off),
+         int(i_off), int(f_off), i_bias.data_ptr(), f_bias.data_ptr(), float(cap), m_state.data_ptr(), batch.seq_slot.data_ptr(),
+         batch.seq_start.data_ptr(), packed.data_ptr(), packed.stride(0), logd.data_ptr(), weight.data_ptr(), floor.data_ptr(),
+         rows.shape[0], batch.n_seqs, batch.max_q_len, int(heads), int(dk), int(dv), int(dvp), _stream())
+
+
+def residual_tanh(x, norms, y=None, mult=1.0, bias=None, rows=None) -> None:
+    """x += mult * (y + bias) (float; y None: x stays), then for each of at most two norms ((alpha, w, b), h):
+    h = tanh(alpha * x) * w + b in h's dtype; `rows` (only without y) chooses the rows of x."""
+    _check(x, torch.float32, "x")
+    if not x.is_contiguous() or len(norms) > 2 or (rows is not None and y is not None):
+        raise BackendError("residual_tanh: x must be contiguous, the norms at most two, and chosen rows without a result")
+    for t, n in ((y, "y"), (bias, "bias")):
+        if t is not None:
+            _check(t, torch.float32, n)
+    n_rows = x.shape[0] if rows is None else rows.shape[0]
+    args, dtype = [], F32
+    for (alpha, w, b), h in norms:
+        _check(w, torch.float32, "w"); _check(b, torch.float32, "b"); _check(h, None, "h")
+        n_rows = h.shape[0] if rows is not None else n_rows
+        if not h.is_contiguous() or tuple(h.shape) != (n_rows, x.shape[1]):
+            raise BackendError("residual_tanh: h must be contiguous, a row of the width for every row asked for")
+        dtype = dtype_code(h.dtype)
+        args += [float(alpha), w.data_ptr(), b.data_ptr(), h.data_ptr()]
+    args += [0.0, None, None, None] * (2 - len(norms))
+    _run("hb_residual_tanh", dtype, _ptr(y), y.stride(0) if y is not None else 0, _ptr(bias), float(mult), x.data_ptr(), _ptr(rows),
+         *args, n_rows, x.shape[1], _stream())
 
 
 def gated_norm_residual(y, w, eps, x, dtype, gate=None, gate_bias=None, next_norm=None, h=None) -> None:
@@ -841,7 +935,7 @@ def moe_tc_ok(h, up, top, gated, act) -> bool:
             and h.shape[0] * int(top) >= MOE_TC_MIN_PAIRS)
 
 
-def moe_experts_tc(h, up, down, ids, weights, y, accumulate, scratch, act_limit=0.0) -> None:
+def moe_experts_tc(h, up, down, ids, weights, y, accumulate, scratch, act_limit=0.0, weigh_input=False) -> None:
     """moe_experts for long prompts, gated experts with silu (or, with act_limit > 0, the clamped activation): the pairs
     sorted by expert into runs padded to tiles of 128 rows, both products on tcgen05 (the first with the gated
     activation in its epilogue)."""
@@ -856,13 +950,14 @@ def moe_experts_tc(h, up, down, ids, weights, y, accumulate, scratch, act_limit=
     srt = scratch((rows, D), torch.bfloat16)
     mid = scratch((rows, F), torch.bfloat16)
     part = scratch((rows, D), torch.float32)
+    row_scale = scratch((rows,), torch.float32) if weigh_input else None
     _tcgen05_workspace(y.device)
     _run("hb_moe_experts_tc_bf16", h.data_ptr(), h.stride(0), up.data_ptr(), down.data_ptr(), ids.data_ptr(), weights.data_ptr(),
          ints.data_ptr(), srt.data_ptr(), mid.data_ptr(), part.data_ptr(), y.data_ptr(), y.stride(0), T, D, E, F, top,
-         float(act_limit), 1 if accumulate else 0, _error_flag(y.device).data_ptr(), _stream())
+         float(act_limit), _ptr(row_scale), 1 if accumulate else 0, _error_flag(y.device).data_ptr(), _stream())
 
 
-def moe_experts_grouped(h, up, down, ids, weights, y, act, accumulate, scratch, gated=0, act_limit=0.0) -> None:
+def moe_experts_grouped(h, up, down, ids, weights, y, act, accumulate, scratch, gated=0, act_limit=0.0, weigh_input=False) -> None:
     """moe_experts for many tokens: pairs grouped by expert on the device, tiles of 64 pairs on the tensor cores."""
     _check(h, torch.bfloat16, "h"); _check(up, torch.bfloat16, "up"); _check(down, torch.bfloat16, "down"); _check(y, torch.float32, "y")
     T, top = ids.shape
@@ -874,20 +969,21 @@ def moe_experts_grouped(h, up, down, ids, weights, y, act, accumulate, scratch, 
     part = scratch((T * top, D), torch.float32)
     _run("hb_moe_experts_grouped_bf16", h.data_ptr(), h.stride(0), up.data_ptr(), down.data_ptr(), ids.data_ptr(), weights.data_ptr(),
          ints.data_ptr(), mid.data_ptr(), part.data_ptr(), y.data_ptr(), y.stride(0), T, D, E, F, top, int(act),
-         int(gated), float(act_limit), 1 if accumulate else 0, _stream())
+         int(gated), float(act_limit), 1 if weigh_input else 0, 1 if accumulate else 0, _stream())
 
 
-def moe_experts(h, up, down, ids, weights, mid, y, act, accumulate=False, gated=0, act_limit=0.0) -> None:
+def moe_experts(h, up, down, ids, weights, mid, y, act, accumulate=False, gated=0, act_limit=0.0, weigh_input=False) -> None:
     """y[t] (+)= sum_r weights[t, r] * down[e] act(up[e] h[t]), e = ids[t, r]; up [E, F, D], down [E, D, F] in
     h's dtype; mid [T * top, F] scratch in h's dtype; y float.  gated: up is [E, 2F, D] and an expert is
     down[e] (act(gate h) * (up h)), with the gate and up rows in turn in groups of 8 (GATED_GROUPS_OF_8) or all
-    gate rows before all up rows (GATED_HALVES).  act ACT_SWISH_CLAMP (gated experts only) takes `act_limit`."""
+    gate rows before all up rows (GATED_HALVES).  act ACT_SWISH_CLAMP (gated experts only) takes `act_limit`.
+    `weigh_input` (gated experts only): the weight multiplies the expert's input instead of its output."""
     _check(h, None, "h"); _check(up, h.dtype, "up"); _check(down, h.dtype, "down"); _check(mid, h.dtype, "mid"); _check(y, torch.float32, "y")
     if not (up.is_contiguous() and down.is_contiguous() and mid.is_contiguous()):
         raise BackendError("moe_experts: up, down and mid must be contiguous")
     _run("hb_moe_experts", dtype_code(h.dtype), h.data_ptr(), h.stride(0), up.data_ptr(), down.data_ptr(), ids.data_ptr(),
          weights.data_ptr(), mid.data_ptr(), y.data_ptr(), y.stride(0), h.shape[0], h.shape[1], down.shape[2], ids.shape[1],
-         int(act), int(gated), float(act_limit), 1 if accumulate else 0, _stream())
+         int(act), int(gated), float(act_limit), 1 if weigh_input else 0, 1 if accumulate else 0, _stream())
 
 
 def rmsnorm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, eps: float, rows: torch.Tensor | None = None) -> None:

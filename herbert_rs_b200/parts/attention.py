@@ -28,6 +28,10 @@ after the projection (its last inputs are state of the sequence); sigmoid weight
 every visible key with nothing normalised over the keys; one output gate per token and head, sigmoid(G h), whose
 rows are part of the one projection; and a mixer without keys and values of its own, whose schedule step reads
 another step's cache with its own queries, window and gates.
+Its queries and keys may be normed head by head, its output projection may have a bias (which a block that joins the result to
+the stream in one kernel adds itself: `take_output_bias`), and its values may be blended, token by token, with those that an
+earlier layer of the step kept (they live in the step's scratch memory, from layer to layer; the blended values are what the cache
+holds).
 It also takes biases on the projections, scaled rotary frequencies (cos and sin times a constant) and `difference`: two
 attention maps per head over the same values.  Their keys lie side by side in one cache head (so the values are stored
 once), the query of either map is a query head that is zero in the other map's channels, and the attention kernels run
@@ -59,7 +63,7 @@ class AttentionMixer(Mixer):
         self.plain = not (spec.bias or spec.values_are_keys or spec.q_temperature or spec.softcap or spec.sink)
         self.pairs = bool(spec.whole_qk_norm or spec.value_dim is not None or spec.value_rotation is not None
                           or getattr(spec.position, "kind", None) in ("rope_pairs", "scaled_rope") or spec.key_weights != "softmax"
-                          or spec.difference is not None or spec.conv_taps is not None or spec.head_gate or spec.reads_kv)
+                          or spec.head_qk_norm or spec.output_bias or spec.value_blend is not None or spec.difference is not None or spec.conv_taps is not None or spec.head_gate or spec.reads_kv)
         if self.pairs:
             self._init_pairs()
             return
@@ -79,11 +83,17 @@ class AttentionMixer(Mixer):
     # -- the third form ------------------------------------------------------------------------
     def _init_pairs(self):
         s = self.spec
-        if s.values_are_keys or s.q_temperature or s.softcap or s.sink or s.qk_norm is not None and not s.whole_qk_norm:
+        if s.values_are_keys or s.q_temperature or s.softcap or s.sink or s.qk_norm is not None and not (s.whole_qk_norm or s.head_qk_norm):
             raise ConfigError("attention with rotated pairs, a norm over the whole projection or rotated values has "
                               "none of the other options (shared values, temperature, cap, sink, head norm)")
-        if s.whole_qk_norm and s.qk_norm is None:
-            raise ConfigError("a norm over the whole q and k projections needs its eps (qk_norm)")
+        if (s.whole_qk_norm or s.head_qk_norm) and s.qk_norm is None:
+            raise ConfigError("a norm over the q and k projections needs its eps (qk_norm)")
+        if s.head_qk_norm and (s.whole_qk_norm or s.difference is not None):
+            raise ConfigError("a norm per head serves one attention map per head, and no norm over the whole projection beside it")
+        if s.value_blend not in (None, "keep", "blend"):
+            raise ConfigError(f"unknown value blend {s.value_blend!r}: keep, blend")
+        if s.value_blend is not None and (s.value_rotation is not None or s.reads_kv or s.conv_taps is not None):
+            raise ConfigError("values that are kept or blended are the layer's own, neither rotated nor convolved")
         self.plain = False
         self.dk = s.head_dim
         self.dv = s.value_dim if s.value_dim is not None else s.head_dim
@@ -92,6 +102,7 @@ class AttentionMixer(Mixer):
         if self.maps > 1:
             if s.key_weights != "softmax" or s.head_gate or s.reads_kv or s.value_rotation is not None:
                 raise ConfigError("the difference of two attention maps has softmax weights, keys of its own, no gates and no rotated values")
+        if self.maps > 1 or s.head_qk_norm:
             self.hd = (self.hd + 15) // 16 * 16      # what the tensor-core kernels take; the channels added are zeros
         self.q_dim, self.kv_dim = self.nh * self.maps * self.dk, self.nkv * self.maps * self.dk
         if s.key_weights not in ("softmax", "sigmoid"):
@@ -104,7 +115,8 @@ class AttentionMixer(Mixer):
         # what the projection's rows hold: q, then (unless another step's are read) k and v, then one gate per head
         self.qkv_dim = self.q_dim + (0 if self.reads_kv else self.kv_dim + self.nkv * self.dv)
         self.proj_dim = self.qkv_dim + (self.nh if s.head_gate else 0)
-        self.key_bias = self.w_conv = self.difference = None
+        self.key_bias = self.w_conv = self.difference = self.bo = None
+        self.blend = 0.0
         self.value_position = build_part("position", s.value_rotation, rt=self.rt) if s.value_rotation is not None else None
         if self.value_position is not None and self.value_position.rotary_dim != self.dv:
             raise ConfigError(f"values of {self.dv} channels are turned over all of them, not {self.value_position.rotary_dim}")
@@ -138,6 +150,13 @@ class AttentionMixer(Mixer):
         if self.maps > 1:
             for n in s.difference_names:
                 p[n] = ParamSpec((self.dk,), role="vector", init="zeros_noise")
+        if s.output_bias:
+            p[self.n_o + s.bias_suffix] = ParamSpec((s.hidden_size,), role="vector", init="normal")
+        if s.value_blend is not None:
+            p[s.value_blend_name] = ParamSpec((), role="vector", init="zeros_noise")
+        if s.head_qk_norm:
+            p[s.norm_names[0]] = ParamSpec((self.dk,), role="vector", init="ones_noise")
+            p[s.norm_names[1]] = ParamSpec((self.dk,), role="vector", init="ones_noise")
         if s.whole_qk_norm:
             p[s.norm_names[0]] = ParamSpec((self.q_dim,), role="vector", init="ones_noise")
             p[s.norm_names[1]] = ParamSpec((self.kv_dim,), role="vector", init="ones_noise")
@@ -158,11 +177,37 @@ class AttentionMixer(Mixer):
             self.difference = (lam, 1.0 - float(s.difference), s.difference_eps, self.dv)
         if self.sigmoid_keys:
             self.key_bias = tensors[s.key_bias_name].contiguous()
-        if s.whole_qk_norm:
+        if s.output_bias:
+            self.bo = tensors[self.n_o + s.bias_suffix].contiguous()
+        if s.value_blend == "blend":
+            self.blend = float(tensors[s.value_blend_name])
+        if s.whole_qk_norm or s.head_qk_norm:
             self.q_norm = tensors[s.norm_names[0]].contiguous()
             self.k_norm = tensors[s.norm_names[1]].contiguous()
 
-    def _forward_pairs(self, h, residual, batch, cache, accumulate):
+    def take_output_bias(self):
+        """The output projection's bias, for a caller that adds it itself right after forward(with_output_bias=False);
+        None if there is none."""
+        return self.bo if self.pairs else None
+
+    def _project(self, y, residual, accumulate, with_output_bias):
+        ops.gemm(y, self.wo, residual, ops.EPI_RESIDUAL if accumulate else ops.EPI_STORE_F32, scratch=self.rt.workspace.take)
+        if self.bo is not None and with_output_bias:
+            ops.add_row_bias(residual, self.bo)
+
+    def _value_blend(self, batch, T):
+        """(what the values are blended with, where they are to be kept) in this step."""
+        s = self.spec
+        if s.value_blend is None:
+            return None, None
+        if s.value_blend == "keep":
+            batch.kept[s.value_blend_name] = kept = self.rt.workspace.take_for_step((T, self.nkv * self.dv), torch.float32)
+            return None, kept
+        if s.value_blend_name not in batch.kept:
+            raise ConfigError("a layer blends its values with an earlier layer's, but none of the step has kept its own")
+        return (batch.kept[s.value_blend_name], self.blend), None
+
+    def _forward_pairs(self, h, residual, batch, cache, accumulate, with_output_bias):
         s, ws, T = self.spec, self.rt.workspace, h.shape[0]
         proj = ws.take((T, self.proj_dim), torch.float32)
         ops.gemm(h, self.wqkv, proj, ops.EPI_STORE_F32, scratch=ws.take)
@@ -180,16 +225,17 @@ class AttentionMixer(Mixer):
         pos, vpos = self.position, self.value_position
         halves = pos.halves if pos is not None else (vpos.halves if vpos is not None else False)
         fv = vpos.freq if vpos is not None else None
+        blend, keep = self._value_blend(batch, T)
         ops.qkv_rotary_cache(rows, self.q_norm, self.k_norm, s.qk_norm.eps if s.qk_norm is not None else 0.0,
                              pos.freq if pos is not None else None, pos.rotary_dim if pos is not None else 0, halves, fv,
                              batch, pages, q, cache.k, cache.v, self.nh, self.nkv, self.dk, self.dv, self.hd,
                              cache.page_size, write_cache=cache.writes_kv and not self.reads_kv, bias=bias,
-                             mscale=pos.mscale if pos is not None else 1.0, maps=self.maps)
+                             mscale=pos.mscale if pos is not None else 1.0, maps=self.maps, head_norm=s.head_qk_norm, blend=blend, keep=keep)
         if self.maps > 1:
             y = ws.take((T, self.nh * self.dv), h.dtype)
             ops.attention(q, q.stride(0), y, cache.k, cache.v, batch, nq, self.nkv, self.hd, cache.page_size, s.scale, s.window, pages,
                           scratch=ws.take, difference=self.difference)
-            ops.gemm(y, self.wo, residual, ops.EPI_RESIDUAL if accumulate else ops.EPI_STORE_F32, scratch=ws.take)
+            self._project(y, residual, accumulate, with_output_bias)
             return
         att = ws.take((T, self.nh * self.hd), h.dtype)
         # the gate per token and head multiplies a head's float result inside the attention kernel, before it is rounded
@@ -203,7 +249,7 @@ class AttentionMixer(Mixer):
         elif self.hd != self.dv:          # heads of the cache's width -> heads of the values' width
             y = ws.take((T, self.nh * self.dv), h.dtype)
             ops.head_gate(att, self.hd, None, y, self.nh, self.dv)
-        ops.gemm(y, self.wo, residual, ops.EPI_RESIDUAL if accumulate else ops.EPI_STORE_F32, scratch=ws.take)
+        self._project(y, residual, accumulate, with_output_bias)
 
     def param_specs(self):
         s = self.spec
@@ -267,9 +313,9 @@ class AttentionMixer(Mixer):
                       self.hd, cache.page_size, s.scale, s.window, pages, scratch=ws.take, softcap=s.softcap, sink=self.sink)
         ops.gemm(att, self.wo, residual, ops.EPI_RESIDUAL if accumulate else ops.EPI_STORE_F32, scratch=ws.take)
 
-    def forward(self, h, residual, batch, cache, next_norm=None, accumulate=True):
+    def forward(self, h, residual, batch, cache, next_norm=None, accumulate=True, with_output_bias=True):
         if self.pairs:
-            return self._forward_pairs(h, residual, batch, cache, accumulate)
+            return self._forward_pairs(h, residual, batch, cache, accumulate, with_output_bias)
         if not self.plain:
             return self._forward_options(h, residual, batch, cache, accumulate)
         ws, T = self.rt.workspace, h.shape[0]

@@ -49,6 +49,16 @@ class ParamSpec:
     free_size: int = 16
 
 
+def stack_rows(matrices, multiple: int = 8) -> torch.Tensor:
+    """Matrices of one width as one, rows below each other, with zero rows up to a multiple of `multiple`: a product with it
+    leaves rows that start on 16 bytes whatever the parts' sizes are."""
+    n = sum(int(m.shape[0]) for m in matrices)
+    pad = -n % multiple
+    if pad:
+        matrices = list(matrices) + [torch.zeros((pad, matrices[0].shape[1]), dtype=matrices[0].dtype, device=matrices[0].device)]
+    return torch.cat(matrices, dim=0).contiguous()
+
+
 class Part:
     # True if forward() takes every per-step fact (tokens, positions, lengths, pages, slots) from
     # the batch's device arrays, so that a recorded CUDA graph of a step can be replayed for later
@@ -82,6 +92,15 @@ class Norm(Part):
         before it and a product after it can compute between them; else None."""
         return None
 
+    def as_pointwise(self):
+        """(alpha, weight [D] float, bias [D] float) if this is tanh(alpha * x) * weight + bias, which a kernel that updates x
+        can apply channel by channel in the same pass; else None."""
+        return None
+
+    def scale_result(self, factor: float) -> bool:
+        """Multiply every later result by `factor`, if the norm can do so at no cost (by scaling its loaded weights)."""
+        return False
+
     def as_stream_norm(self):
         """(weight [D] float, bias [D] float or None, eps, rms) if this is a layer norm, or (rms True) a plain RMS norm, which
         the kernel that joins a sublayer's result to a stream of several copies can apply to what it mixes; else None."""
@@ -108,6 +127,10 @@ class Block(Part):
     # True if forward() takes the keywords `normed` and `next_norm` below; a block without the flag is
     # called as forward(x, batch, cache) and its neighbours run their norms themselves.
     chains_norms = False
+    # What `first_norm().shareable()` gives and `next_norm` takes: only blocks of one kind hand norms to one another.
+    #   "norm": (weight, eps) of an RMS norm; "pointwise": a tuple of norms without statistics, one per sublayer;
+    #   "streams": a block of several copies of the stream.
+    chain_kind = "norm"
     # How many copies of the stream forward() works on, as an array [T, streams, H]; None: one stream [T, H].
     streams = None
 

@@ -204,9 +204,11 @@ class SublayerNormBlock(Block):
 class ParallelBlock(Block):
     """h = norm1(x); x += m * (mixer(h) + ffn(h)): one norm whose result both sublayers read, one
     factor m on their sum.  The sublayers write into one float array (the mixer stores, the
-    feed-forward adds), and one kernel adds it, times m, to the stream and runs the RMS norm the next
+    feed-forward adds), and one kernel adds it, times m, to the stream and runs the norm the next
     block begins with, so that between two layers the stream is read and written once.  The spec may
-    leave out the feed-forward."""
+    leave out the feed-forward.  With a norm2 the feed-forward reads norm2(x), of the same x: x += m * (mixer(norm1(x)) +
+    ffn(norm2(x))).  That kernel runs an RMS norm (one norm1 for both sublayers), or any of one or two norms without
+    statistics (`Norm.as_pointwise`); other norms are kernels of their own at the block's start."""
 
     chains_norms = True
 
@@ -215,8 +217,12 @@ class ParallelBlock(Block):
         self.norm1 = build_part("norm", spec.norm1, rt=rt)
         self.mixer = build_part("mixer", spec.mixer, rt=rt)
         self.ffn = build_part("ffn", spec.ffn, rt=rt) if spec.ffn is not None else None
+        self.norm2 = build_part("norm", spec.norm2, rt=rt) if spec.norm2 is not None and self.ffn is not None else None
+        self.norms = [n for n in (self.norm1, self.norm2) if n is not None]
         self.mult = float(spec.residual_mult)
         self._names = dict(spec.names)
+        self.pointwise = all(n.as_pointwise() is not None for n in self.norms)
+        self.chain_kind = "pointwise" if self.pointwise else "norm"
         for part in (self.mixer, self.ffn):
             if part is not None and not part.can_store:
                 raise ConfigError(f"{type(part).__name__} cannot store its result apart from the residual stream, "
@@ -228,6 +234,8 @@ class ParallelBlock(Block):
 
     def children(self):
         parts = [("norm1", self.norm1), ("mixer", self.mixer)]
+        if self.norm2 is not None:
+            parts.append(("norm2", self.norm2))
         if self.ffn is not None:
             parts.append(("ffn", self.ffn))
         return tuple(parts)
@@ -250,28 +258,63 @@ class ParallelBlock(Block):
         return self.mixer.cache_need()
 
     def first_norm(self):
-        return self.norm1
+        if self.pointwise:
+            return _PointwiseEntry(self)
+        return self.norm1 if self.norm2 is None else None      # two norms with statistics: the block runs them itself
+
+    def _outputs(self, norms, x):
+        """The given norms of x as (norm, where its result goes)."""
+        return [(n, self.rt.workspace.take(x.shape, self.rt.dtype)) for n in norms]
+
+    def _inputs(self, x, normed):
+        """What the mixer and the feed-forward read: as many tensors as the block has norms."""
+        if isinstance(normed, tuple):
+            return normed
+        if isinstance(normed, torch.Tensor):
+            return (normed,)
+        if normed is None and self.pointwise:
+            outs = self._outputs([n.as_pointwise() for n in self.norms], x)
+            ops.residual_tanh(x, outs)
+            return tuple(h for _, h in outs)
+        outs = self._outputs(self.norms, x)
+        if normed is not None:
+            ops.finish_norm(normed, outs[0][1])
+        else:
+            for norm, h in outs:
+                norm.forward(x, h)
+        return tuple(h for _, h in outs)
 
     def forward(self, x, batch, cache, normed=None, next_norm=None):
         ws, dtype = self.rt.workspace, self.rt.dtype
-        if isinstance(normed, torch.Tensor):
-            h = normed
-        else:
-            h = ws.take(x.shape, dtype)
-            if normed is not None:
-                ops.finish_norm(normed, h)
-            else:
-                self.norm1.forward(x, h)
+        inputs = self._inputs(x, normed)
         y = ws.take(x.shape, torch.float32)
-        self.mixer.forward(h, y, batch, cache, accumulate=False)
+        bias = self.mixer.take_output_bias() if self.pointwise and getattr(self.mixer, "take_output_bias", None) is not None else None
+        if bias is not None:
+            self.mixer.forward(inputs[0], y, batch, cache, accumulate=False, with_output_bias=False)
+        else:
+            self.mixer.forward(inputs[0], y, batch, cache, accumulate=False)
         if self.ffn is not None:
-            self.ffn.forward(h, y, batch, accumulate=True)
+            self.ffn.forward(inputs[-1], y, batch, accumulate=True)
+        if self.pointwise:
+            outs = self._outputs(next_norm or (), x)
+            ops.residual_tanh(x, outs, y=y, mult=self.mult, bias=bias)
+            return tuple(h for _, h in outs) if next_norm else None
         if next_norm is None:
             ops.scaled_residual_norm(y, self.mult, x)
             return None
         h_next = ws.take(x.shape, dtype)
         ops.scaled_residual_norm(y, self.mult, x, next_norm[0], h_next, next_norm[1])
         return h_next
+
+
+class _PointwiseEntry:
+    """The norms without statistics that a parallel block begins with, for the block before it to run."""
+
+    def __init__(self, block):
+        self.block = block
+
+    def shareable(self):
+        return tuple(n.as_pointwise() for n in self.block.norms)
 
 
 class SandwichBlock(Block):
@@ -442,6 +485,7 @@ class StreamsBlock(Block):
     sublayers every copy is read and written once.  The spec may leave out the feed-forward."""
 
     chains_norms = True
+    chain_kind = "streams"
 
     def __init__(self, spec, rt):
         self.spec, self.rt = spec, rt

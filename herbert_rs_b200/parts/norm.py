@@ -1,5 +1,6 @@
-"""RMSNorm: y = (x / sqrt(mean(x^2) + eps)) * w, in float
-(crates/backends/backend_common/src/kernels.rs:54-64), and the layer norm with a weight and, if the spec asks, a bias.
+"""Norms.  RMSNorm: y = (x / sqrt(mean(x^2) + eps)) * w, in float
+(crates/backends/backend_common/src/kernels.rs:54-64), the layer norm with a weight and, if the spec asks, a bias, and a
+"norm" without statistics, tanh(alpha * x) * w + b.
 A spec with `weight_offset` c stores w - c (weights around zero with c = 1); the offset is added once,
 in float, when the tensor is loaded, so every kernel and the norm shared between two products see w."""
 
@@ -40,6 +41,10 @@ class RMSNorm(Norm):
         else:
             ops.rmsnorm(x, self.weight, out, self.eps, rows)
 
+    def scale_result(self, factor):
+        self.weight = self.weight * factor
+        return True
+
     def shareable(self):
         return (self.weight, self.eps) if self.groups == 1 else None
 
@@ -74,6 +79,12 @@ class LayerNorm(RMSNorm):
     def forward(self, x, out, rows=None):
         ops.layernorm(x, self.weight, out, self.eps, rows, bias=self.bias)
 
+    def scale_result(self, factor):
+        super().scale_result(factor)
+        if self.bias is not None:
+            self.bias = self.bias * factor
+        return True
+
     def shareable(self):
         return None         # the products' shared norm is the RMS form only
 
@@ -81,5 +92,37 @@ class LayerNorm(RMSNorm):
         return self.weight, self.bias, self.eps, False
 
 
+class DynamicTanh(Norm):
+    """y = tanh(alpha * x) * w + b, channel by channel; alpha is one number, read from its tensor when it is loaded."""
+
+    def __init__(self, spec, rt):
+        self.dim, self.rt = spec.dim, rt
+        self.name, self.bias_name, self.alpha_name = spec.weight_name, spec.weight_name + spec.bias_suffix, spec.weight_name + spec.alpha_suffix
+        self.alpha = self.weight = self.bias = None
+
+    def param_specs(self):
+        return {self.name: ParamSpec((self.dim,), role="vector", init="ones_noise"),
+                self.bias_name: ParamSpec((self.dim,), role="vector", init="zeros_noise"),
+                self.alpha_name: ParamSpec((), role="vector", init="ones_noise")}
+
+    def load(self, tensors):
+        self.alpha = float(tensors[self.alpha_name])
+        self.weight, self.bias = tensors[self.name].contiguous(), tensors[self.bias_name].contiguous()
+
+    def weight_bytes(self):
+        return self.dim * 8
+
+    def forward(self, x, out, rows=None):
+        ops.residual_tanh(x, [(self.as_pointwise(), out)], rows=rows)
+
+    def scale_result(self, factor):
+        self.weight, self.bias = self.weight * factor, self.bias * factor
+        return True
+
+    def as_pointwise(self):
+        return self.alpha, self.weight, self.bias
+
+
+register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "rmsnorm", RMSNorm)
 register_part("norm", "layernorm", LayerNorm)
