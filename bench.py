@@ -259,6 +259,33 @@ def _putazen_config(width, heads, kv_heads, dim, vdim, latent_heads, latent_dim,
             "streams": streams, "layers": layers}
 
 
+def _muzasun_config(width, heads, kv_heads, dim, vdim, memory_heads, memory_dim, memory_vdim, delta_heads, delta_qk_heads, delta_dim,
+                    delta_vdim, rank, ff, experts, top, expert_ff, shared_ff, vocab, taps=4):
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "v_mix": True,
+           "rot": {"base": 10000.0, "dims": dim}}
+    memory = {"heads": memory_heads, "dim": memory_dim, "vdim": memory_vdim, "gate_cap": 20.0}
+    delta = {"heads": delta_heads, "kv_heads": delta_qk_heads, "dim": delta_dim, "vdim": delta_vdim, "conv": taps, "low_rank": rank}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared_ff}}
+    layers = [{"type": "mlstm", "mixer": memory, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe},
+              {"type": "channel_delta", "mixer": delta, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe}]
+    return {"architecture": "Muzasun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_scale": 1.0,
+            "layers": layers}
+
+
+MUZASUN_SIZES = {
+    # Muzasun layer sizes (a matrix memory of twice the width, attention, the delta rule with a decay per channel, attention;
+    # dense and routed feed-forwards in turn); beside them Nefivik (the closest in its delta rule, its attention and its gated
+    # experts), Putazen (the closest in its recurrence: a state of the same number of entries on the same kernels), Votapel
+    # (the closest in its residual sum) and the dense decoder, each of the same width and depth
+    "1k": (dict(width=1024, heads=8, kv_heads=4, dim=128, vdim=128, memory_heads=8, memory_dim=128, memory_vdim=256, delta_heads=8,
+                delta_qk_heads=8, delta_dim=128, delta_vdim=128, rank=64, ff=3072, experts=16, top=2, expert_ff=768, shared_ff=1536,
+                vocab=32000), "1k"),
+    "2k": (dict(width=2048, heads=16, kv_heads=8, dim=128, vdim=128, memory_heads=16, memory_dim=128, memory_vdim=256, delta_heads=16,
+                delta_qk_heads=16, delta_dim=128, delta_vdim=128, rank=128, ff=8192, experts=32, top=4, expert_ff=1408, shared_ff=2560,
+                vocab=32000), "2k"),
+}
+
 PUTAZEN_SIZES = {
     # Putazen layer sizes (differential attention, a state-space mixer of twice the width, latent attention, the state-space mixer
     # again; four copies of the stream); beside them Begupel (the closest in its recurrence, convolution, gated norm and the
@@ -437,6 +464,38 @@ def _launcher_work(name, n, ctx):
             return n * 6.0 * T * rows, n * T * rows * (4 + es)
         if name == "hb_difference_heads":
             return n * 6.0 * T * H * dv, n * T * H * dv * (8 + es)
+    elif ctx["kind"] == "muzasun":
+        H, KV, dk, dv, D = ctx["heads"], ctx["kv_heads"], ctx["dim"], ctx["vdim"], ctx["width"]
+        mh, md, mv = ctx["memory_heads"], ctx["memory_dim"], ctx["memory_vdim"]
+        dh, dn, dw, dg = ctx["delta_heads"], ctx["delta_dim"], ctx["delta_vdim"], ctx["delta_qk_heads"]
+        conv = 2 * dg * dn + dh * dw
+        if name in ("hb_attention_prefill_tc_bf16", "hb_attention_prefill_bf16", "hb_attention_decode_bf16", "hb_attention_simt"):
+            return n * 2.0 * pairs * H * (dk + dv), n * (B * L * KV * (dk + dv) * es + T * H * (dk + dv) * es)
+        if name in ("hb_ssd_chunked_bf16", "hb_ssd_scan"):
+            # as Putazen's: 5 operations a state entry and token; reads values, keys, queries and gates, writes the read-outs as
+            # floats, reads and writes every sequence's state
+            return n * 5.0 * T * mh * md * mv, n * (T * (mh * (mv + 2 * md) * es + mh * mv * 4 + 2 * mh * 4) + 2 * B * mh * md * mv * 4)
+        if name == "hb_matrix_memory_prepare":
+            return n * 2.0 * T * mh * (mv + 2 * md), n * T * mh * ((mv + 2 * md) * (4 + es) + 5 * 4)
+        if name == "hb_general_delta_scan":      # as Nefivik's: 9 operations a state entry and token, five key-side vectors, v and o as floats
+            return n * 9.0 * T * dh * dn * dw, n * (T * dh * (5 * dn + 2 * dw) * 4 + 2 * B * dh * dn * dw * 4)
+        if name == "hb_channel_delta_prepare":
+            return n * 8.0 * T * dh * dn, n * T * (2 * dg * dn + 6 * dh * dn + dh) * 4
+        if name == "hb_residual_tanh":      # one per layer updates the stream and leaves two norms; the first and the last only read
+            return n * 8.0 * T * D, n * T * D * (4 + 4 + 4 + 2 * es)
+        if name == "hb_short_conv":
+            return n * 8.0 * T * conv, n * T * conv * 8
+        if name == "hb_qkv_rotary_cache":
+            rows = H * dk + KV * (dk + dv)
+            return n * 6.0 * T * rows, n * T * (rows * (4 + es) + KV * dv * 4)
+        if name == "hb_gated_rmsnorm":
+            per = n / 2.0
+            return per * 8.0 * T * (mh * mv + dh * dw), per * T * (mh * mv + dh * dw) * (4 + 4 + es)
+        if name in ("hb_moe_experts", "hb_moe_experts_grouped_bf16", "hb_moe_experts_tc_bf16"):
+            E, top, F = ctx["experts"], ctx["top"], ctx["expert_ff"]
+            return n * 6.0 * T * top * F * D, n * (min(E, T * top) * 3 * F * D * es + T * D * (es + 4))
+        if name == "hb_moe_route":
+            return n * 2.0 * T * ctx["experts"] * D, n * (T * D * es + ctx["experts"] * D * es)
     else:
         H, KV, hd, D = ctx["heads"], ctx["kv_heads"], ctx["head_dim"], ctx["width"]
         if name in ("hb_attention_prefill_tc_bf16", "hb_attention_prefill_bf16", "hb_attention_decode_bf16",
@@ -514,10 +573,10 @@ def _design_point(hb, ops, torch, np, cfg, ctx, pk, prompt_len, batch, steps, wa
 
 
 def run_design(args) -> int:
-    """`--design begupel|kebisun|nefivik|putazen|votapel`: prefill and decode of that design at layer sizes that resemble a
+    """`--design begupel|kebisun|muzasun|nefivik|putazen|votapel`: prefill and decode of that design at layer sizes that resemble a
     real model's, beside the dense decoder of equal width, depth and feed-forward width (random weights,
     bfloat16, four layers each); Begupel also beside Kebisun with recurrent heads of equal sizes, Nefivik also beside
-    Begupel and Votapel, Putazen also beside Begupel and Kebisun."""
+    Begupel and Votapel, Putazen also beside Begupel and Kebisun, Muzasun also beside Nefivik, Putazen and Votapel."""
     import numpy as np
     import torch
 
@@ -530,13 +589,13 @@ def run_design(args) -> int:
     result = {}
     table, make = {"kebisun": (DESIGN_SIZES, _kebisun_config), "votapel": (VOTAPEL_SIZES, _votapel_config),
                    "begupel": (BEGUPEL_SIZES, _begupel_config), "nefivik": (NEFIVIK_SIZES, _nefivik_config),
-                   "putazen": (PUTAZEN_SIZES, _putazen_config)}[args.design]
+                   "putazen": (PUTAZEN_SIZES, _putazen_config), "muzasun": (MUZASUN_SIZES, _muzasun_config)}[args.design]
     for size in (sorted(table) if args.design_size == "all" else [args.design_size]):
         closest = None
         beside = None
         if args.design == "begupel":
             kb, closest, dense = table[size]
-        elif args.design in ("nefivik", "putazen"):
+        elif args.design in ("muzasun", "nefivik", "putazen"):
             kb, beside = table[size]
             dense = BEGUPEL_SIZES[beside][2]
         else:
@@ -556,7 +615,9 @@ def run_design(args) -> int:
                                                     args.prompt_len, args.batch, args.steps, args.warmup, windows)
         if beside is not None:
             others = {"nefivik": (("begupel", BEGUPEL_SIZES, _begupel_config), ("votapel", VOTAPEL_SIZES, _votapel_config)),
-                      "putazen": (("begupel", BEGUPEL_SIZES, _begupel_config), ("kebisun", DESIGN_SIZES, _kebisun_config))}[args.design]
+                      "putazen": (("begupel", BEGUPEL_SIZES, _begupel_config), ("kebisun", DESIGN_SIZES, _kebisun_config)),
+                      "muzasun": (("nefivik", NEFIVIK_SIZES, _nefivik_config), ("putazen", PUTAZEN_SIZES, _putazen_config),
+                                  ("votapel", VOTAPEL_SIZES, _votapel_config))}[args.design]
             for other, sizes, maker in others:
                 ob = sizes[beside][0]
                 result[size][other] = _design_point(hb, ops, torch, np, maker(**ob), dict(ob, kind=other), pk, args.prompt_len,
@@ -590,7 +651,7 @@ def main() -> int:
     ap.add_argument("--pdl-graph", type=int, default=None, help="programmatic dependent launch inside recorded decode steps (0, 1, 2)")
     ap.add_argument("--workload", default=None, choices=["0.6b", "32b"],
                     help="run only this workload of the baseline and print its line")
-    ap.add_argument("--design", default=None, choices=["begupel", "kebisun", "nefivik", "putazen", "votapel"],
+    ap.add_argument("--design", default=None, choices=["begupel", "kebisun", "muzasun", "nefivik", "putazen", "votapel"],
                     help="measure this design beside the dense decoder at equal sizes instead of the headline workload")
     ap.add_argument("--design-size", default="all", choices=["all"] + sorted(DESIGN_SIZES))
     args = ap.parse_args()

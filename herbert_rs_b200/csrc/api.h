@@ -238,10 +238,11 @@ int hb_head_gate(int dtype, const void* att, int ld, int hd, const float* gate, 
 int hb_general_delta_prepare(int dtype, const float* rows, int ld, int r_off, int k_off, int a_off, int low_off,
     const void* w2, const float* w0, const float* a0, float decay_c, float unit_eps, float* prep, int n_tokens, int
     heads, int dk, int rank, void* stream);
-int hb_channel_delta_prepare(int dtype, const float* qk, int ldqk, int q_off, int k_off, const float* rows,
-    int ld, int b_off, int low_off, const void* w2, const float* dt_bias, const float* a_log, float unit_eps,
-    float qscale, float* prep, int gate_off, int gate_rank, void* gate_low, int ldgl, int n_tokens, int heads,
-    int qk_heads, int dk, int rank, void* stream);
+int hb_channel_delta_prepare(const float* qk, int ldqk, int q_off, int k_off, const float* z, int ldz, const
+    float* b, int ldb, const float* dt_bias, const float* a_log, float unit_eps, float qscale, float* prep,
+    int n_tokens, int heads, int qk_heads, int dk, void* stream);
+int hb_operand_parts(const float* x, int ld, int fine, int coarse, void* out, int ldo, int n_rows, void*
+    stream);
 int hb_general_delta_scan(const float* prep, const float* v, int ldv, float* state, const int* seq_slot, const int*
     seq_start, float* out, int ldo, int n_seqs, int heads, int dk, int dv, void* stream);
 

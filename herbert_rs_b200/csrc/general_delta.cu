@@ -18,7 +18,9 @@
 // case w = g, u = g * k, a * u -> beta k, k -> beta k.
 //
 //   hb_channel_delta_prepare   that form's vectors, in the same packing, from convolved q and k rows: unit vectors per head
-//                              (q also times a scale), beta = sigmoid(b), g = exp(-exp(A_log) softplus(W2 low + dt_bias))
+//                              (q also times a scale), beta = sigmoid(b), g = exp(-exp(A_log) softplus(W2 low + dt_bias)) from
+//                              the float sums W2 low
+//   hb_operand_parts           float low-rank rows as bfloat16 operands (high and low parts) of the product with W2
 //   hb_general_delta_prepare   from the projection's float rows: the five key-side vectors of every (token, head),
 //                              packed as [T][H][5][dk]: r, k, w, u, a * u
 //   hb_general_delta_scan      the recurrence
@@ -130,117 +132,121 @@ extern "C" int hb_general_delta_prepare(int dtype, const float* rows, int ld, in
 }
 
 // ---------------------------------------------------------------------------------------------
-// The same for the delta rule with a decay per key channel.  Value head h reads query/key head h / (H / G).  The CTAs of
-// head 0 also round the inner row of a low-rank output gate to the compute type, for the product that widens it.
+// The same for the delta rule with a decay per key channel.  Value head h reads query/key head h / (H / G).  The product that
+// widens the decay's low-rank rows has left its float sums; what remains is one warp per (token, head), V channels a lane at a time.
+#define CD_WARPS 8
 struct CdPrepArgs {
   const float* qk; int ldqk; int q_off, k_off;      // convolved rows: [G dk] each
-  const float* rows; int ld; int b_off, low_off;    // the projection's rows: [H] and [rank]
-  const void* w2;                                   // [H dk][rank], compute type
+  const float* z; int ldz;                          // W2 low: [H dk]
+  const float* b; int ldb;                          // [H]
   const float* dt_bias;                             // [H dk]
   const float* a_log;                               // [H]
   float unit_eps, qscale;
   float* prep;                                      // [T][H][5][dk]
-  int gate_off, gate_rank; void* gate_low; int ldgl;      // rows[:, gate_off ..] -> gate_low [T][ldgl]; gate_rank 0: none
-  int n_tokens, H, G, dk, rank;
+  int n_tokens, H, G, dk;
 };
 
-template <typename T>
-__global__ void __launch_bounds__(GP_MAX_THREADS) channel_delta_prepare_kernel(CdPrepArgs a) {
-  extern __shared__ float lows[];   // [GP_TOK][rank]
-  __shared__ float red[2][GP_TOK][GP_MAX_THREADS / 32];
-  __shared__ float coef[3][GP_TOK];           // q's factor, k's factor, beta
+template <int V>
+__global__ void __launch_bounds__(CD_WARPS * 32) channel_delta_prepare_kernel(CdPrepArgs a) {
   pdl_wait();
   pdl_launch();
-  const int t0 = blockIdx.x * GP_TOK, h = blockIdx.y;
-  const int nt = a.n_tokens - t0 < GP_TOK ? a.n_tokens - t0 : GP_TOK;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
+  const int lane = threadIdx.x & 31;
+  const long long unit = (long long)blockIdx.x * CD_WARPS + (threadIdx.x >> 5);
+  if (unit >= (long long)a.n_tokens * a.H) return;
+  const int t = (int)(unit / a.H), h = (int)(unit - (long long)t * a.H);
   const size_t qh = (size_t)(h / (a.H / a.G)) * a.dk;
-  const float* q = a.qk + (size_t)t0 * a.ldqk + a.q_off + qh;
-  const float* k = a.qk + (size_t)t0 * a.ldqk + a.k_off + qh;
-  for (int i = threadIdx.x; i < nt * a.rank; i += blockDim.x) {
-    const int tt = i / a.rank, j = i - tt * a.rank;
-    lows[i] = a.rows[(size_t)(t0 + tt) * a.ld + a.low_off + j];
+  const float* q = a.qk + (size_t)t * a.ldqk + a.q_off + qh;
+  const float* k = a.qk + (size_t)t * a.ldqk + a.k_off + qh;
+  const float* z = a.z + (size_t)t * a.ldz + (size_t)h * a.dk;
+  const float* bias = a.dt_bias + (size_t)h * a.dk;
+  float* out = a.prep + (size_t)unit * 5 * a.dk;
+  auto load = [](float* v, const float* p) {
+    if constexpr (V == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(p);
+      v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+    } else v[0] = p[0];
+  };
+  auto store = [](float* p, const float* v) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else p[0] = v[0];
+  };
+  const float beta = 1.0f / (1.0f + expf(-a.b[(size_t)t * a.ldb + h])), rate = expf(a.a_log[h]);
+  float sq = 0.0f, sk = 0.0f;
+  for (int i = lane * V; i < a.dk; i += 32 * V) {
+    float x[V], y[V];
+    load(x, q + i);
+    load(y, k + i);
+#pragma unroll
+    for (int j = 0; j < V; ++j) { sq = fmaf(x[j], x[j], sq); sk = fmaf(y[j], y[j], sk); }
   }
-  if (h == 0)
-    for (int i = threadIdx.x; i < nt * a.gate_rank; i += blockDim.x) {
-      const int tt = i / a.gate_rank, j = i - tt * a.gate_rank;
-      ((T*)a.gate_low)[(size_t)(t0 + tt) * a.ldgl + j] = from_f32<T>(a.rows[(size_t)(t0 + tt) * a.ld + a.gate_off + j]);
+  const float fq = a.qscale / sqrtf(warp_sum(sq) + a.unit_eps), fk = 1.0f / sqrtf(warp_sum(sk) + a.unit_eps);
+  for (int i = lane * V; i < a.dk; i += 32 * V) {
+    float x[V], y[V], w[V], c[V], g[V], u[V];
+    load(x, q + i);
+    load(y, k + i);
+    load(w, z + i);
+    load(c, bias + i);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float s = w[j] + c[j];
+      g[j] = expf(-rate * (fmaxf(s, 0.0f) + log1pf(expf(-fabsf(s)))));
+      x[j] *= fq;
+      y[j] *= fk;
+      u[j] = g[j] * y[j];
+      y[j] *= beta;
     }
-  float sq[GP_TOK], sk[GP_TOK];
-#pragma unroll
-  for (int tt = 0; tt < GP_TOK; ++tt) sq[tt] = sk[tt] = 0.0f;
-  for (int i = threadIdx.x; i < a.dk; i += blockDim.x) {
-#pragma unroll
-    for (int tt = 0; tt < GP_TOK; ++tt)
-      if (tt < nt) {
-        const float x = q[(size_t)tt * a.ldqk + i], y = k[(size_t)tt * a.ldqk + i];
-        sq[tt] = fmaf(x, x, sq[tt]);
-        sk[tt] = fmaf(y, y, sk[tt]);
-      }
-  }
-#pragma unroll
-  for (int tt = 0; tt < GP_TOK; ++tt) {
-    const float x = warp_sum(sq[tt]), y = warp_sum(sk[tt]);
-    if (lane == 0) { red[0][tt][warp] = x; red[1][tt][warp] = y; }
-  }
-  __syncthreads();
-  if (threadIdx.x < 2 * GP_TOK) {
-    const int which = threadIdx.x / GP_TOK, tt = threadIdx.x % GP_TOK;
-    float v = 0.0f;
-    for (int w = 0; w < nwarp; ++w) v += red[which][tt][w];
-    coef[which][tt] = (which == 0 ? a.qscale : 1.0f) / sqrtf(v + a.unit_eps);
-    if (which == 0 && tt < nt) coef[2][tt] = 1.0f / (1.0f + expf(-a.rows[(size_t)(t0 + tt) * a.ld + a.b_off + h]));
-  }
-  __syncthreads();
-  const T* w2 = (const T*)a.w2;
-  const float rate = expf(a.a_log[h]);
-  for (int i = threadIdx.x; i < a.dk; i += blockDim.x) {
-    const int c = h * a.dk + i;
-    const T* wr = w2 + (size_t)c * a.rank;
-    float z[GP_TOK];
-    const float z0 = a.dt_bias[c];
-#pragma unroll
-    for (int tt = 0; tt < GP_TOK; ++tt) z[tt] = z0;
-    for (int j = 0; j < a.rank; ++j) {
-      const float w = to_f32(wr[j]);
-#pragma unroll
-      for (int tt = 0; tt < GP_TOK; ++tt)
-        if (tt < nt) z[tt] = fmaf(lows[tt * a.rank + j], w, z[tt]);
-    }
-#pragma unroll
-    for (int tt = 0; tt < GP_TOK; ++tt)
-      if (tt < nt) {
-        float* out = a.prep + ((size_t)(t0 + tt) * a.H + h) * 5 * a.dk;
-        const float g = expf(-rate * (fmaxf(z[tt], 0.0f) + log1pf(expf(-fabsf(z[tt])))));
-        const float ku = k[(size_t)tt * a.ldqk + i] * coef[1][tt], bk = coef[2][tt] * ku;
-        out[i] = q[(size_t)tt * a.ldqk + i] * coef[0][tt];
-        out[a.dk + i] = bk;
-        out[2 * a.dk + i] = g;
-        out[3 * a.dk + i] = g * ku;
-        out[4 * a.dk + i] = bk;
-      }
+    store(out + i, x);
+    store(out + a.dk + i, y);
+    store(out + 2 * a.dk + i, g);
+    store(out + 3 * a.dk + i, u);
+    store(out + 4 * a.dk + i, y);
   }
 }
 
-extern "C" int hb_channel_delta_prepare(int dtype, const float* qk, int ldqk, int q_off, int k_off, const float* rows, int ld,
-                                        int b_off, int low_off, const void* w2, const float* dt_bias, const float* a_log,
-                                        float unit_eps, float qscale, float* prep, int gate_off, int gate_rank, void* gate_low,
-                                        int ldgl, int n_tokens, int heads, int qk_heads, int dk, int rank, void* stream) {
-  HB_REQUIRE(n_tokens > 0 && heads > 0 && qk_heads > 0 && dk > 0 && rank > 0, "channel_delta_prepare: sizes must be positive");
+extern "C" int hb_channel_delta_prepare(const float* qk, int ldqk, int q_off, int k_off, const float* z, int ldz, const float* b, int ldb,
+                                        const float* dt_bias, const float* a_log, float unit_eps, float qscale, float* prep,
+                                        int n_tokens, int heads, int qk_heads, int dk, void* stream) {
+  HB_REQUIRE(n_tokens > 0 && heads > 0 && qk_heads > 0 && dk > 0, "channel_delta_prepare: sizes must be positive");
   HB_REQUIRE(heads % qk_heads == 0, "channel_delta_prepare: %d heads are not a multiple of %d query/key heads", heads, qk_heads);
-  const size_t smem = (size_t)GP_TOK * rank * sizeof(float);
-  HB_REQUIRE(smem <= 40 * 1024, "channel_delta_prepare: the decay's inner width %d exceeds what a block keeps in shared memory", rank);
-  HB_REQUIRE(heads <= 65535, "channel_delta_prepare: too many heads");
-  HB_REQUIRE(gate_rank == 0 || (gate_rank > 0 && gate_low != nullptr && ldgl >= gate_rank), "channel_delta_prepare: the gate's inner row needs a place");
-  const CdPrepArgs a{qk, ldqk, q_off, k_off, rows, ld, b_off, low_off, w2, dt_bias, a_log, unit_eps, qscale, prep,
-                     gate_off, gate_rank, gate_low, ldgl, n_tokens, heads, qk_heads, dk, rank};
-  dim3 grid(ceil_div(n_tokens, GP_TOK), heads);
-  const int threads = dk >= GP_MAX_THREADS ? GP_MAX_THREADS : ceil_div(dk, 32) * 32;
-  if (dtype == HB_F32)
-    hb_launch(channel_delta_prepare_kernel<float>, grid, dim3(threads), smem, (cudaStream_t)stream, a);
-  else
-    hb_launch(channel_delta_prepare_kernel<bf16>, grid, dim3(threads), smem, (cudaStream_t)stream, a);
+  const long long blocks = ceil_div_ll((long long)n_tokens * heads, CD_WARPS);
+  HB_REQUIRE(blocks < 2147483647LL, "channel_delta_prepare: too many (token, head) pairs");
+  const CdPrepArgs a{qk, ldqk, q_off, k_off, z, ldz, b, ldb, dt_bias, a_log, unit_eps, qscale, prep, n_tokens, heads, qk_heads, dk};
+  const bool v4 = ((dk | ldqk | q_off | k_off | ldz) & 3) == 0 &&
+                  (((uintptr_t)qk | (uintptr_t)z | (uintptr_t)dt_bias | (uintptr_t)prep) & 15) == 0;
+  if (v4) hb_launch(channel_delta_prepare_kernel<4>, dim3((unsigned)blocks), dim3(CD_WARPS * 32), 0, (cudaStream_t)stream, a);
+  else hb_launch(channel_delta_prepare_kernel<1>, dim3((unsigned)blocks), dim3(CD_WARPS * 32), 0, (cudaStream_t)stream, a);
   HB_CHECK_LAUNCH("channel_delta_prepare");
+  return 0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// Float columns of a row as operands of a bfloat16 product: the first `fine` columns as a high and a low part (about 16
+// bits of them reach the product when its matrix holds their weights twice), the next `coarse` ones rounded once, zeros
+// up to the row's end:   out[t] = [high(fine) | low(fine) | coarse | 0].
+__global__ void __launch_bounds__(256)
+operand_parts_kernel(const float* __restrict__ x, int ld, int fine, int coarse, bf16* __restrict__ out, int ldo, long long total) {
+  pdl_wait();
+  pdl_launch();
+  const long long at = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (at >= total) return;
+  const int t = (int)(at / ldo), c = (int)(at - (long long)t * ldo);
+  const float* row = x + (size_t)t * ld;
+  bf16 r = __float2bfloat16_rn(0.0f);
+  if (c < fine) r = __float2bfloat16_rn(row[c]);
+  else if (c < 2 * fine) {
+    const float v = row[c - fine];
+    r = __float2bfloat16_rn(v - __bfloat162float(__float2bfloat16_rn(v)));
+  } else if (c < 2 * fine + coarse) r = __float2bfloat16_rn(row[c - fine]);
+  out[at] = r;
+}
+
+extern "C" int hb_operand_parts(const float* x, int ld, int fine, int coarse, void* out, int ldo, int n_rows, void* stream) {
+  HB_REQUIRE(n_rows > 0 && fine >= 0 && coarse >= 0 && fine + coarse > 0 && ld >= fine + coarse, "operand_parts: sizes must be positive");
+  HB_REQUIRE(ldo >= 2 * fine + coarse, "operand_parts: rows of %d have no room for 2 x %d and %d columns", ldo, fine, coarse);
+  const long long total = (long long)n_rows * ldo, blocks = ceil_div_ll(total, 256);
+  HB_REQUIRE(blocks < 2147483647LL, "operand_parts: too many elements");
+  hb_launch(operand_parts_kernel, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, x, ld, fine, coarse, (bf16*)out, ldo, total);
+  HB_CHECK_LAUNCH("operand_parts");
   return 0;
 }
 

@@ -658,6 +658,69 @@ gated_rmsnorm_kernel(const float* __restrict__ o, int ldo, int o_stride, const f
   }
 }
 
+// The same with one warp per (token, unit), for units of at most 128 GN_PIECES numbers in steps of four: no barrier, and
+// a CTA's eight units go their own ways.
+#define GN_WARPS 8
+#define GN_PIECES 4
+template <typename T>
+__global__ void __launch_bounds__(GN_WARPS * 32)
+gated_rmsnorm_warp_kernel(const float* __restrict__ o, int ldo, int o_stride, const float* __restrict__ w, float eps, const float* __restrict__ gate,
+                          int ldg, T* __restrict__ y, int ldy, int units, int n, int act, int w_stride, int gate_first, HeadDivide hd, long long total) {
+  pdl_wait();
+  pdl_launch();
+  const int lane = threadIdx.x & 31;
+  const long long unit = (long long)blockIdx.x * GN_WARPS + (threadIdx.x >> 5);
+  if (unit >= total) return;
+  const int t = (int)(unit / units), u = (int)(unit - (long long)t * units);
+  const float* orow = o + (size_t)t * ldo + (size_t)u * o_stride;
+  const float* g = gate + (size_t)t * ldg + (size_t)u * n;
+  w += (size_t)u * w_stride;
+  T* yr = y + (size_t)t * ldy + (size_t)u * n;
+  float4 v[GN_PIECES], ga[GN_PIECES];
+#pragma unroll
+  for (int q = 0; q < GN_PIECES; ++q) {
+    const int i = (lane + 32 * q) * 4;
+    if (i >= n) continue;
+    v[q] = *reinterpret_cast<const float4*>(orow + i);
+    ga[q] = *reinterpret_cast<const float4*>(g + i);
+  }
+  const float pre = hd.floor_ ? hd.scale / (fmaxf(fabsf(hd.scale * orow[n]), hd.floor_[unit]) + hd.eps) : 1.0f;
+  auto gate_of = [&](float gv) {
+    const float sg = sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(-gv)) : 1.0f / (1.0f + expf(-gv));
+    return act == 0 ? gv * sg : sg;
+  };
+  float s = 0.0f;
+#pragma unroll
+  for (int q = 0; q < GN_PIECES; ++q) {
+    if ((lane + 32 * q) * 4 >= n) continue;
+    ga[q] = make_float4(gate_of(ga[q].x), gate_of(ga[q].y), gate_of(ga[q].z), gate_of(ga[q].w));
+    v[q] = make_float4(v[q].x * pre, v[q].y * pre, v[q].z * pre, v[q].w * pre);
+    if (gate_first) {
+      v[q] = make_float4(v[q].x * ga[q].x, v[q].y * ga[q].y, v[q].z * ga[q].z, v[q].w * ga[q].w);
+      ga[q] = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+    }
+    s += (v[q].x * v[q].x + v[q].y * v[q].y) + (v[q].z * v[q].z + v[q].w * v[q].w);
+  }
+  const float k = 1.0f / sqrtf(warp_sum(s) / (float)n + eps);
+#pragma unroll
+  for (int q = 0; q < GN_PIECES; ++q) {
+    const int i = (lane + 32 * q) * 4;
+    if (i >= n) continue;
+    const float4 w4 = *reinterpret_cast<const float4*>(w + i);
+    const float r0 = ((v[q].x * k) * w4.x) * ga[q].x, r1 = ((v[q].y * k) * w4.y) * ga[q].y;
+    const float r2 = ((v[q].z * k) * w4.z) * ga[q].z, r3 = ((v[q].w * k) * w4.w) * ga[q].w;
+    if constexpr (sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(yr + i) = make_float4(r0, r1, r2, r3);
+    } else {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(r0, r1), hi = __floats2bfloat162_rn(r2, r3);
+      uint2 pk;
+      pk.x = *reinterpret_cast<const unsigned*>(&lo);
+      pk.y = *reinterpret_cast<const unsigned*>(&hi);
+      *reinterpret_cast<uint2*>(yr + i) = pk;
+    }
+  }
+}
+
 extern "C" int hb_gated_rmsnorm(int dtype, const float* o, int ldo, int o_stride, const float* w, float eps, const float* gate, int ldg,
                                 void* y, int ldy, int n_tokens, int units, int n, int act, int w_stride, int gate_first,
                                 const float* floor_, float div_scale, float div_eps, void* stream) {
@@ -668,6 +731,18 @@ extern "C" int hb_gated_rmsnorm(int dtype, const float* o, int ldo, int o_stride
   const HeadDivide hd{floor_, div_scale, div_eps};
   const long long blocks = (long long)n_tokens * units;
   HB_REQUIRE(blocks < 2147483647LL, "gated_rmsnorm: too many (token, unit) pairs");
+  if (units > 1 && n % 4 == 0 && n <= 128 * GN_PIECES && ((ldo | ldg | ldy | o_stride) & 3) == 0 &&
+      (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)y | (uintptr_t)w) & 15) == 0) {
+    const dim3 grid((unsigned)ceil_div_ll(blocks, GN_WARPS));
+    if (dtype == HB_F32)
+      hb_launch(gated_rmsnorm_warp_kernel<float>, grid, dim3(GN_WARPS * 32), 0, (cudaStream_t)stream, o, ldo, o_stride, w, eps, gate, ldg,
+                (float*)y, ldy, units, n, act, w_stride, gate_first, hd, blocks);
+    else
+      hb_launch(gated_rmsnorm_warp_kernel<bf16>, grid, dim3(GN_WARPS * 32), 0, (cudaStream_t)stream, o, ldo, o_stride, w, eps, gate, ldg,
+                (bf16*)y, ldy, units, n, act, w_stride, gate_first, hd, blocks);
+    HB_CHECK_LAUNCH("gated_rmsnorm");
+    return 0;
+  }
   const int threads = n >= 1024 ? 256 : n >= 128 ? 128 : (n >= 64 ? 64 : 32);
   if (dtype == HB_F32)
     hb_launch(gated_rmsnorm_kernel<float>, dim3((unsigned)blocks), dim3(threads), 0, (cudaStream_t)stream, o, ldo, o_stride, w, eps, gate,

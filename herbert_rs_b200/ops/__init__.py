@@ -144,9 +144,9 @@ _SIGS = {
     "hb_gated_norm_residual": [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
                                c_float, c_void_p, c_int, c_int, c_void_p],
     "hb_token_gate": [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-    "hb_channel_delta_prepare": [c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
-                                 c_void_p, c_float, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                 c_int, c_void_p],
+    "hb_channel_delta_prepare": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                                 c_float, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "hb_operand_parts": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
     "hb_matrix_memory_prepare": [c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
                                  c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                  c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -814,23 +814,27 @@ def general_delta_scan(prep, v, state, batch, out, heads, dk, dv) -> None:
          batch.seq_start.data_ptr(), out.data_ptr(), out.stride(0), batch.n_seqs, int(heads), int(dk), int(dv), _stream())
 
 
-def channel_delta_prepare(qk, q_off, k_off, rows, b_off, low_off, w2, dt_bias, a_log, unit_eps, qscale, prep, heads, qk_heads, dk,
-                          gate_off=0, gate_low=None) -> None:
+def channel_delta_prepare(qk, q_off, k_off, z, b, dt_bias, a_log, unit_eps, qscale, prep, heads, qk_heads, dk) -> None:
     """The delta rule with a decay per key channel, for `general_delta_scan`: from float rows qk (q and k, qk_heads * dk numbers
-    each) and rows (b: one number per head, low: the decay's inner row of w2.shape[1] numbers): prep [T, heads, 5, dk] = q' , beta k',
-    g, g k', beta k' with unit vectors x / sqrt(sum x^2 + unit_eps) per head, q' also times qscale, beta = sigmoid(b),
-    g = exp(-exp(a_log) softplus(w2 low + dt_bias)).  `gate_low` [T, r], if given, receives rows[:, gate_off : gate_off + r] in its dtype."""
-    for t, n in ((qk, "qk"), (rows, "rows"), (dt_bias, "dt_bias"), (a_log, "a_log"), (prep, "prep")):
+    each, at their offsets), z [T, heads * dk] and b [T, heads]: prep [T, heads, 5, dk] = q', beta k', g, g k', beta k' with unit vectors
+    x / sqrt(sum x^2 + unit_eps) per head, q' also times qscale, beta = sigmoid(b), g = exp(-exp(a_log) softplus(z + dt_bias))."""
+    for t, n in ((qk, "qk"), (z, "z"), (b, "b"), (dt_bias, "dt_bias"), (a_log, "a_log"), (prep, "prep")):
         _check(t, torch.float32, n)
-    _check(w2, None, "w2")
-    if not (w2.is_contiguous() and prep.is_contiguous()) or w2.shape[0] != heads * dk:
-        raise BackendError("channel_delta_prepare: w2 must be [heads * dk, rank] and contiguous, prep contiguous")
-    if gate_low is not None:
-        _check(gate_low, w2.dtype, "gate_low")
-    _run("hb_channel_delta_prepare", dtype_code(w2.dtype), qk.data_ptr(), qk.stride(0), int(q_off), int(k_off), rows.data_ptr(),
-         rows.stride(0), int(b_off), int(low_off), w2.data_ptr(), dt_bias.data_ptr(), a_log.data_ptr(), float(unit_eps), float(qscale),
-         prep.data_ptr(), int(gate_off), 0 if gate_low is None else gate_low.shape[1], _ptr(gate_low),
-         0 if gate_low is None else gate_low.stride(0), qk.shape[0], int(heads), int(qk_heads), int(dk), w2.shape[1], _stream())
+    if not prep.is_contiguous() or tuple(prep.shape) != (qk.shape[0], heads, 5, dk) or z.shape[1] != heads * dk or b.shape[1] != heads:
+        raise BackendError(f"channel_delta_prepare: prep must be a contiguous [{qk.shape[0]}, {heads}, 5, {dk}] array, z and b of its heads")
+    _run("hb_channel_delta_prepare", qk.data_ptr(), qk.stride(0), int(q_off), int(k_off), z.data_ptr(), z.stride(0), b.data_ptr(), b.stride(0),
+         dt_bias.data_ptr(), a_log.data_ptr(), float(unit_eps), float(qscale), prep.data_ptr(), qk.shape[0], int(heads), int(qk_heads),
+         int(dk), _stream())
+
+
+def operand_parts(x, fine, coarse, out) -> None:
+    """Float columns x [T, fine + coarse] as bfloat16 operands: out[t] = [high part of the first `fine` columns | their low part |
+    the next `coarse` columns rounded | zeros]; a matrix that holds the weights of the fine columns twice multiplies about 16 bits
+    of them."""
+    _check(x, torch.float32, "x"); _check(out, torch.bfloat16, "out")
+    if not out.is_contiguous() or x.shape[1] != fine + coarse:
+        raise BackendError("operand_parts: out must be contiguous, x have the fine and the coarse columns")
+    _run("hb_operand_parts", x.data_ptr(), x.stride(0), int(fine), int(coarse), out.data_ptr(), out.stride(0), x.shape[0], _stream())
 
 
 def matrix_memory_prepare(rows, q_off, k_off, v_off, i_off, f_off, i_bias, f_bias, cap, m_state, batch, packed, logd, weight, floor,

@@ -9,8 +9,9 @@ corrected toward the token's value along its key, and read with the query.
 
 conv is a short causal convolution over time on each channel whose last taps - 1 inputs are kept per sequence, beside the state
 matrix, in the cache's fixed-size region of the sequence's slot.  The six products that read h are one matrix (rows q, k, v, A1, G1,
-b) that leaves float sums; unit vectors, beta, decays (with the product A2), the state and the norm are float on both paths.  The
-recurrence is the generalised delta rule's (`ops.general_delta_scan`), of which this is a case.
+b) that leaves float sums; unit vectors, beta, decays, the state and the norm are float on both paths.  A2 and G2 are one matrix too,
+over the inner rows of both; on the bfloat16 path A1 h enters it as a high and a low part, so that about 16 bits of it reach the
+decay.  The recurrence is the generalised delta rule's (`ops.general_delta_scan`), of which this is a case.
 """
 
 from __future__ import annotations
@@ -71,13 +72,21 @@ class ChannelDeltaMixer(Mixer):
         self.rank, self.gate_rank = t[n["decay_down"]].shape[0], t[n["gate_down"]].shape[0]
         self.w_in = stack_rows([t[n[r]] for r in ("q", "k", "v", "decay_down", "gate_down", "beta")])
         self.w_conv = torch.cat([t[n["q"] + c], t[n["k"] + c], t[n["v"] + c]], dim=0).contiguous()
-        self.w_decay, self.w_gate = t[n["decay_up"]].contiguous(), t[n["gate_up"]].contiguous()
+        # [A2 | 0; 0 | G2] over [A1 h | G1 h]; bfloat16: [A2 | A2 | 0; 0 | 0 | G2] over [high | low | G1 h], a multiple of 8 columns
+        decay, gate = t[n["decay_up"]], t[n["gate_up"]]
+        self.parts = 2 if self.rt.dtype == torch.bfloat16 else 1
+        columns = self.parts * self.rank + self.gate_rank
+        self.w_low = torch.zeros((decay.shape[0] + gate.shape[0], (columns + 7) // 8 * 8 if self.parts > 1 else columns), dtype=decay.dtype,
+                                 device=decay.device)
+        for p in range(self.parts):
+            self.w_low[:decay.shape[0], p * self.rank:(p + 1) * self.rank] = decay
+        self.w_low[decay.shape[0]:, self.parts * self.rank:columns] = gate
         self.a_log, self.dt_bias = t[n["A_log"]].contiguous(), t[n["dt_bias"]].contiguous()
         self.norm = t[n["norm"]].contiguous()
         self.w_out = t[n["out"]].contiguous()
 
     def weight_bytes(self):
-        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_conv, self.w_decay, self.w_gate, self.w_out))
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_conv, self.w_low, self.w_out))
 
     def cache_need(self):
         states = ()
@@ -91,19 +100,22 @@ class ChannelDeltaMixer(Mixer):
         proj = ws.take((T, self.w_in.shape[0]), f32)
         ops.gemm(h, self.w_in, proj, ops.EPI_STORE_F32, scratch=ws.take)
         C = self.conv_channels
-        v_off, low_off, gate_off, b_off = 2 * G * dk, C, C + self.rank, C + self.rank + self.gate_rank
+        v_off, low_off, b_off = 2 * G * dk, C, C + self.rank + self.gate_rank
         qkv = ws.take((T, C), f32)
         ops.short_conv(proj[:, :C], self.w_conv, cache.states.get("conv"), batch, qkv, add_input=False, silu=True)
+        low = proj[:, low_off:b_off]
+        if self.parts > 1:
+            low = ws.take((T, self.w_low.shape[1]), h.dtype)
+            ops.operand_parts(proj[:, low_off:b_off], self.rank, self.gate_rank, low)
+        wide = ws.take((T, self.w_low.shape[0]), f32)
+        ops.gemm(low, self.w_low, wide, ops.EPI_STORE_F32, scratch=ws.take)
         prep = ws.take((T, H, 5, dk), f32)
-        low = ws.take((T, self.gate_rank), h.dtype)
-        ops.channel_delta_prepare(qkv, 0, G * dk, proj, b_off, low_off, self.w_decay, self.dt_bias, self.a_log, s.unit_eps, dk ** -0.5,
-                                  prep, H, G, dk, gate_off=gate_off, gate_low=low)
-        gate = ws.take((T, H * dv), f32)
-        ops.gemm(low, self.w_gate, gate, ops.EPI_STORE_F32, scratch=ws.take)
+        ops.channel_delta_prepare(qkv, 0, G * dk, wide[:, :H * dk], proj[:, b_off:b_off + H], self.dt_bias, self.a_log, s.unit_eps,
+                                  dk ** -0.5, prep, H, G, dk)
         o = ws.take((T, H * dv), f32)
         ops.general_delta_scan(prep, qkv[:, v_off:], cache.state, batch, o, H, dk, dv)
         y = ws.take((T, H * dv), h.dtype)
-        ops.gated_rmsnorm(o, self.norm, s.norm_eps, gate, y, H, dv, sigmoid_gate=True)
+        ops.gated_rmsnorm(o, self.norm, s.norm_eps, wide[:, H * dk:], y, H, dv, sigmoid_gate=True)
         ops.gemm(y, self.w_out, residual, ops.EPI_RESIDUAL if accumulate else ops.EPI_STORE_F32, scratch=ws.take)
 
 
