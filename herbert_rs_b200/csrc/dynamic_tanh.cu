@@ -16,6 +16,13 @@ struct TanhNorm {
   void* out;           // null: not asked for
 };
 
+// tanh in float; where the result is rounded to bfloat16 next, as 1 - 2 / (1 + e^{2z}) with the fast exponential and
+// division (absolute error about 1e-7; e^{2z} = inf gives 1, 0 gives -1).
+template <typename T> __device__ __forceinline__ float tanh_of(float z) {
+  if constexpr (sizeof(T) == 4) return tanhf(z);
+  else return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * z));
+}
+
 // V: channels per thread (4: every pointer on 16 bytes and every row length a multiple of 4).
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
@@ -55,7 +62,7 @@ residual_tanh_kernel(const float* __restrict__ y, int ldy, const float* __restri
     load(w, n.w + c);
     load(b, n.b + c);
 #pragma unroll
-    for (int j = 0; j < V; ++j) o[j] = fmaf(tanhf(n.alpha * v[j]), w[j], b[j]);
+    for (int j = 0; j < V; ++j) o[j] = fmaf(tanh_of<T>(n.alpha * v[j]), w[j], b[j]);
     T* p = (T*)n.out + (size_t)r * dim + c;
     if constexpr (V == 4 && sizeof(T) == 2) {
       const __nv_bfloat162 lo = __floats2bfloat162_rn(o[0], o[1]), hi = __floats2bfloat162_rn(o[2], o[3]);
