@@ -481,8 +481,10 @@ def _launcher_work(name, n, ctx):
             return n * 9.0 * T * dh * dn * dw, n * (T * dh * (5 * dn + 2 * dw) * 4 + 2 * B * dh * dn * dw * 4)
         if name == "hb_channel_delta_prepare":
             return n * 8.0 * T * dh * dn, n * T * (2 * dg * dn + 6 * dh * dn + dh) * 4
-        if name == "hb_residual_tanh":      # one per layer updates the stream and leaves two norms; the first and the last only read
-            return n * 8.0 * T * D, n * T * D * (4 + 4 + 4 + 2 * es)
+        if name == "hb_residual_tanh":
+            # one per layer updates the stream and (but for the last layer) leaves two norms; the first launch only reads and
+            # leaves two, the last one norms the rows whose logits are asked for
+            return n * 8.0 * T * D, (n - 3) * T * D * (12 + 2 * es) + T * D * 12 + T * D * (4 + 2 * es)
         if name == "hb_short_conv":
             return n * 8.0 * T * conv, n * T * conv * 8
         if name == "hb_qkv_rotary_cache":
